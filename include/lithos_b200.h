@@ -190,12 +190,10 @@ int lb_gemv_chain_supports(lb_ctx* ctx, int K, int N, int swiglu);
 /* Batched projection: Y[B,N] = X[B,K] W for B = 1..LB_GEMM_MAX_BATCH tokens, W in the same three GPTQ
  * buffers as lb_gemv_int4 (read once for the whole batch), x fp16 [B,K] row-major, y fp32 [B,N]
  * (flags = LB_GEMV_Y_F32) or fp16 [B,N] (flags = 0).  K % 128 == 0, N % 16 == 0.
- * The reference's batched path is its prefill projection (kernels/projection_gemm.sass:390-631:
- * int4 -> fp16 dequantisation into shared memory, eight 16x8x16 tensor-core products per k-step);
  * One token is handed to the GEMV kernel of lb_gemv_int4.
  * 33..256 tokens run on the 5th-generation tensor cores (tcgen05.mma, accumulators in tensor memory):
- * the weights are dequantised to fp16 - (q - z) * s, q - z exact, one fp16 rounding for the scale - as the
- * reference kernel does, and handed to the tensor cores through tensor memory (129..256 tokens: one
+ * the weights are dequantised to fp16 - (q - z) * s, q - z exact, one fp16 rounding for the scale -
+ * and handed to the tensor cores through tensor memory (129..256 tokens: one
  * product of 128 columns x 256 tokens per k step, the weights converted once for all of them).  Up to 32 tokens use mma.sync (faster there, measured):
  * q - z stays exact and the group scale multiplies the group's fp32 sum, so row b of Y equals
  * lb_gemv_int4 on row b of X to fp32 rounding.  LB_GEMM_TCGEN05 forces the tensor-memory kernel for
@@ -370,7 +368,7 @@ int lb_model_reset_state(lb_model* m); /* zero DeltaNet states, conv history and
 int lb_model_state_ptr(lb_model* m, int layer, int which, uint64_t* dptr_out, size_t* bytes_out);
 /* Snapshot / restore of the recurrent state (every DeltaNet layer's state matrix and convolution history), for
  * speculative decoding: decode ahead, then lb_model_rollback and continue from the checkpointed position.
- * Replaces the reference's state_rollback copy kernel (inference/recur.ls:82-86, kernels/recurrence_rollback.sass).
+ * Replaces the reference's state_rollback copy kernel (inference/recur.ls:82-86).
  * Stream-ordered device-to-device copies; the KV caches are not copied (rows past the position are never read).
  * LB_ERR_STATE from lb_model_rollback when no checkpoint was taken. */
 int lb_model_checkpoint(lb_model* m);
@@ -392,8 +390,7 @@ int lb_model_read_next(lb_model* m, int* next_out);   /* synchronises */
  * the state a token-by-token lb_model_decode of the same tokens leaves (DeltaNet states, convolution rings, KV rows);
  * *next_out (may be NULL) receives the greedy token that follows the prompt, the logits of the last prompt token are
  * in lb_model_logits_ptr, and lb_model_replay / lb_model_decode continue from position pos0+n.  Every projection of a
- * chunk is one lb_gemm_int4 call (the reference's prompt path is its dequantising tensor-core GEMM,
- * kernels/projection_gemm.sass:390-631; layer order compiler/megakernel-link.ls:281-525), the recurrence keeps the state
+ * chunk is one lb_gemm_int4 call (layer order compiler/megakernel-link.ls:281-525), the recurrence keeps the state
  * on chip for the chunk, attention is one causal tensor-core kernel per chunk.  Up to four chunks are in flight on
  * streams of the library's own (a layer of a chunk waits for the same layer of the chunk before it); they start behind
  * what the context's stream holds when the call is made and the context's stream continues behind them.  The first call

@@ -4,8 +4,10 @@
 // kernel and inference/reduce.ls:85-147 compute it; activations fp32, weight bf16 (the launcher
 // hands over the checkpoint tensor, src/launcher.s:140-141).
 #include <stdint.h>
-// "norm" is also a CUDA math function with C linkage: the build renames compat_entry_norm to norm.
-extern "C" __global__ void __launch_bounds__(256) compat_entry_norm(const float* __restrict__ x, const float* __restrict__ res,
+// "norm" is also a CUDA math function with C linkage.  The build compiles this file with the header's declaration renamed by a
+// preprocessor macro (see the Makefile), which ends here, so that the kernel can have the name.
+#undef norm
+extern "C" __global__ void __launch_bounds__(256) norm(const float* __restrict__ x, const float* __restrict__ res,
                                                        const uint16_t* __restrict__ w, float* __restrict__ y,
                                                        uint32_t D, float eps) {
     __shared__ float red[33];

@@ -1,8 +1,8 @@
-// Drop-in for the reference's sampling kernel (kernels/README.md:104-117, kernels/sample.sass): file
+// Drop-in for the reference's sampling kernel (kernels/README.md:104-117): file
 // sample.cubin, entry sample, parameters (u64 logits_f32, u64 output_token_u32, u32 vocab_size,
-// f32 temperature, u32 top_k), grid 1 x 256.  The reference kernel scales every logit by 1/temperature
-// and takes the arg-max with a strict ">" (inference/reduce.ls:214-313); it reads top_k and never
-// uses it.  Same here, with the tie rule of the launcher's own CPU loop (src/launcher.s:1060-1063):
+// f32 temperature, u32 top_k), grid 1 x 256.  Every logit is scaled by 1/temperature
+// and the arg-max taken with a strict ">" (inference/reduce.ls:214-313); top_k is accepted and not
+// used.  The tie rule is that of the launcher's own CPU loop (src/launcher.s:1060-1063):
 // the first maximum wins.  temperature <= 0 is taken as 1.  Only block 0 works, whatever the grid.
 #include <stdint.h>
 extern "C" __global__ void __launch_bounds__(1024) sample(const float* logits, uint32_t* out_token, uint32_t vocab, float temperature,

@@ -118,7 +118,7 @@ LB_API int lb_model_reset_state(lb_model* m) {
 }
 
 /* Checkpoint / rollback of the recurrent state: the reference's state_rollback kernel is an element-wise copy
- * state[i] = checkpoint[i] (inference/recur.ls:82-86, kernels/recurrence_rollback.sass).  Here both directions
+ * state[i] = checkpoint[i] (inference/recur.ls:82-86).  Here both directions
  * are device-to-device copies of every DeltaNet layer's state matrix and convolution history on the context
  * stream (ordered with the decode steps around them).  The KV caches need no copy: a row is rewritten when
  * its position is decoded again, and rows past the current position are never read. */

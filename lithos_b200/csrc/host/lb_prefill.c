@@ -2,8 +2,7 @@
  * token-by-token decode of the same tokens leaves (DeltaNet states, convolution rings, KV rows), then samples the token
  * that follows the prompt.
  *
- * The reference's prompt path is its dequantising tensor-core GEMM (kernels/projection_gemm.sass:390-631) in the layer
- * order of compiler/megakernel-link.ls:281-525.  Here every projection of a chunk is one lb_gemm_int4 call (the weights
+ * The layer order is that of compiler/megakernel-link.ls:281-525.  Every projection of a chunk is one lb_gemm_int4 call (the weights
  * are read once per chunk: tcgen05 for 33..256 tokens), the DeltaNet recurrence walks the chunk's tokens inside one
  * launch with the state held on chip (lb_deltanet_step, n_steps = chunk), and attention is two launches per chunk: the
  * per-token part (norm, RoPE, KV append) with the decode kernel's own routine, then one causal tensor-core kernel over

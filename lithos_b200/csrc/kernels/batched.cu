@@ -15,8 +15,7 @@
 //   * Up to 32 tokens: products of a 5-bit integer and an fp16 value are exact in the fp32 accumulator; the
 //     fp16 group scale multiplies the group's fp32 sum, so no weight is ever rounded.  33..64 tokens (one
 //     warp keeps all 64 tokens' accumulators, so there is no room for per-group sums): the A registers are
-//     (q - z) * s rounded to fp16, the dequantised weight the reference's own batched kernel multiplies
-//     (kernels/projection_gemm.sass:477-631).
+//     (q - z) * s rounded to fp16.
 //   * The CTA is 8 warps = 8 column sets (128 columns).  Packed words
 //     are prefetched three or four K-groups ahead in registers; the activations travel K-group by K-group through a
 //     cp.async ring of as many stages in shared memory (16-byte chunks; rows of 320 bytes, so that the 128-bit

@@ -1,15 +1,14 @@
 // Batched int4 projection on the 5th-generation tensor cores (tcgen05 + TMEM) for 9..128 tokens on sm_100a:
 // Y[b][n] = sum_k W(k,n) X[b][k], W in the GPTQ buffers of the batch-1 GEMV (qweight [K/8,N], scales fp16
 // [K/128,N], qzeros [K/128,N/8] or NULL = zero-point 8; inference/gemv.ls:44-130), X fp16 [B,K],
-// Y fp32 or fp16 [B,N].  The reference's batched kernel is kernels/projection_gemm.sass:390-631
-// (int4 -> fp16 into shared memory, then 16x8x16 tensor-core products); the product here is one
+// Y fp32 or fp16 [B,N].  The product is one
 // tcgen05.mma of 128 weight columns x NT tokens x 16 k per instruction, accumulated in tensor memory.
 //
 // One CTA = 128 output columns x one K slice: 16 dequantising warps, one issuing thread, one activation thread.
 // Per K-group (128 k):
 //   * every dequantising thread converts 4 packed words of one column (prefetched four groups earlier): a packed
 //     word is 8 consecutive k of one column, so its eight fp16 values (q - z) * s - q - z exact through the 0x6400
-//     exponent trick, then one fp16 multiply: the weight the reference kernel multiplies - are one 16-byte
+//     exponent trick, then one fp16 multiply - are one 16-byte
 //     shared-memory store into the K-major operand tile with the 128-byte swizzle: two halves of 64 k, a row of
 //     128 bytes per column, 16-byte slot (chunk % 8) ^ (column % 8) inside the row;
 //   * the activations of the group arrive by two tiled TMA loads (64 k x NT tokens each, 128-byte swizzle by the

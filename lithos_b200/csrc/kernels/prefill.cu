@@ -1,6 +1,5 @@
 // Prompt pass (prefill): the small kernels between the batched int4 projections (gemm_int4_*) when a chunk of up to 128
-// prompt tokens goes through a layer at once.  The reference's prefill path is its dequantising GEMM
-// (kernels/projection_gemm.sass:390-631) around the same element-wise / recurrence kernels as decoding
+// prompt tokens goes through a layer at once.  The layers run the same element-wise / recurrence kernels as decoding
 // (compiler/megakernel-link.ls:281-525 layer order); here every kernel takes a chunk [T, ...] and leaves exactly the
 // state a token-by-token decode of the same tokens leaves: DeltaNet state, convolution ring (slot = position & 3), KV rows.
 // All activations are fp32 except the projection inputs, which are rounded to fp16 (the decode step's contract).

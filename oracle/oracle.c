@@ -285,7 +285,7 @@ ORC_API void orc_silu(const float* x, float* y, int n) {
     for (int i = 0; i < n; i++) y[i] = siluf_(x[i]);
 }
 /* SwiGLU: silu(gate)*up (kernels.ls:61-66); swap_operands=1 gives the
- * shipped SASS variant gate*silu(up) (kernels/activate.sass) */
+ * variant gate*silu(up) (kernels/README.md:69) */
 ORC_API void orc_swiglu(const float* gate, const float* up, float* y, int n, int swap_operands) {
     for (int i = 0; i < n; i++) y[i] = swap_operands ? gate[i] * siluf_(up[i]) : siluf_(gate[i]) * up[i];
 }
@@ -389,7 +389,7 @@ ORC_API void orc_rope(float* x /*[heads,d] in place*/, int heads, int d, int rot
 /* (gate) as attend_full.ls:236-248.  K,V bf16, fp32 maths.             */
 /* compat: the launcher's table-driven half-split rotation.  Tables as precompute_rope_tables fills them
  * (src/launcher.s:3139-3148): t[p * half + i] = cosf / sinf(p * expf(-i * ln(theta) / half)), float32 libm calls;
- * rotation of pair (i, i + d/2) over the whole head (src/launcher.s:2260-2272, kernels/rotate.sass). */
+ * rotation of pair (i, i + d/2) over the whole head (src/launcher.s:2260-2272). */
 ORC_API void orc_rope_tables(float* cos_t, float* sin_t, int n_pos, int half, float theta) {
     const float step = logf(theta) / (float)half;
     for (int p = 0; p < n_pos; p++)

@@ -111,8 +111,7 @@ def test_prefill_single_token_and_continuation(ctx, lb, oracle):
 
 def test_prefill_full_width_layers(ctx, lb, oracle):
     """four layers at the benchmark's widths (hidden 5120, SwiGLU 17408, 48/16 and 24/4 heads), 64-token prompt: the tcgen05
-    projections on 64 tokens.  That kernel multiplies weights dequantised to fp16, (q - z) * s rounded once, as the
-    reference's prompt GEMM does (kernels/projection_gemm.sass:390-631), so every projection carries a 2^-11 weight rounding
+    projections on 64 tokens.  That kernel multiplies weights dequantised to fp16, (q - z) * s rounded once, so every projection carries a 2^-11 weight rounding
     the token-by-token path does not have; tokens and logits stay inside 2e-3, the recurrent state after 64 accumulated
     updates is allowed 4e-3 (measured 2.2e-3)."""
     from lithos_b200 import model as M
