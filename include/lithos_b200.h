@@ -47,6 +47,9 @@ const char* lb_version(void);
  * Unlike the reference, a cubin or entry point that cannot be found is an
  * error here (the launcher stores NULL and skips every launch of it). */
 int lb_init(int device, const char* kernel_dir, lb_ctx** out);
+/* the same with only the named kernel images (lb_config_images gives a model's; names without .cubin, separated by blanks):
+ * launching a kernel of an image left out is an error */
+int lb_init_images(int device, const char* kernel_dir, const char* images, lb_ctx** out);
 void lb_destroy(lb_ctx* ctx);
 const char* lb_last_error(const lb_ctx* ctx);
 int lb_device_sm_count(const lb_ctx* ctx);
@@ -396,6 +399,11 @@ int lb_model_read_next(lb_model* m, int* next_out);   /* synchronises */
  * what the context's stream holds when the call is made and the context's stream continues behind them.  The first call
  * allocates the chunks' buffers (about 90 MB each at the 27B widths).  Single GPU (tp_size 1) only. */
 int lb_model_prefill(lb_model* m, const int* tokens, int n, int pos0, int* next_out);
+/* The same pass without sampling: tokens[0..n) at positions pos0..pos0+n-1 through the model; logits_out [n_want, vocab] (host)
+ * receives the logits at the places want[0..n_want) of the portion (ascending; n_want may be 0).  A portion may be cut anywhere.
+ * One token (n == 1) runs as the captured decode step.  Synchronises.  Single GPU only. */
+int lb_model_forward(lb_model* m, const int* tokens, int n, int pos0, const int* want, int n_want, float* logits_out);
+const char* lb_model_arch_name(const lb_model* m);
 int lb_model_step_kernels(const lb_model* m);         /* kernels per decode step */
 /* top_k == 0 (default): greedy; else every step samples among the top_k largest logits at `temperature`, the draw being a
  * function of (seed, position).  Takes effect at the next lb_model_decode / lb_model_capture.  Single GPU only. */

@@ -127,9 +127,14 @@ static int load_cubin(lb_ctx* c, const char* dir, const char* file) {
     return LB_OK;
 }
 
-static const char* const k_cubins[] = {"gemv.cubin", "chain.cubin", "batched.cubin", "batched_tc.cubin", "deltanet.cubin", "attention.cubin", "attention_mma.cubin", "small.cubin", "comm.cubin", "prefill.cubin"};
+static const char* const k_cubins[] = {"gemv.cubin", "chain.cubin", "batched.cubin", "batched_tc.cubin", "deltanet.cubin", "attention.cubin", "attention_mma.cubin", "small.cubin", "comm.cubin", "prefill.cubin",
+                                       "rows_gemv.cubin", "dense_gemm.cubin", "window_attention.cubin", "decay_attention.cubin"};
 
-LB_API int lb_init(int device, const char* kernel_dir, lb_ctx** out) {
+LB_API int lb_init(int device, const char* kernel_dir, lb_ctx** out) { return lb_init_images(device, kernel_dir, NULL, out); }
+
+/* images: names (without .cubin) separated by blanks; NULL = all of them.  Kernels of images left out stay unset: launching
+ * one is an error. */
+LB_API int lb_init_images(int device, const char* kernel_dir, const char* images, lb_ctx** out) {
     if (!out) return LB_ERR_INVALID;
     *out = NULL;
     lb_ctx* c = (lb_ctx*)calloc(1, sizeof *c);
@@ -163,11 +168,25 @@ LB_API int lb_init(int device, const char* kernel_dir, lb_ctx** out) {
         self_dir(sd, sizeof sd);
         snprintf(dir, sizeof dir, "%s/kernels", sd);
     }
-    for (size_t i = 0; i < sizeof k_cubins / sizeof k_cubins[0]; i++) LB_TRY(load_cubin(c, dir, k_cubins[i]));
+    if (!images) {
+        for (size_t i = 0; i < sizeof k_cubins / sizeof k_cubins[0]; i++) LB_TRY(load_cubin(c, dir, k_cubins[i]));
+    } else {
+        char name[64];
+        for (const char* q = images; *q;) {
+            const size_t n = strcspn(q, " ");
+            if (n && n < sizeof name - 8) {
+                snprintf(name, sizeof name, "%.*s.cubin", (int)n, q);
+                LB_TRY(load_cubin(c, dir, name));
+            }
+            q += n;
+            while (*q == ' ') q++;
+        }
+    }
     for (int k = 0; k < LBK_COUNT; k++) {
         CUresult r = CUDA_ERROR_NOT_FOUND;
         for (int m = 0; m < c->n_modules && r != CUDA_SUCCESS; m++)
             r = lb_drv.ModuleGetFunction(&c->fn[k], c->modules[m], k_kernel_names[k]);
+        if (r != CUDA_SUCCESS && images) { c->fn[k] = NULL; continue; }
         if (r != CUDA_SUCCESS)
             return lb_fail(c, LB_ERR_NO_KERNEL, "entry point %s not found in any kernel image under %s",
                            k_kernel_names[k], dir);

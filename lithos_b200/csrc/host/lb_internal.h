@@ -119,6 +119,35 @@ int lb_driver_load(char* err, size_t errlen); /* LB_OK or LB_ERR_NO_DRIVER */
     X(pf_add)                         \
     X(pf_attn_prepare)                \
     X(pf_attn_chunk)                  \
+    X(rows_gemv)                      \
+    X(gemm_bf16_tc)                   \
+    X(gemm_f32_simt)                  \
+    X(norm_rows2)                     \
+    X(wattn_rows_b2n2)                \
+    X(wattn_rows_b4n2)                \
+    X(wattn_rows_b8n2)                \
+    X(wattn_rows_b2n4)                \
+    X(wattn_rows_b4n4)                \
+    X(wattn_rows_b8n4)                \
+    X(wattn_rows_f2n2)                \
+    X(wattn_rows_f4n2)                \
+    X(wattn_rows_f8n2)                \
+    X(wattn_rows_f2n4)                \
+    X(wattn_rows_f4n4)                \
+    X(wattn_rows_f8n4)                \
+    X(wattn_prepare_bf16)             \
+    X(wattn_prepare_f32)              \
+    X(wattn_chunk_64)                 \
+    X(wattn_chunk_128)                \
+    X(wattn_chunk_256)                \
+    X(da_step_64)                     \
+    X(da_step_128)                    \
+    X(da_step_256)                    \
+    X(da_inputs)                      \
+    X(da_scan_64)                     \
+    X(da_scan_128)                    \
+    X(da_scan_256)                    \
+    X(da_finish)                      \
     X(l2_flush)
 
 enum {
@@ -187,6 +216,8 @@ int lb_launch(lb_ctx* c, int kernel, unsigned gx, unsigned gy, unsigned gz, unsi
               int pdl);
 int lb_launch_cluster(lb_ctx* c, int kernel, unsigned gx, unsigned gy, unsigned gz, unsigned bx, unsigned smem,
                       void** params, int pdl, unsigned cluster_y);
+
+unsigned char* lb_map_file(const char* path, size_t* bytes); /* lb_safetensors.c: a whole file, read-only */
 
 /* rng helpers used by the synthetic model builder */
 uint64_t lb_rng_u64(uint64_t seed, uint64_t stream, uint64_t i);

@@ -1,4 +1,6 @@
-/* Private view of the decode-step model shared by lb_model.c (the step) and lb_prefill.c (the prompt pass). */
+/* Private view of a model: what the shared runtime (lb_model.c: decode step, graph, sampling, generation; lb_prefill.c: prompt
+ * pass) keeps for every architecture, and the table of calls an architecture fills in (lb_hybrid.c: the int4 DeltaNet /
+ * attention hybrid; lb_stack.c: bf16 models described by a list of layers). */
 #ifndef LB_MODEL_PRIV_H
 #define LB_MODEL_PRIV_H
 #include "lb_internal.h"
@@ -31,9 +33,37 @@ typedef struct {
     int loaded;
 } layer_t;
 
+/* the activations of one prompt chunk: an architecture names the buffers it uses; the residual stream comes first */
+#define LB_PF_MAX_BUFS 16
+typedef union {
+    CUdeviceptr b[LB_PF_MAX_BUFS];
+    struct { CUdeviceptr X, xn16, proj, q, k, v, g, beta, mix, mix16, y, gu, act16; } hy; /* lb_hybrid.c */
+    struct { CUdeviceptr X, h1, h2, proj, cat, q, k, a, o; } st;                            /* lb_stack.c */
+} pf_set;
+
+/* What an architecture supplies.  The runtime owns embedding, order of calls, positions, graph capture, chunking and
+ * streams of the prompt pass, sampling and the generation loop. */
+typedef struct lb_arch {
+    const char* name;
+    int pf_chunk, pf_streams;                          /* prompt pass: tokens per chunk, chunks in flight (<= LB_PF_MAX_STREAMS) */
+    int (*reset_state)(lb_model* m);                    /* caches and recurrent states of the sequence back to empty (stream-ordered) */
+    int (*snapshot)(lb_model* m, int restore);          /* checkpoint / rollback of the recurrent states */
+    int (*state_ptr)(lb_model* m, int layer, int which, uint64_t* dptr, size_t* bytes);
+    int (*step_layers)(lb_model* m);                    /* one token: m->X (its embedding) through every layer; position in m->d_pos */
+    int (*head)(lb_model* m, CUdeviceptr x_row);        /* final norm + LM head of one row -> m->logits, arg-max candidates */
+    int (*head_ctas)(lb_model* m);                      /* how many candidates head leaves */
+    int (*head_rows)(lb_model* m, CUdeviceptr rows, int n, CUdeviceptr logits); /* the same for n <= pf_chunk rows, no candidates */
+    void (*pf_sizes)(const lb_model* m, size_t bytes[LB_PF_MAX_BUFS]);          /* bytes of each buffer of a chunk (0 = unused) */
+    int (*pf_layer)(lb_model* m, pf_set* w, int l, int pos0, int T);           /* one layer over a chunk; on c->stream */
+    void (*destroy)(lb_model* m);
+} lb_arch;
+#define LB_PF_MAX_STREAMS 4
+
 struct lb_model {
     lb_ctx* c;
-    lb_model_cfg cfg;
+    const lb_arch* arch;
+    void* impl;       /* lb_stack.c: its own description and weights */
+    lb_model_cfg cfg; /* n_layers, hidden, vocab, max_ctx and eps hold for every architecture, the rest for the hybrid */
     int tp_rank, tp_size;
     /* per-shard sizes */
     int HV, HK, HQ, HKV, inter_s; /* heads / intermediate columns on this shard */
@@ -65,7 +95,7 @@ typedef struct lb_prefill_ws lb_prefill_ws;
 
 int lb_model_is_fa(const lb_model_cfg* c, int l);
 int lb_model_launch_sampler(lb_model* m);
-/* the decode-attention launch of one attention layer: inputs are the fused projection's fp32 row (per head 256 query then
- * 256 gate columns, then the key and value heads); pos_ptr != 0 reads the position from device memory (graph replay) */
-int lb_model_launch_attention(lb_model* m, const layer_t* L, CUdeviceptr proj_row, CUdeviceptr out, CUdeviceptr pos_ptr, int pos, int splits_for);
+int lb_model_alloc_common(lb_model* m); /* the buffers every architecture uses; cfg and vocab_s must be set */
+int lb_dalloc(lb_model* m, CUdeviceptr* p, size_t bytes);
+int lb_upload(lb_model* m, CUdeviceptr* p, const void* src, size_t bytes);
 #endif

@@ -17,12 +17,10 @@
  */
 #define _GNU_SOURCE
 #include "lb_internal.h"
+#include "lb_safetensors.h"
 #include <errno.h>
-#include <fcntl.h>
 #include <stdarg.h>
 #include <sys/mman.h>
-#include <sys/stat.h>
-#include <unistd.h>
 
 #define WIDX_MAGIC 0x4C575449u
 #define WIDX_VERSION 1u
@@ -51,19 +49,6 @@ static int wfail(char* err, size_t errlen, int status, const char* fmt, ...) {
 static uint32_t rd32(const unsigned char* p) { uint32_t v; memcpy(&v, p, 4); return v; }
 static uint64_t rd64(const unsigned char* p) { uint64_t v; memcpy(&v, p, 8); return v; }
 
-/* map a whole file read-only (private); *bytes receives its size */
-static unsigned char* map_file(const char* path, size_t* bytes) {
-    int fd = open(path, O_RDONLY);
-    if (fd < 0) return NULL;
-    struct stat st;
-    if (fstat(fd, &st) != 0 || st.st_size <= 0) { close(fd); return NULL; }
-    void* p = mmap(NULL, (size_t)st.st_size, PROT_READ, MAP_PRIVATE, fd, 0);
-    close(fd);
-    if (p == MAP_FAILED) return NULL;
-    *bytes = (size_t)st.st_size;
-    return (unsigned char*)p;
-}
-
 LB_API void lb_weight_index_close(lb_weight_index* w) {
     if (!w) return;
     for (uint32_t s = 0; s < w->n_shards && s < WIDX_MAX_SHARDS; s++)
@@ -79,7 +64,7 @@ LB_API int lb_weight_index_open(const char* model_dir, lb_weight_index** out, ch
     snprintf(path, sizeof path, "%s/weight_index.bin", model_dir);
     lb_weight_index* w = (lb_weight_index*)calloc(1, sizeof *w);
     if (!w) return wfail(err, errlen, LB_ERR_NOMEM, "weight index: out of memory");
-    w->idx = map_file(path, &w->idx_bytes);
+    w->idx = lb_map_file(path, &w->idx_bytes);
     if (!w->idx) { free(w); return wfail(err, errlen, LB_ERR_IO, "weight index: cannot open %s (%s)", path, strerror(errno)); }
     int st = LB_OK;
     if (w->idx_bytes < 32) st = wfail(err, errlen, LB_ERR_IO, "weight index: %s is %zu bytes, shorter than its header", path, w->idx_bytes);
@@ -100,7 +85,7 @@ LB_API int lb_weight_index_open(const char* model_dir, lb_weight_index** out, ch
         const unsigned char* e = w->idx + 32 + (size_t)s * WIDX_SHARD_ENTRY;
         if (!memchr(e, 0, 256)) { st = wfail(err, errlen, LB_ERR_IO, "weight index: shard %u file name is not terminated", s); break; }
         snprintf(path, sizeof path, "%s/%s", model_dir, (const char*)e);
-        w->shard[s] = map_file(path, &w->shard_bytes[s]);
+        w->shard[s] = lb_map_file(path, &w->shard_bytes[s]);
         if (!w->shard[s]) { st = wfail(err, errlen, LB_ERR_IO, "weight index: cannot map shard %u '%s' (%s)", s, path, strerror(errno)); break; }
         const uint64_t want = rd64(e + 256);
         if (want != w->shard_bytes[s]) {
@@ -299,9 +284,7 @@ LB_API int lb_load_weights(lb_ctx* c, const char* model_dir, lb_model* m) {
  * The reference resolves its slots from a safetensors checkpoint by tensor name (compiler/megakernel-link.ls:220-269 for the
  * layers, :825-827 for the globals; slot names in src/launcher.s:92-141) and its launcher then reads weight_index.bin, whose
  * generator is not in the tree.  This is that generator: every *.safetensors file of the directory becomes a shard, every slot
- * the (shard, file offset, size) of the tensor `model.layers.<n>.<suffix>`.
- * A safetensors file is: u64 LE header length, a JSON object {"<name>": {"dtype": .., "shape": [..], "data_offsets": [b, e]},
- * ..., "__metadata__": {..}}, then the data; offsets are relative to the end of the header. */
+ * the (shard, file offset, size) of the tensor `model.layers.<n>.<suffix>`. */
 static const char* const k_dn_suffix[LB_WS_SLOTS] = {
     "linear_attn.in_proj_qkv.qweight", "linear_attn.in_proj_qkv.scales", "linear_attn.in_proj_qkv.qzeros",
     "linear_attn.in_proj_z.qweight", "linear_attn.in_proj_z.scales", "linear_attn.in_proj_z.qzeros",
@@ -316,119 +299,15 @@ static const char* const k_fa_suffix[15] = {
     "self_attn.o_proj.scales", "self_attn.o_proj.qzeros", "self_attn.q_norm.weight", "self_attn.k_norm.weight", NULL};
 static const char* const k_global_name[LB_WG_SLOTS] = {"model.embed_tokens.weight", "lm_head.weight", "model.norm.weight"};
 
-typedef struct { char* name; uint32_t shard; uint64_t off, size; } st_tensor;
-
-/* p at an opening quote: returns the position after the closing quote, *s / *n the text between (escapes are skipped, not decoded) */
-static const char* st_string(const char* p, const char* end, const char** s, size_t* n) {
-    if (p >= end || *p != '"') return NULL;
-    const char* q = ++p;
-    while (q < end && *q != '"') q += (*q == '\\' && q + 1 < end) ? 2 : 1;
-    if (q >= end) return NULL;
-    *s = p; *n = (size_t)(q - p);
-    return q + 1;
-}
-static const char* st_ws(const char* p, const char* end) { while (p < end && (*p == ' ' || *p == '\n' || *p == '\t' || *p == '\r')) p++; return p; }
-/* p at the first character of a JSON value: returns the position after it (strings, nesting and escapes respected) */
-static const char* st_skip_value(const char* p, const char* end) {
-    int depth = 0;
-    while (p < end) {
-        if (*p == '"') { const char* s; size_t n; p = st_string(p, end, &s, &n); if (!p) return NULL; if (!depth) return p; continue; }
-        if (*p == '{' || *p == '[') depth++;
-        else if (*p == '}' || *p == ']') { if (--depth == 0) return p + 1; if (depth < 0) return NULL; }
-        else if (!depth && (*p == ',')) return p;
-        p++;
-    }
-    return depth ? NULL : p;
-}
-
-/* the tensors of one header; data_base = file offset of the data section */
-static int st_parse_header(const char* js, size_t len, uint32_t shard, uint64_t data_base, uint64_t file_bytes, st_tensor** tab, size_t* n_tab,
-                           size_t* cap, char* err, size_t errlen, const char* file) {
-    const char *p = st_ws(js, js + len), *end = js + len;
-    if (p >= end || *p != '{') return wfail(err, errlen, LB_ERR_IO, "%s: the header is not a JSON object", file);
-    p = st_ws(p + 1, end);
-    while (p < end && *p != '}') {
-        const char* key; size_t klen;
-        p = st_string(p, end, &key, &klen);
-        if (!p) return wfail(err, errlen, LB_ERR_IO, "%s: malformed header (tensor name)", file);
-        p = st_ws(p, end);
-        if (p >= end || *p != ':') return wfail(err, errlen, LB_ERR_IO, "%s: malformed header (':' after a name)", file);
-        p = st_ws(p + 1, end);
-        const char* v0 = p;
-        const char* v1 = st_skip_value(p, end);
-        if (!v1) return wfail(err, errlen, LB_ERR_IO, "%s: malformed header (value of %.*s)", file, (int)klen, key);
-        if (!(klen == 12 && !memcmp(key, "__metadata__", 12))) {
-            /* "data_offsets": [begin, end] inside the value */
-            const char* d = NULL;
-            for (const char* q = v0; q + 14 <= v1; q++)
-                if (!memcmp(q, "\"data_offsets\"", 14)) { d = q + 14; break; }
-            unsigned long long b = 0, e = 0;
-            char num[96]; /* a bounded, terminated copy: the header is a slice of a mapped file */
-            size_t nn = d ? (size_t)(v1 - d) : 0;
-            if (nn > sizeof num - 1) nn = sizeof num - 1;
-            if (d) memcpy(num, d, nn);
-            num[nn] = 0;
-            if (!d || sscanf(num, " : [ %llu , %llu ]", &b, &e) != 2 || e < b || data_base + e > file_bytes)
-                return wfail(err, errlen, LB_ERR_IO, "%s: tensor %.*s has no valid data_offsets", file, (int)klen, key);
-            if (*n_tab == *cap) {
-                *cap = *cap ? *cap * 2 : 1024;
-                st_tensor* t = (st_tensor*)realloc(*tab, *cap * sizeof **tab);
-                if (!t) return wfail(err, errlen, LB_ERR_NOMEM, "weight index: out of memory");
-                *tab = t;
-            }
-            st_tensor* t = &(*tab)[(*n_tab)++];
-            t->name = (char*)malloc(klen + 1);
-            if (!t->name) return wfail(err, errlen, LB_ERR_NOMEM, "weight index: out of memory");
-            memcpy(t->name, key, klen); t->name[klen] = 0;
-            t->shard = shard; t->off = data_base + b; t->size = e - b;
-        }
-        p = st_ws(v1, end);
-        if (p < end && *p == ',') p = st_ws(p + 1, end);
-    }
-    return LB_OK;
-}
-
-static int st_cmp_name(const void* a, const void* b) { return strcmp(((const st_tensor*)a)->name, ((const st_tensor*)b)->name); }
-static int st_cmp_str(const void* a, const void* b) { return strcmp(*(const char* const*)a, *(const char* const*)b); }
-
-#include <dirent.h>
-
 LB_API int lb_weight_index_from_safetensors(const char* model_dir, const lb_model_cfg* c, char* err, size_t errlen) {
     if (!model_dir || !c) return wfail(err, errlen, LB_ERR_INVALID, "lb_weight_index_from_safetensors: NULL argument");
-    /* the shard files, in name order */
-    char* files[WIDX_MAX_SHARDS];
-    int n_files = 0, st = LB_OK;
-    DIR* d = opendir(model_dir);
-    if (!d) return wfail(err, errlen, LB_ERR_IO, "cannot open %s (%s)", model_dir, strerror(errno));
-    for (struct dirent* e; (e = readdir(d)) != NULL;) {
-        const size_t n = strlen(e->d_name);
-        if (n < 13 || n > 255 || strcmp(e->d_name + n - 12, ".safetensors")) continue;
-        if (n_files == WIDX_MAX_SHARDS) { st = wfail(err, errlen, LB_ERR_IO, "%s holds more than %d safetensors files", model_dir, WIDX_MAX_SHARDS); break; }
-        files[n_files++] = strdup(e->d_name);
-    }
-    closedir(d);
-    if (st == LB_OK && !n_files) st = wfail(err, errlen, LB_ERR_IO, "%s holds no *.safetensors file", model_dir);
-    qsort(files, (size_t)n_files, sizeof files[0], st_cmp_str);
-    st_tensor* tab = NULL;
-    size_t n_tab = 0, cap = 0;
-    uint64_t shard_bytes[WIDX_MAX_SHARDS] = {0};
-    for (int i = 0; i < n_files && st == LB_OK; i++) {
-        char path[1536];
-        snprintf(path, sizeof path, "%s/%s", model_dir, files[i]);
-        size_t bytes = 0;
-        unsigned char* m = map_file(path, &bytes);
-        if (!m) { st = wfail(err, errlen, LB_ERR_IO, "cannot map %s (%s)", path, strerror(errno)); break; }
-        shard_bytes[i] = bytes;
-        uint64_t hlen = bytes >= 8 ? rd64(m) : 0;
-        if (bytes < 8 || hlen > bytes - 8) st = wfail(err, errlen, LB_ERR_IO, "%s: header length %llu does not fit the file", path, (unsigned long long)hlen);
-        else st = st_parse_header((const char*)m + 8, (size_t)hlen, (uint32_t)i, 8 + hlen, bytes, &tab, &n_tab, &cap, err, errlen, files[i]);
-        munmap(m, bytes);
-    }
+    lb_st_set set; /* the shard files, in name order, and their tensors */
+    int st = lb_st_open(model_dir, &set, err, errlen);
+    if (st != LB_OK) return st;
     const size_t n_entries = (size_t)LB_WG_SLOTS + (size_t)c->n_layers * LB_WS_SLOTS;
     unsigned char* out = st == LB_OK ? (unsigned char*)calloc(n_entries, WIDX_ENTRY) : NULL;
     if (st == LB_OK && !out) st = wfail(err, errlen, LB_ERR_NOMEM, "weight index: out of memory");
     if (st == LB_OK) {
-        qsort(tab, n_tab, sizeof *tab, st_cmp_name);
         for (size_t i = 0; i < n_entries && st == LB_OK; i++) {
             char name[320];
             size_t want;
@@ -442,13 +321,11 @@ LB_API int lb_weight_index_from_safetensors(const char* model_dir, const lb_mode
                 if (!suffix || !want) continue; /* slot unused in this kind of layer */
                 snprintf(name, sizeof name, "model.layers.%d.%s", l, suffix);
             }
-            st_tensor key;
-            key.name = name;
-            const st_tensor* t = (const st_tensor*)bsearch(&key, tab, n_tab, sizeof *tab, st_cmp_name);
+            const lb_st_tensor* t = lb_st_find(&set, name);
             if (!t) { st = wfail(err, errlen, LB_ERR_INVALID, "tensor %s is not in the checkpoint", name); break; }
             if (t->size != want) { st = wfail(err, errlen, LB_ERR_IO, "tensor %s holds %llu bytes, the model shape needs %zu", name, (unsigned long long)t->size, want); break; }
             unsigned char* e = out + i * WIDX_ENTRY;
-            memcpy(e, &t->shard, 4); memcpy(e + 8, &t->off, 8); memcpy(e + 16, &t->size, 8);
+            memcpy(e, &t->file, 4); memcpy(e + 8, &t->off, 8); memcpy(e + 16, &t->size, 8);
         }
     }
     if (st == LB_OK) {
@@ -457,13 +334,14 @@ LB_API int lb_weight_index_from_safetensors(const char* model_dir, const lb_mode
         FILE* f = fopen(path, "wb");
         if (!f) st = wfail(err, errlen, LB_ERR_IO, "cannot create %s (%s)", path, strerror(errno));
         else {
-            uint32_t hdr[8] = {WIDX_MAGIC, WIDX_VERSION, (uint32_t)n_files, (uint32_t)c->n_layers, LB_WS_SLOTS, LB_WG_SLOTS, 0, 0};
+            uint32_t hdr[8] = {WIDX_MAGIC, WIDX_VERSION, (uint32_t)set.n_files, (uint32_t)c->n_layers, LB_WS_SLOTS, LB_WG_SLOTS, 0, 0};
             int bad = put(f, hdr, 32);
-            for (int i = 0; i < n_files; i++) {
+            for (int i = 0; i < set.n_files; i++) {
                 unsigned char se[WIDX_SHARD_ENTRY];
                 memset(se, 0, sizeof se);
-                memcpy(se, files[i], strlen(files[i]));
-                memcpy(se + 256, &shard_bytes[i], 8);
+                memcpy(se, set.file[i], strlen(set.file[i]));
+                const uint64_t fb = set.bytes[i];
+                memcpy(se + 256, &fb, 8);
                 bad |= put(f, se, sizeof se);
             }
             bad |= put(f, out, n_entries * WIDX_ENTRY);
@@ -471,9 +349,7 @@ LB_API int lb_weight_index_from_safetensors(const char* model_dir, const lb_mode
             if (bad) st = wfail(err, errlen, LB_ERR_IO, "writing %s failed", path);
         }
     }
-    for (size_t i = 0; i < n_tab; i++) free(tab[i].name);
-    free(tab);
     free(out);
-    for (int i = 0; i < n_files; i++) free(files[i]);
+    lb_st_close(&set);
     return st;
 }

@@ -1,0 +1,253 @@
+// Dense products of a prompt chunk for bf16 models: Y[T, N] = X[T, K] W[N, K]^T with fused epilogues, one or two of them (the mixer's
+// and the feed-forward's input projections read differently normed copies of the same rows) in one launch; and the chunk's RMS norm.
+//
+// gemm_bf16_tc: 5th-generation tensor cores.  A tile is 128 weight rows x NT (16..256) tokens: tcgen05.mma 128 x NT x 16, both operands by
+// tiled TMA (64 k x rows, 128-byte swizzle), accumulators in tensor memory.  Persistent CTAs of six warps: one lane brings operands, one
+// lane issues products, four warps read accumulators (lane = weight row, column = token) and finish them.  Two accumulators, so the
+// epilogue of a tile runs beside the products of the next.  Weight rows are the lanes, so 32 neighbouring outputs of a token are one
+// coalesced store and a (gate, up) pair sits in neighbouring lanes.  Every wait is bounded and reports through the status word.
+// gemm_f32_simt: the same products in fp32 throughout (fp32 activations, weights exact in fp32, fp32 fused multiply-adds).
+#include "tcgen05.cuh"
+#include "params.h"
+
+#define DG_FAIL_EMPTY 0x1201u // status: a stage's products never completed
+#define DG_FAIL_FULL 0x1202u  // status: a stage's operands never landed
+#define DG_FAIL_ACC 0x1203u   // status: an accumulator was never completed / never freed
+
+__device__ __forceinline__ void dg_tma(uint32_t dst_smem, const void* tmap, int k, int row, uint64_t* bar) {
+    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst_smem),
+                 "l"(tmap), "r"(k), "r"(row), "r"(smem_u32(bar))
+                 : "memory");
+}
+
+extern "C" __global__ void __launch_bounds__(LB_DG_THREADS, 1) gemm_bf16_tc(const __grid_constant__ lb_dgemm_params p) {
+    extern __shared__ __align__(1024) unsigned char dg_sm[];
+    __shared__ __align__(8) uint64_t bar_full[LB_DG_MAX_STAGES], bar_empty[LB_DG_MAX_STAGES], bar_acc[2], bar_free[2];
+    __shared__ uint32_t tmem_slot;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int S = p.stages, NT = p.NT;
+    const uint32_t a_bytes = LB_DG_ROWS * LB_DG_KB * 2, b_bytes = (uint32_t)NT * LB_DG_KB * 2, stage_bytes = a_bytes + b_bytes;
+    const int ksteps = p.K / LB_DG_KB, n_tiles = (p.tiles[0] + p.tiles[1]) * p.t_tiles;
+    if (tid == 0) {
+        for (int s = 0; s < S; ++s) {
+            mbar_init(&bar_full[s], 1);
+            mbar_init(&bar_empty[s], 1);
+        }
+        for (int s = 0; s < 2; ++s) {
+            mbar_init(&bar_acc[s], 1);
+            mbar_init(&bar_free[s], 4);
+        }
+        mbar_fence_init();
+    }
+    if (warp == 1) tmem_alloc(&tmem_slot, (uint32_t)p.tmem_cols);
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = tmem_slot;
+    pdl_wait();
+
+    if (warp == 0 && lane == 0) {
+        // ---------------- operands ----------------
+        int s = 0, issued = 0;
+        uint32_t ph = 0;
+        bool ok = true;
+        for (int tile = blockIdx.x; tile < n_tiles && ok; tile += gridDim.x) {
+            const int rt = tile / p.t_tiles, tt = tile - rt * p.t_tiles, m = rt >= p.tiles[0];
+            const int row = (m ? rt - p.tiles[0] : rt) * LB_DG_ROWS, tok = tt * NT;
+            for (int k = 0; k < ksteps; ++k) {
+                if (issued >= S && !tc_wait(&bar_empty[s], ph ^ 1u)) {
+                    ok = false;
+                    if (p.status) atomicExch(p.status, DG_FAIL_EMPTY);
+                    break;
+                }
+                mbar_arrive_expect_tx(&bar_full[s], stage_bytes);
+                const uint32_t dst = smem_u32(dg_sm) + (uint32_t)s * stage_bytes;
+                dg_tma(dst, p.tmap_w[m], k * LB_DG_KB, row, &bar_full[s]);
+                dg_tma(dst + a_bytes, p.tmap_x[m], k * LB_DG_KB, tok, &bar_full[s]);
+                ++issued;
+                if (++s == S) { s = 0; ph ^= 1u; }
+            }
+        }
+        if (!ok) // nothing may still be on its way into this CTA's shared memory when it ends
+            for (int d = 0; d < S && d < issued; ++d) {
+                if (--s < 0) { s = S - 1; ph ^= 1u; }
+                tc_wait(&bar_full[s], ph);
+            }
+    } else if (warp == 1 && lane == 0) {
+        // ---------------- products ----------------
+        const uint32_t idesc = tc_idesc_bf16(LB_DG_ROWS, (uint32_t)NT);
+        int s = 0, it = 0;
+        uint32_t ph = 0;
+        bool ok = true;
+        for (int tile = blockIdx.x; tile < n_tiles && ok; tile += gridDim.x, ++it) {
+            const int b = it & 1;
+            if (it >= 2 && !tc_wait(&bar_free[b], (uint32_t)((it >> 1) - 1) & 1u)) { // the epilogue has read this accumulator
+                ok = false;
+                if (p.status) atomicExch(p.status, DG_FAIL_ACC);
+                break;
+            }
+            tc_fence_after();
+            const uint32_t d = tmem + (uint32_t)(b * NT);
+            for (int k = 0; k < ksteps; ++k) {
+                if (!tc_wait(&bar_full[s], ph)) {
+                    ok = false;
+                    if (p.status) atomicExch(p.status, DG_FAIL_FULL);
+                    break;
+                }
+                tc_fence_after();
+                const uint32_t base = smem_u32(dg_sm) + (uint32_t)s * stage_bytes;
+                const uint64_t ad = tc_smem_desc(base, 16, 1024), bd = tc_smem_desc(base + a_bytes, 16, 1024);
+#pragma unroll
+                for (int kk = 0; kk < LB_DG_KB / 16; ++kk)
+                    tc_mma(d, ad + (uint64_t)(kk * 2), bd + (uint64_t)(kk * 2), idesc, (k > 0 || kk > 0) ? 1u : 0u);
+                tc_commit(&bar_empty[s]);
+                if (++s == S) { s = 0; ph ^= 1u; }
+            }
+            if (ok) tc_commit(&bar_acc[b]);
+        }
+    } else if (warp >= 2) {
+        // ---------------- epilogue: warp w reads the tensor-memory lanes 32 (w % 4) .. + 31 ----------------
+        const int quad = warp & 3;
+        int it = 0;
+        for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x, ++it) {
+            const int b = it & 1;
+            const int rt = tile / p.t_tiles, tt = tile - rt * p.t_tiles, m = rt >= p.tiles[0];
+            const int n = (m ? rt - p.tiles[0] : rt) * LB_DG_ROWS + quad * 32 + lane, t0 = tt * NT;
+            const bool got = tc_wait(&bar_acc[b], (uint32_t)(it >> 1) & 1u);
+            if (!__all_sync(0xffffffffu, got)) {
+                if (lane == 0 && p.status) atomicExch(p.status, DG_FAIL_ACC);
+                break;
+            }
+            tc_fence_after();
+            const int mode = p.y_mode[m], ld = p.ld_y[m], n_t = min(NT, p.T - t0);
+            const bool live = n < p.rows[m];
+            for (int c = 0; c < n_t; c += 16) {
+                uint32_t r[16];
+                tmem_ld16(tmem + ((uint32_t)(32 * quad) << 16) + (uint32_t)(b * NT + c), r);
+                tmem_ld_wait();
+                if (mode == LB_DY_RELU_GLU) {
+                    const bool st = live && !(lane & 1);
+#pragma unroll
+                    for (int j = 0; j < 16; ++j) {
+                        const float up = __uint_as_float(__shfl_xor_sync(0xffffffffu, r[j], 1)), v = fmaxf(__uint_as_float(r[j]), 0.f) * up;
+                        if (st && c + j < n_t) {
+                            const size_t o = (size_t)(t0 + c + j) * ld + (n >> 1);
+                            if (p.y_f32[m]) reinterpret_cast<float*>(p.y[m])[o] = v;
+                            else reinterpret_cast<__nv_bfloat16*>(p.y[m])[o] = __float2bfloat16_rn(v);
+                        }
+                    }
+                } else {
+                    float* y = reinterpret_cast<float*>(p.y[m]) + (size_t)(t0 + c) * ld + n;
+                    float old[16];
+                    if (mode == LB_DY_RESIDUAL) {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) old[j] = live && c + j < n_t ? y[(size_t)j * ld] : 0.f;
+                    }
+#pragma unroll
+                    for (int j = 0; j < 16; ++j) {
+                        float v = __uint_as_float(r[j]);
+                        if (mode == LB_DY_RESIDUAL) v = fmaf(p.mult, v, old[j]);
+                        else if (mode == LB_DY_SOFTCAP && p.cap > 0.f) v = p.cap * tanhf(v / p.cap);
+                        if (live && c + j < n_t) y[(size_t)j * ld] = v;
+                    }
+                }
+            }
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&bar_free[b]);
+        }
+    }
+    pdl_launch_dependents();
+    __syncthreads();
+    if (warp == 1) {
+        tc_fence_after();
+        tmem_dealloc(tmem, (uint32_t)p.tmem_cols);
+    }
+}
+
+// ---- fp32 ----------------------------------------------------------------------------------------------------------
+#define SG_TN 64 // weight rows per tile
+#define SG_TT 64 // tokens per tile
+#define SG_KB 16
+// grid (row tiles of both products, token tiles), block 256: a thread owns 4 rows x 4 tokens.  K is a multiple of 64.
+extern "C" __global__ void __launch_bounds__(256) gemm_f32_simt(const __grid_constant__ lb_dgemm_params p) {
+    __shared__ __align__(16) float ws[SG_KB][SG_TN + 4], xs[SG_KB][SG_TT + 4];
+    pdl_wait();
+    const int tid = threadIdx.x, tn = tid & 15, tt = tid >> 4;
+    const int nt0 = (p.rows[0] + SG_TN - 1) / SG_TN, m = (int)blockIdx.x >= nt0;
+    const int row0 = ((int)blockIdx.x - (m ? nt0 : 0)) * SG_TN, t0 = blockIdx.y * SG_TT;
+    const uint16_t* W = p.w[m];
+    const float* X = reinterpret_cast<const float*>(p.x[m]);
+    float acc[4][4] = {};
+    const int lr = tid >> 2, lk = (tid & 3) * 4; // load: row / token of the tile, 4 k
+    for (int k0 = 0; k0 < p.K; k0 += SG_KB) {
+        uint2 w = make_uint2(0u, 0u);
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (row0 + lr < p.rows[m]) w = *reinterpret_cast<const uint2*>(W + (size_t)(row0 + lr) * p.K + k0 + lk);
+        if (t0 + lr < p.T) x = *reinterpret_cast<const float4*>(X + (size_t)(t0 + lr) * p.ld_x + k0 + lk);
+        __syncthreads();
+        ws[lk][lr] = __uint_as_float(w.x << 16);
+        ws[lk + 1][lr] = __uint_as_float(w.x & 0xffff0000u);
+        ws[lk + 2][lr] = __uint_as_float(w.y << 16);
+        ws[lk + 3][lr] = __uint_as_float(w.y & 0xffff0000u);
+        xs[lk][lr] = x.x;
+        xs[lk + 1][lr] = x.y;
+        xs[lk + 2][lr] = x.z;
+        xs[lk + 3][lr] = x.w;
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < SG_KB; ++k) {
+            const float4 a = *reinterpret_cast<const float4*>(&ws[k][tn * 4]), b = *reinterpret_cast<const float4*>(&xs[k][tt * 4]);
+            const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+        }
+    }
+    pdl_launch_dependents();
+    const int mode = p.y_mode[m], ld = p.ld_y[m];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const int t = t0 + tt * 4 + j;
+        if (t >= p.T) continue;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int n = row0 + tn * 4 + i;
+            if (n >= p.rows[m]) continue;
+            float v = acc[i][j];
+            float* y = reinterpret_cast<float*>(p.y[m]) + (size_t)t * ld;
+            if (mode == LB_DY_RELU_GLU) {
+                if (i & 1) continue;
+                v = fmaxf(v, 0.f) * acc[i | 1][j];
+                if (p.y_f32[m]) y[n >> 1] = v;
+                else reinterpret_cast<__nv_bfloat16*>(p.y[m])[(size_t)t * ld + (n >> 1)] = __float2bfloat16_rn(v);
+            } else if (mode == LB_DY_RESIDUAL) y[n] = fmaf(p.mult, v, y[n]);
+            else y[n] = mode == LB_DY_SOFTCAP && p.cap > 0.f ? p.cap * tanhf(v / p.cap) : v;
+        }
+    }
+}
+
+// h_i[t] = x[t] / sqrt(mean x^2 + eps) * (1 + w_i), columns width..ld are zero.  grid T, block 256
+extern "C" __global__ void __launch_bounds__(256) norm_rows2(const __grid_constant__ lb_norm2_params p) {
+    __shared__ float red[40];
+    pdl_wait();
+    const float* x = p.x + (size_t)blockIdx.x * p.width;
+    float ss = 0.f;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < p.width; i += 256) ss += x[i] * x[i];
+    ss = block_sum(ss, red);
+    const float rinv = 1.0f / sqrtf(ss / (float)p.width + p.eps);
+    pdl_launch_dependents();
+    const size_t o = (size_t)blockIdx.x * p.ld;
+    for (int i = threadIdx.x; i < p.ld; i += 256) {
+        const float v = i < p.width ? x[i] * rinv : 0.f;
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            if (!p.h[e]) continue;
+            const float r = i < p.width ? v * (1.0f + bf16_bits_to_f32(p.w[e][i])) : 0.f;
+            if (p.f32) reinterpret_cast<float*>(p.h[e])[o + i] = r;
+            else reinterpret_cast<__nv_bfloat16*>(p.h[e])[o + i] = __float2bfloat16_rn(r);
+        }
+    }
+}

@@ -258,6 +258,122 @@ typedef struct {
                              LB_DEV_POS_RANGE and the kernel returns without reading or writing a cache row */
 } lb_attn_params;
 
+/* ---- dense bf16 rows x one fp32 vector with fused prologue and epilogue (rows_gemv) ------------------------
+ * One or two row-major bf16 matrices [rows, K] against vectors built in shared memory.  Rows are taken two at a time (a
+ * pair), pair p of the launch (matrix 0 first) by CTA p % gridDim.x; the number of rows is even (a zero row pads an odd
+ * matrix) and K is a multiple of 64. */
+#define LB_RG_THREADS 256
+#define LB_RG_WARPS 8
+#define LB_RG_SEG 1024 /* elements of one row in a pipeline stage */
+enum { LB_RG_X_NORM = 0, /* vector of matrix i = rmsnorm(x) * (1 + norm_w[i]) */
+       LB_RG_X_CAT = 1   /* one vector: the mixer's output (per-head norm and gate applied here), then the feed-forward's activations */ };
+/* epilogues, shared with the matrix products of a prompt chunk (lb_dgemm_params) */
+enum { LB_DY_STORE = 0,    /* y[n] = r */
+       LB_DY_RELU_GLU = 1, /* rows come as (gate, up) pairs: y[pair] = relu(gate) * up */
+       LB_DY_RESIDUAL = 2, /* y[n] += mult * r */
+       LB_DY_SOFTCAP = 3   /* y[n] = cap * tanh(r / cap), cap 0: y[n] = r; with part_val: arg-max candidates */ };
+typedef struct {
+    const uint16_t* w;      /* bf16 [rows, K] */
+    const uint16_t* norm_w; /* bf16 [width] (LB_RG_X_NORM) */
+    float* y;
+    int32_t rows;           /* rows with a result (the allocation holds an even number) */
+    int32_t y_mode;
+} lb_rg_mat;
+typedef struct {
+    lb_rg_mat mat[2];
+    const float* x;         /* LB_RG_X_NORM: fp32 [width] */
+    const float* mix;       /* LB_RG_X_CAT: fp32 [n_mix] */
+    const float* gate;      /* fp32 [n_mix]: mix *= silu(gate); NULL = no gate */
+    const uint16_t* head_w; /* bf16 [vdim]: mix = per-head rmsnorm * head_w first; NULL = none */
+    const float* act;       /* fp32 [n_act] */
+    float* part_val;        /* [gridDim.x] arg-max candidates (LB_DY_SOFTCAP), or NULL */
+    int32_t* part_idx;
+    uint32_t* status;
+    int32_t n_mat, K, width, x_mode;
+    int32_t n_mix, n_mix_pad, vdim, n_act; /* the feed-forward part starts at n_mix_pad */
+    int32_t stages;         /* ring stages per warp */
+    int32_t split;          /* pieces a row pair is cut into along K: 1, or one per stage segment */
+    int32_t segs;           /* ceil(K / LB_RG_SEG) */
+    float eps, mult, cap;
+} lb_rows_gemv_params;
+
+/* ---- dense products of a prompt chunk: Y[T, N] = X[T, K] W[N, K]^T, one or two of them in one launch --------- */
+#define LB_DG_ROWS 128  /* weight rows per tile = M of the product */
+#define LB_DG_KB 64     /* k per pipeline stage: one 128-byte swizzled row */
+#define LB_DG_THREADS 192
+#define LB_DG_MAX_STAGES 8
+typedef struct {
+    unsigned char tmap_w[2][128] __attribute__((aligned(64))); /* bf16 [rows, K], box 64 x 128, 128-byte swizzle */
+    unsigned char tmap_x[2][128] __attribute__((aligned(64))); /* bf16 [T, K], box 64 x NT, 128-byte swizzle */
+    const uint16_t* w[2]; /* the same operands as pointers (gemm_f32_simt) */
+    const void* x[2];
+    void* y[2];
+    int32_t rows[2], y_mode[2], ld_y[2];
+    int32_t tiles[2];     /* row tiles of each product (tiles[1] = 0: one product) */
+    int32_t y_f32[2];     /* LB_DY_RELU_GLU: y is fp32 (else bf16) */
+    int32_t T, NT, t_tiles, K, ld_x, stages, tmem_cols;
+    float mult, cap;
+    uint32_t* status;
+} lb_dgemm_params;
+
+/* rmsnorm of a chunk with up to two weights: h_i[t] = rmsnorm(x[t]) * (1 + w_i) */
+typedef struct {
+    const float* x;      /* fp32 [T, width] */
+    const uint16_t* w[2];
+    void* h[2];          /* bf16 (or fp32) [T, ld]; h[1] may be NULL */
+    int32_t width, ld, f32;
+    float eps;
+} lb_norm2_params;
+
+/* ---- attention over the current block of positions, general head sizes (window_attention.cu) ---------------- */
+#define LB_WA_MAX_DIM 256
+typedef struct {
+    const float* proj;   /* fp32 [T, ld]: q | k | v sections at the given offsets */
+    void* k_cache;       /* bf16 (or fp32) [max_ctx, KV, dim_p]: rotated keys; padding columns are zero */
+    void* v_cache;       /* [max_ctx, KV, vdim_p]: normed, rotated values */
+    const double* freq_k; /* [rot_dims / 2] radians per position */
+    const double* freq_v; /* [vdim / 2]; NULL: values are not rotated */
+    float* out;          /* fp32 [H * vdim] of one token (decode) ... */
+    void* cat;           /* ... or, when not NULL, rows [T, cat_ld] of bf16 / fp32 (prompt) */
+    uint16_t* qh;        /* prompt, bf16: rotated queries x scale x log2(e) as two bf16 terms [T, H, dim_p] */
+    uint16_t* ql;
+    float* scratch;      /* partials of the position slices: [groups][splits][heads per CTA][vdim_p + 2] */
+    uint32_t* counters;  /* one per (KV head, head group), zero between launches */
+    const int32_t* pos_ptr; /* position of token 0 in device memory, or NULL: pos0 */
+    uint32_t* status;
+    int32_t ld, q_off, k_off, v_off; /* k_off < 0: the cache belongs to another layer, which has filled it */
+    int32_t H, KV, dim, vdim, dim_p, vdim_p, rot_dims;
+    int32_t block;       /* position i sees j <= i with the same floor(j / block); 0: every j <= i */
+    int32_t v_norm;      /* values are divided by their root mean square */
+    int32_t sink;        /* 1 is added to the soft-max denominator */
+    int32_t pos0, T, max_ctx, splits, cat_ld;
+    float scale, eps;
+} lb_wattn_params;
+/* wattn_chunk_*: query rows per CTA (16 per warp), keys per staged block */
+#define LB_WA_ROWS 64
+#define LB_WA_THREADS 128
+#define LB_WA_KV 32
+
+/* ---- linear attention with one decay per key channel (decay_attention.cu) ----------------------------------- */
+enum { LB_DA_HGRN2 = 0, LB_DA_GLA = 1 };
+typedef struct {
+    const float* proj;    /* fp32 [T, ld]: sections at the offsets below */
+    const uint16_t* a2;   /* GLA: bf16 [H * dk, rank] */
+    const uint16_t* bias; /* bf16 [H * dk]: added to the gate's pre-activation */
+    const uint16_t* lower; /* HGRN2: bf16 [H * dk] */
+    const uint16_t* head_w; /* bf16 [dv]: per-head norm of the output (prompt: da_finish) */
+    float* state;         /* fp32 [H, dk, dv] */
+    float* q;             /* prompt: fp32 [T, H, dk_p], likewise k and a (padding columns zero) */
+    float* k;
+    float* a;
+    float* o;             /* fp32 [T, H * dv] */
+    void* cat;            /* prompt: bf16 / fp32 rows [T, cat_ld] */
+    int32_t kind, ld, q_off, k_off, v_off, g_off; /* k_off: HGRN2 the gate's section; g_off < 0: no output gate */
+    int32_t a1_off, rank; /* GLA: section of the low-rank pre-activation */
+    int32_t H, dk, dv, dk_p, T, cat_ld, cat_f32;
+    float q_scale, inv_tau, eps;
+} lb_decay_params2;
+
 /* ---- tensor-parallel exchange (comm.cu) ----------------------------------------------- */
 #define LB_TP_MAX 8
 /* Exchange buffer of one rank (every rank maps every peer's): float [2][size][n_max] partial vectors (slot = exchange

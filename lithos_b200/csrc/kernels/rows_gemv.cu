@@ -1,0 +1,195 @@
+// Dense bf16 rows x one fp32 vector for the decode step of bf16 models: one launch takes one or two matrices, builds the input
+// vector(s) in shared memory (RMS norm with the layer's weights; or the mixer's output with its per-head norm and gate, followed
+// by the feed-forward's activations) and finishes every row (store, ReLU-gated product of neighbouring rows, residual add, soft cap
+// with arg-max candidates).  The vector stays fp32; weights are exact in fp32, sums are fp32 in a fixed order.
+//
+// HBM-bound: one CTA per SM, every warp streams its own row segments with 1-D bulk copies through its own ring, so what is in flight
+// (ring bytes x 148) does not depend on registers.  Two rows share every read of the vector: shared memory moves 2 bytes of weights in,
+// 2 out and 2 bytes of vector per weight.  Narrow launches (few pairs per CTA, long rows) cut a pair into segments, one per warp turn;
+// the segments of a pair are added in order, so a result does not depend on the schedule.
+#include "common.cuh"
+#include "params.h"
+
+__device__ __forceinline__ float rg_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const __grid_constant__ lb_rows_gemv_params p) {
+    extern __shared__ __align__(16) unsigned char rg_sm[];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int G = gridDim.x, c = blockIdx.x, S = p.stages;
+    const int pairs0 = (p.mat[0].rows + 1) >> 1, pairs1 = p.n_mat > 1 ? (p.mat[1].rows + 1) >> 1 : 0, P = pairs0 + pairs1;
+    const int my_pairs = P > c ? (P - c + G - 1) / G : 0;
+    const int n_vec = p.x_mode == LB_RG_X_NORM ? p.n_mat : 1;
+    unsigned char* ring = rg_sm;                                                              // [warps][S][2][SEG] bf16
+    float* xsm = reinterpret_cast<float*>(ring + (size_t)LB_RG_WARPS * S * LB_RG_SEG * 4);     // [n_vec][K]
+    float* part = xsm + (size_t)n_vec * p.K;                                                   // [my_pairs * split][2]
+    const int max_pairs = (P + G - 1) / G;
+    float* red = part + (size_t)2 * max_pairs * p.split;                                       // [40]
+    uint64_t* bars = reinterpret_cast<uint64_t*>(red + 40);                                    // [warps][S]
+    if (lane == 0)
+        for (int s = 0; s < S; ++s) mbar_init(&bars[warp * S + s], 1);
+    mbar_fence_init();
+    __syncwarp();
+
+    // the warp's stages: items warp, warp + 8, ... (item = pair * split + piece), segments of the item in order
+    const int items = my_pairs * p.split, spp = p.segs / p.split;
+    const uint64_t pol = l2_policy_evict_first();
+    auto row_ptr = [&](int pair, int& mi) -> const uint16_t* {
+        const int g = c + pair * G;
+        mi = g >= pairs0;
+        return mi ? p.mat[1].w + (size_t)(g - pairs0) * 2 * p.K : p.mat[0].w + (size_t)g * 2 * p.K;
+    };
+    int r_item = warp, r_seg = 0, r_slot = 0; // next stage to request
+    auto request = [&]() {
+        if (r_item >= items) return;
+        if (lane == 0) {
+            const int pair = r_item / p.split, seg = (r_item - pair * p.split) * spp + r_seg;
+            int mi;
+            const uint16_t* w = row_ptr(pair, mi) + (size_t)seg * LB_RG_SEG;
+            const uint32_t bytes = (uint32_t)min(LB_RG_SEG, p.K - seg * LB_RG_SEG) * 2u;
+            unsigned char* dst = ring + (size_t)(warp * S + r_slot) * (LB_RG_SEG * 4);
+            uint64_t* bar = &bars[warp * S + r_slot];
+            mbar_arrive_expect_tx(bar, 2 * bytes);
+            bulk_g2s(dst, w, bytes, bar, pol);
+            bulk_g2s(dst + LB_RG_SEG * 2, w + p.K, bytes, bar, pol);
+        }
+        if (++r_seg == spp) { r_seg = 0; r_item += LB_RG_WARPS; }
+        if (++r_slot == S) r_slot = 0;
+    };
+    for (int s = 0; s < S; ++s) request(); // weights are constants: asked for before the previous kernel has finished
+
+    pdl_wait();
+    if (p.x_mode == LB_RG_X_NORM) {
+        float ss = 0.f;
+#pragma unroll 4
+        for (int i = tid; i < p.K; i += LB_RG_THREADS) {
+            const float v = i < p.width ? p.x[i] : 0.f;
+            xsm[i] = v;
+            ss += v * v;
+        }
+        ss = block_sum(ss, red);
+        const float rinv = 1.0f / sqrtf(ss / (float)p.width + p.eps);
+        const uint16_t *w0 = p.mat[0].norm_w, *w1 = n_vec > 1 ? p.mat[1].norm_w : nullptr;
+#pragma unroll 4
+        for (int i = tid; i < p.width; i += LB_RG_THREADS) {
+            const float v = xsm[i] * rinv;
+            xsm[i] = v * (1.0f + bf16_bits_to_f32(w0[i]));
+            if (w1) xsm[p.K + i] = v * (1.0f + bf16_bits_to_f32(w1[i]));
+        }
+        if (w1)
+            for (int i = p.width + tid; i < p.K; i += LB_RG_THREADS) xsm[p.K + i] = 0.f;
+    } else {
+#pragma unroll 4
+        for (int i = tid; i < p.n_act; i += LB_RG_THREADS) xsm[p.n_mix_pad + i] = p.act[i];
+        for (int i = p.n_mix_pad + p.n_act + tid; i < p.K; i += LB_RG_THREADS) xsm[i] = 0.f;
+        for (int i = p.n_mix + tid; i < p.n_mix_pad; i += LB_RG_THREADS) xsm[i] = 0.f;
+        if (p.head_w) {
+            const int heads = p.n_mix / p.vdim;
+            for (int h = warp; h < heads; h += LB_RG_WARPS) {
+                const float* src = p.mix + (size_t)h * p.vdim;
+                float ss = 0.f;
+                for (int i = lane; i < p.vdim; i += 32) ss += src[i] * src[i];
+                const float rinv = 1.0f / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
+                for (int i = lane; i < p.vdim; i += 32) {
+                    float v = src[i] * rinv * bf16_bits_to_f32(p.head_w[i]);
+                    if (p.gate) {
+                        const float g = p.gate[(size_t)h * p.vdim + i];
+                        v *= g * rg_sigmoid(g);
+                    }
+                    xsm[h * p.vdim + i] = v;
+                }
+            }
+        } else {
+            for (int i = tid; i < p.n_mix; i += LB_RG_THREADS) xsm[i] = p.mix[i];
+        }
+    }
+    __syncthreads();
+    pdl_launch_dependents();
+
+    int slot = 0;
+    uint32_t phase = 0;
+    bool ok = true;
+    for (int item = warp; item < items && ok; item += LB_RG_WARPS) {
+        const int pair = item / p.split, seg0 = (item - pair * p.split) * spp;
+        const float* xv = xsm + ((n_vec > 1 && c + pair * G >= pairs0) ? p.K : 0);
+        float a0 = 0.f, a1 = 0.f, b0 = 0.f, b1 = 0.f;
+        for (int s = 0; s < spp; ++s) {
+            if (!__all_sync(0xffffffffu, mbar_wait(&bars[warp * S + slot], phase))) { // bounded: the rows left keep their old result
+                if (lane == 0 && p.status) atomicExch(p.status, LB_DEV_TIMEOUT_FULL);
+                ok = false;
+                break;
+            }
+            const int k0 = (seg0 + s) * LB_RG_SEG, n8 = min(LB_RG_SEG, p.K - k0) >> 3;
+            const uint4* wa = reinterpret_cast<const uint4*>(ring + (size_t)(warp * S + slot) * (LB_RG_SEG * 4));
+            const uint4* wb = wa + LB_RG_SEG / 8;
+#pragma unroll 4
+            for (int i = lane; i < n8; i += 32) {
+                const uint4 u = wa[i], v = wb[i];
+                const float4 x0 = *reinterpret_cast<const float4*>(xv + k0 + i * 8), x1 = *reinterpret_cast<const float4*>(xv + k0 + i * 8 + 4);
+                a0 = fmaf(__uint_as_float(u.x << 16), x0.x, a0);
+                a1 = fmaf(__uint_as_float(u.x & 0xffff0000u), x0.y, a1);
+                b0 = fmaf(__uint_as_float(v.x << 16), x0.x, b0);
+                b1 = fmaf(__uint_as_float(v.x & 0xffff0000u), x0.y, b1);
+                a0 = fmaf(__uint_as_float(u.y << 16), x0.z, a0);
+                a1 = fmaf(__uint_as_float(u.y & 0xffff0000u), x0.w, a1);
+                b0 = fmaf(__uint_as_float(v.y << 16), x0.z, b0);
+                b1 = fmaf(__uint_as_float(v.y & 0xffff0000u), x0.w, b1);
+                a0 = fmaf(__uint_as_float(u.z << 16), x1.x, a0);
+                a1 = fmaf(__uint_as_float(u.z & 0xffff0000u), x1.y, a1);
+                b0 = fmaf(__uint_as_float(v.z << 16), x1.x, b0);
+                b1 = fmaf(__uint_as_float(v.z & 0xffff0000u), x1.y, b1);
+                a0 = fmaf(__uint_as_float(u.w << 16), x1.z, a0);
+                a1 = fmaf(__uint_as_float(u.w & 0xffff0000u), x1.w, a1);
+                b0 = fmaf(__uint_as_float(v.w << 16), x1.z, b0);
+                b1 = fmaf(__uint_as_float(v.w & 0xffff0000u), x1.w, b1);
+            }
+            __syncwarp(); // every lane has its words in registers (the sums depend on them): the slot can be refilled
+            request();    // the slot just freed is the next one the request cursor fills
+            if (++slot == S) { slot = 0; phase ^= 1u; }
+        }
+        const float ya = warp_sum(a0 + a1), yb = warp_sum(b0 + b1);
+        if (lane == 0) { part[2 * item] = ya; part[2 * item + 1] = yb; }
+    }
+    const bool all_ok = __syncthreads_and(ok ? 1 : 0) != 0;
+
+    float best_v = -INFINITY;
+    int best_i = 0x7fffffff;
+    for (int m = tid; m < my_pairs && all_ok; m += LB_RG_THREADS) {
+        float r[2] = {0.f, 0.f};
+        for (int q = 0; q < p.split; ++q) {
+            r[0] += part[2 * (m * p.split + q)];
+            r[1] += part[2 * (m * p.split + q) + 1];
+        }
+        const int g = c + m * G, mi = g >= pairs0, n = 2 * (mi ? g - pairs0 : g);
+        const lb_rg_mat& M = p.mat[mi];
+        if (M.y_mode == LB_DY_RELU_GLU) {
+            M.y[n >> 1] = fmaxf(r[0], 0.f) * r[1];
+        } else {
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                if (n + e >= M.rows) continue;
+                float v = r[e];
+                if (M.y_mode == LB_DY_RESIDUAL) v = fmaf(p.mult, v, M.y[n + e]);
+                else if (M.y_mode == LB_DY_SOFTCAP && p.cap > 0.f) v = p.cap * tanhf(v / p.cap);
+                M.y[n + e] = v;
+                if (v > best_v || (v == best_v && n + e < best_i)) { best_v = v; best_i = n + e; }
+            }
+        }
+    }
+    if (p.part_val) { // this CTA's candidate for the arg-max: greater value, smaller row on ties
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, best_v, o);
+            const int oi = __shfl_xor_sync(0xffffffffu, best_i, o);
+            if (ov > best_v || (ov == best_v && oi < best_i)) { best_v = ov; best_i = oi; }
+        }
+        int* ri = reinterpret_cast<int*>(red + 16);
+        if (lane == 0) { red[warp] = best_v; ri[warp] = best_i; }
+        __syncthreads();
+        if (tid == 0) {
+            for (int w = 1; w < LB_RG_WARPS; ++w)
+                if (red[w] > best_v || (red[w] == best_v && ri[w] < best_i)) { best_v = red[w]; best_i = ri[w]; }
+            p.part_val[c] = best_v;
+            p.part_idx[c] = best_i;
+        }
+    }
+}
