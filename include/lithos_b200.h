@@ -413,6 +413,21 @@ int lb_model_set_sampling(lb_model* m, float temperature, int top_k, uint64_t se
  * the generated tokens, *n_out their number. */
 int lb_model_generate(lb_model* m, const int* prompt, int n_prompt, int max_new, int eos, int* out, int* n_out);
 
+/* ---- model registry -----------------------------------------------------------------------
+ * A model directory holds config.json and the weights; config.json's "architecture" names the model class:
+ *   "Nufalorn"        bf16 models built from a list of layers (config.json: layers, width, vocab, norm, ...; *.safetensors)
+ *   "Qwen3.5-hybrid"  the int4 hybrid above (config.json: the fields of lb_model_cfg; weight_index.bin, written over the
+ *                     directory's *.safetensors files when missing)
+ * The model is then driven through the same lb_model_* calls, whatever its class.  max_ctx: positions the caches hold.
+ * dtype: LB_DTYPE_BF16 (16-bit matrix operands, fp32 accumulation, fp32 residual, scores and states) or LB_DTYPE_F32
+ * (fp32 throughout; LB_ERR_INVALID for a class without it). */
+enum { LB_DTYPE_BF16 = 0, LB_DTYPE_F32 = 1 };
+int lb_model_open(lb_ctx* ctx, const char* model_dir, int max_ctx, int dtype, lb_model** out);
+/* the same from the text of a config.json, with seeded random weights */
+int lb_model_open_synthetic(lb_ctx* ctx, const char* config_json, int max_ctx, int dtype, uint64_t seed, lb_model** out);
+const char* lb_registry_name(int i);                      /* i-th architecture name, NULL past the last */
+const char* lb_config_images(const char* config_json);    /* kernel images this config's class launches (lb_init_images), or NULL */
+
 #ifdef __cplusplus
 }
 #endif

@@ -35,9 +35,11 @@ class LithosError(RuntimeError):
         self.status = status
 
 
-def build(verbose: bool = False) -> None:
-    """Compile the host library and every kernel image in-tree (make)."""
-    r = subprocess.run(["make", "-C", str(_SRC_DIR), "-j8"], capture_output=True, text=True)
+def build(verbose: bool = False, images=None) -> None:
+    """Compile the host library and every kernel image in-tree (make); images: only these kernel images (names without
+    .cubin; an empty list: the host library alone)."""
+    targets = [] if images is None else [str(_LIB_PATH)] + [str(_HERE / "kernels" / f"{i}.cubin") for i in images]
+    r = subprocess.run(["make", "-C", str(_SRC_DIR), "-j8"] + targets, capture_output=True, text=True)
     if verbose or r.returncode != 0:
         print(r.stdout[-4000:])
         print(r.stderr[-4000:])
@@ -67,6 +69,7 @@ def lib() -> C.CDLL:
     sig("lb_status_string", C.c_char_p, i32)
     sig("lb_version", C.c_char_p)
     sig("lb_init", i32, i32, C.c_char_p, P(vp))
+    sig("lb_init_images", i32, i32, C.c_char_p, C.c_char_p, P(vp))
     sig("lb_destroy", None, vp)
     sig("lb_last_error", C.c_char_p, vp)
     sig("lb_device_sm_count", i32, vp)
@@ -240,9 +243,11 @@ class Graph:
 class Context:
     """One GPU, one stream: the host-side owner of every buffer and launch."""
 
-    def __init__(self, device: int = 0, kernel_dir: str | None = None):
+    def __init__(self, device: int = 0, kernel_dir: str | None = None, images=None):
+        """images: load only these kernel images (model.config_images gives a model's); default all"""
         self.h = C.c_void_p(None)
-        st = lib().lb_init(device, kernel_dir.encode() if kernel_dir else None, C.byref(self.h))
+        st = lib().lb_init_images(device, kernel_dir.encode() if kernel_dir else None, " ".join(images).encode() if images is not None else None,
+                                  C.byref(self.h))
         if st != LB_OK:
             msg = lib().lb_last_error(self.h).decode() if self.h else lib().lb_status_string(st).decode()
             if self.h:

@@ -96,6 +96,7 @@ typedef struct lb_prefill_ws lb_prefill_ws;
 int lb_model_is_fa(const lb_model_cfg* c, int l);
 int lb_model_launch_sampler(lb_model* m);
 int lb_model_alloc_common(lb_model* m); /* the buffers every architecture uses; cfg and vocab_s must be set */
+pf_set* lb_prefill_set(lb_model* m, int s);    /* buffers of prompt stream s (after a prompt pass) */
 int lb_dalloc(lb_model* m, CUdeviceptr* p, size_t bytes);
 int lb_upload(lb_model* m, CUdeviceptr* p, const void* src, size_t bytes);
 #endif

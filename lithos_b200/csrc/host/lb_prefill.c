@@ -56,6 +56,8 @@ static int ws_alloc(lb_model* m) {
     return st;
 }
 
+pf_set* lb_prefill_set(lb_model* m, int s) { return &m->ws->set[s]; }
+
 static int rows_reserve(lb_model* m, int n) {
     lb_prefill_ws* ws = m->ws;
     if (n <= ws->rows_cap) return LB_OK;

@@ -2,6 +2,7 @@
 from __future__ import annotations
 
 import ctypes as C
+import json
 
 import numpy as np
 
@@ -114,14 +115,61 @@ def _sigs():
     L.lb_model_replay.argtypes = [vp, i32]
     L.lb_model_read_next.argtypes = [vp, P(i32)]
     L.lb_model_prefill.argtypes = [vp, P(i32), i32, i32, P(i32)]
+    L.lb_model_forward.argtypes = [vp, P(i32), i32, i32, P(i32), i32, vp]
+    L.lb_model_arch_name.argtypes = [vp]
+    L.lb_model_arch_name.restype = C.c_char_p
+    L.lb_model_config.argtypes = [vp]
+    L.lb_model_config.restype = P(ModelCfg)
+    L.lb_model_open.argtypes = [vp, C.c_char_p, i32, i32, P(vp)]
+    L.lb_model_open_synthetic.argtypes = [vp, C.c_char_p, i32, i32, u64, P(vp)]
     L.lb_model_set_sampling.argtypes = [vp, C.c_float, i32, u64]
     L.lb_model_generate.argtypes = [vp, P(i32), i32, i32, i32, P(i32), P(i32)]
     L.lb_model_step_kernels.argtypes = [vp]
     _sigs_done = True
 
 
+DTYPES = {"bfloat16": 0, "float32": 1}
+
+
+def architectures():
+    """the architecture names of the model registry (config.json's "architecture")"""
+    L, out = lib(), []
+    L.lb_registry_name.restype = C.c_char_p
+    while (n := L.lb_registry_name(len(out))) is not None:
+        out.append(n.decode())
+    return out
+
+
+def config_images(config_json: str):
+    """kernel images the model class of this config.json launches, or None when no class has that architecture"""
+    L = lib()
+    L.lb_config_images.argtypes, L.lb_config_images.restype = [C.c_char_p], C.c_char_p
+    r = L.lb_config_images(config_json.encode())
+    return r.decode().split() if r is not None else None
+
+
 class Model:
     """The decode step on one GPU (or one tensor-parallel shard)."""
+
+    @classmethod
+    def open(cls, ctx: Context, model_dir, max_ctx: int, dtype: str = "bfloat16") -> "Model":
+        """a model directory (config.json + weights) through the model registry"""
+        return cls._from_registry(ctx, lambda h: lib().lb_model_open(ctx.h, str(model_dir).encode(), max_ctx, DTYPES[dtype], h))
+
+    @classmethod
+    def open_synthetic(cls, ctx: Context, config: dict, max_ctx: int, dtype: str = "bfloat16", seed: int = 0) -> "Model":
+        """a config.json (as a dict) with seeded random weights"""
+        text = json.dumps(config).encode()
+        return cls._from_registry(ctx, lambda h: lib().lb_model_open_synthetic(ctx.h, text, max_ctx, DTYPES[dtype], seed, h))
+
+    @classmethod
+    def _from_registry(cls, ctx, call):
+        _sigs()
+        m = cls.__new__(cls)
+        m.ctx, m.tp_rank, m.tp_size, m.h = ctx, 0, 1, C.c_void_p(None)
+        ctx._check(call(C.byref(m.h)))
+        m.cfg = ModelCfg.from_buffer_copy(lib().lb_model_config(m.h).contents)
+        return m
 
     def __init__(self, ctx: Context, cfg: ModelCfg, tp_rank: int = 0, tp_size: int = 1):
         _sigs()
@@ -254,6 +302,18 @@ class Model:
         nxt = C.c_int(0)
         self.ctx._check(lib().lb_model_prefill(self.h, arr, len(tokens), pos0, C.byref(nxt)))
         return nxt.value
+
+    def forward(self, tokens, pos0: int, want=()) -> np.ndarray:
+        """a portion of a sequence (cut anywhere): logits [len(want), vocab] at the wanted places of it"""
+        arr = (C.c_int * len(tokens))(*[int(t) for t in tokens])
+        w = (C.c_int * max(len(want), 1))(*[int(i) for i in want])
+        out = np.empty((len(want), self.cfg.vocab), dtype=np.float32)
+        self.ctx._check(lib().lb_model_forward(self.h, arr, len(tokens), pos0, w, len(want), out.ctypes.data_as(C.c_void_p)))
+        return out
+
+    @property
+    def architecture(self) -> str:
+        return lib().lb_model_arch_name(self.h).decode()
 
     def set_sampling(self, temperature: float, top_k: int, seed: int = 0):
         """top_k == 0: greedy; else temperature / top-k sampling, repeatable from (seed, position)"""
