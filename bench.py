@@ -714,6 +714,106 @@ def bench_prompt_chunks(args, local):
             "config": {"workload": "2 chunks x 256 tokens, positions 3584..4095, 6 DeltaNet + 2 attention layers of the 27B widths, vocabulary 4096"}}
 
 
+# ------------------------------------------------------------------------------------------
+# workload "nufalorn": decode and prompt throughput of the layer-list model at layer sizes of real models, beside the
+# int4 hybrid at equal width, feed-forward and number of layers
+# ------------------------------------------------------------------------------------------
+def nufalorn_config(width, ff, heads, kv_heads, dim, layers, vocab, block):
+    """one period = attention, HGRN2, GLA, GLA; the second attention layer of a pair reads the first one's cache"""
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": block},
+           "rot": {"base": 500000.0, "dims": dim}}
+    rec = {"heads": heads, "dim": dim, "vdim": dim}
+    out = []
+    for i in range(layers):
+        if i % 4 == 0:
+            mixer = dict(att, kv_from=i - 4) if i % 8 == 4 else dict(att)
+            out.append({"type": "attention", "mixer": mixer, "mlp": {"ff": ff, "kind": "dense"}})
+        elif i % 4 == 1:
+            out.append({"type": "hgrn2", "mixer": dict(rec), "mlp": {"ff": ff, "kind": "dense"}})
+        else:
+            out.append({"type": "gla", "mixer": dict(rec, tau=16.0), "mlp": {"ff": ff, "kind": "dense"}})
+    return {"architecture": "Nufalorn", "layers": out, "logit_softcap": 30.0, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "vocab": vocab, "width": width}
+
+
+NUFALORN_SIZES = {  # width, feed-forward, heads, KV heads, head size, and the hybrid of equal size: DeltaNet k / v heads, attention q / kv heads
+    "5120": (5120, 17408, 40, 8, 128, (16, 48, 24, 4)),
+    "4096": (4096, 12288, 32, 8, 128, (16, 32, 16, 4)),
+    "2048": (2048, 8192, 16, 4, 128, (8, 16, 8, 2)),
+}
+
+
+def bench_nufalorn(args, local):
+    import lithos_b200 as lb
+    from lithos_b200 import model as M
+    peak, which = measured_hbm_peak()
+    try:
+        tflops = float(json.loads(PEAKS_FILE.read_text())["bf16_tflops_sustained"])
+    except Exception:
+        tflops = 1400.0
+    n_layers, n_prompt, vocab, block = (8 if args.layers == 64 else args.layers), args.prompt, 32768, 2048
+    steps = min(args.steps, 200)
+    ctx = lb.Context(local)
+    sampler = ClockSampler(local)
+    sampler.start()
+    rows = []
+
+    def timed(m, algo_weights, state_bytes, attended_bytes, macs_per_token, name):
+        toks = [int(t) for t in lb.fill_u32(n_prompt, 3, 999) % vocab]
+        m.prefill(toks)                     # untimed: allocates the prompt-pass buffers, brings the clocks up
+        m.prefill(toks)
+        best = None
+        for _ in range(5):
+            m.reset_state()
+            ctx.timer_start()
+            m.prefill(toks)
+            ms = ctx.timer_stop()
+            best = ms if best is None or ms < best else best
+        m.capture()
+        m.set_input(1, n_prompt)
+        m.replay(max(args.warmup, 10))
+        ctx.sync()
+        ctx.reset_launches()
+        ctx.timer_start()
+        m.replay(steps)
+        ms = ctx.timer_stop() / steps
+        assert ctx.device_status() == 0
+        by = algo_weights + state_bytes + attended_bytes
+        rows.append({"model": name, "decode_ms": round(ms, 4), "decode_tok_s": round(1e3 / ms, 1), "decode_bytes": by,
+                     "decode_frac_of_measured_hbm": round(by / (ms * 1e-3) / 1e9 / peak, 3), "kernels_per_step": m.step_kernels,
+                     "prompt_ms": round(best, 3), "prompt_tok_s": round(n_prompt / best * 1e3),
+                     "prompt_tflops": round(2 * macs_per_token * n_prompt / best / 1e9, 1),
+                     "prompt_frac_of_measured_bf16": round(2 * macs_per_token * n_prompt / best / 1e9 / tflops, 3)})
+
+    for key, (W, F, H, KV, D, (dk, dv, fq, fkv)) in NUFALORN_SIZES.items():
+        if args.sizes and key not in args.sizes.split(","):
+            continue
+        if args.only in ("", "nufalorn"):
+            cfg = nufalorn_config(W, F, H, KV, D, n_layers, vocab, block)
+            m = M.Model.open_synthetic(ctx, cfg, n_prompt + steps + 512, "bfloat16", 5)
+            macs = m.weight_bytes // 2 - vocab * W
+            n_att = sum(l["type"] == "attention" for l in cfg["layers"])
+            seen = (n_prompt % block) + steps // 2 + 1
+            timed(m, m.weight_bytes, (n_layers - n_att) * 2 * H * D * D * 4, n_att * seen * KV * D * 2 * 2, macs, f"Nufalorn {W}x{F}, {n_layers} layers, bf16 weights")
+            m.close()
+        if args.only in ("", "hybrid"):
+            hc = M.ModelCfg(n_layers=n_layers, hidden=W, inter=F, vocab=vocab, dn_k_heads=dk, dn_v_heads=dv, dn_dim=128, conv_taps=4, fa_q_heads=fq, fa_kv_heads=fkv,
+                            fa_dim=256, rot_dims=64, group=128, fa_period=4, max_ctx=n_prompt + steps + 512, reserved=0, eps=1e-6, rope_theta=1e7)
+            m = M.Model(ctx, hc)
+            m.fill_synthetic(5)
+            n_fa = sum(hc.is_fa(l) for l in range(n_layers))
+            n_dn = n_layers - n_fa
+            macs = (n_dn * (W * (hc.conv_channels + dv * 128) + dv * 128 * W) + n_fa * (W * (2 * fq + 2 * fkv) * 256 + fq * 256 * W) + n_layers * 3 * W * F)
+            timed(m, m.weight_bytes, n_dn * 2 * dv * 128 * 128 * 4, n_fa * (n_prompt + steps // 2) * fkv * 256 * 2 * 2, macs, f"hybrid {W}x{F}, {n_layers} layers, int4 weights")
+            m.close()
+    clocks = sampler.stop()
+    ctx.close()
+    return {"metric": "decode and prompt throughput, Nufalorn beside the int4 hybrid of equal size", "value": rows[0]["decode_tok_s"], "unit": "tok/s",
+            "n_gpus": 1, "higher_is_better": True, "data": "synthetic", "rows": rows, "clocks": clocks,
+            "peaks": {"hbm_gbs": peak, "bf16_tflops_sustained": tflops, "source": which},
+            "config": {"prompt_tokens": n_prompt, "decode_steps": steps, "vocab": vocab, "attention_block": block,
+                       "timing": "CUDA events; decode: graph replays back to back; prompt: best of 5; weights of a step exceed L2"}}
+
+
 def bench_chain(args, local):
     """--workload chain: gemv_chain on the decode step's GEMV mix, alone (1.2 GB on the device)"""
     import lithos_b200 as lb
@@ -886,13 +986,16 @@ def main():
     ap.add_argument("--steps", type=int, default=None)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="native", choices=["native", "reference"])
-    ap.add_argument("--workload", default="decode", choices=["decode", "gemv", "chain", "batched", "timeline", "small", "prompt"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "gemv", "chain", "batched", "timeline", "small", "prompt", "nufalorn"],
                     help="decode: the benchmark; gemv: config 0 alone; chain: the decode step's four GEMVs between two token "
                          "mixers as persistent gemv_chain launches alone (the small case used for ncu captures); small: the "
                          "one-figure measurements of configs 0, 1 and 2 alone (the ncu target for the DeltaNet and attention kernels)")
     ap.add_argument("--layers", type=int, default=64, help="decode workload: number of layers (64 = the benchmark definition)")
     ap.add_argument("--batched-shapes", default="", help="batched workload: comma-separated substrings of the shape names to run (default all)")
     ap.add_argument("--batched-batches", default="1,4,16,32,64,128,256", help="batched workload: batch sizes")
+    ap.add_argument("--sizes", default="", help="nufalorn workload: comma-separated widths to run (default all)")
+    ap.add_argument("--only", default="", choices=["", "nufalorn", "hybrid"], help="nufalorn workload: one of the two models")
+    ap.add_argument("--prompt", type=int, default=4096, help="nufalorn workload: prompt tokens")
     ap.add_argument("--seed", type=int, default=20260413)
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     ap.add_argument("--prefill", action="store_true", help="decode workload, 1 GPU: build the 4096-token state by running a seeded random prompt through "
@@ -927,8 +1030,8 @@ def main():
         if rank == 0:
             print(json.dumps(out), flush=True)
         return
-    if args.workload in ("chain", "batched", "prompt"):
-        out = {"chain": bench_chain, "batched": bench_batched, "prompt": bench_prompt_chunks}[args.workload](args, local)
+    if args.workload in ("chain", "batched", "prompt", "nufalorn"):
+        out = {"chain": bench_chain, "batched": bench_batched, "prompt": bench_prompt_chunks, "nufalorn": bench_nufalorn}[args.workload](args, local)
         if rank == 0:
             print(json.dumps(out), flush=True)
         return

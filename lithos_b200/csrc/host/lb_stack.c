@@ -264,7 +264,8 @@ static int launch_rows(lb_model* m, lb_rows_gemv_params* p) {
     p->status = (uint32_t*)c->dev_status;
     size_t smem = 0;
     for (p->stages = 5; p->stages >= 1; p->stages--) {
-        smem = (size_t)LB_RG_WARPS * p->stages * LB_RG_SEG * 4 + (size_t)n_vec * p->K * 4 + (size_t)2 * max_pairs * p->split * 4 + 40 * 4 + (size_t)LB_RG_WARPS * p->stages * 8;
+        smem = (size_t)LB_RG_WARPS * p->stages * LB_RG_SEG * 4 + (size_t)n_vec * p->K * 4 + (size_t)2 * max_pairs * p->split * 4 + 40 * 4 + ((size_t)LB_RG_WARPS * p->stages + 1) * 8 +
+               (p->gate ? (size_t)((p->n_mix + 3) & ~3) * 4 : 0);
         if ((int)smem <= c->max_smem_optin - ((c->fn_static_smem[LBK_rows_gemv] + 1023) & ~1023)) break;
     }
     if (p->stages < 1) return lb_fail(c, LB_ERR_INVALID, "model: a row of %d columns does not fit the decode step's shared memory", p->K);
@@ -401,7 +402,7 @@ static int stack_pf_layer(lb_model* m, pf_set* w, int i, int pos0, int T) {
         p.cat = (void*)w->st.cat; p.cat_ld = L->out.K; p.cat_f32 = f32;
         void* params[] = {&p};
         LB_TRY(lb_launch(c, LBK_da_inputs, (unsigned)((D->heads * L->dk_p + 255) / 256), (unsigned)((T + 7) / 8), 1, 256, (unsigned)(8 * (D->rank > 0 ? D->rank : 1) * 4), params, 1));
-        const int R = L->dk_p / 4, tok = 3 * 4 * (R + 4) + 32;
+        const int tok = 3 * (L->dk_p + 8 * 4) + 32; /* floats a token's operands take in a stage */
         LB_TRY(lb_launch(c, L->dk_p == 64 ? LBK_da_scan_64 : L->dk_p == 128 ? LBK_da_scan_128 : LBK_da_scan_256, (unsigned)D->heads, (unsigned)((D->vdim + 31) / 32), 1, 128,
                          (unsigned)(3 * 4 * tok * 4), params, 1));
         LB_TRY(lb_launch(c, LBK_da_finish, (unsigned)T, (unsigned)((D->heads + 3) / 4), 1, 128, 0, params, 1));

@@ -2,7 +2,7 @@
 //   HGRN2: f = l + (1 - l) sigmoid(z + b), a = f, k = 1 - f, q = silu(zq)
 //   GLA:   a = sigmoid(W2 (W1 h) + b)^(1/tau), k = zk, q = dk^-1/2 zq
 // A column j of a head's state needs only v_j, so a CTA owns a 32-column slab of one head and holds it in registers: thread (column,
-// row quarter) has R rows of its column (4 R >= dk; rows past dk stay zero), the sum over rows is R local terms and two shuffles.
+// row part) has R rows of its column (rows past dk stay zero), the sum over rows is local terms and a few shuffles.
 //   da_step_*   one token (decode): makes q, k, a of its head from the projections, state read and written once
 //   da_inputs   a prompt chunk's q, k, a
 //   da_scan_*   a prompt chunk through the recurrence, the state on chip for all of it
@@ -120,8 +120,11 @@ extern "C" __global__ void __launch_bounds__(256) da_inputs(const __grid_constan
     pdl_launch_dependents();
 }
 
-// grid (H, ceil(dv / 32)), block 128.  Operands of DA_U tokens at a time come DA_AHEAD stages ahead by cp.async (a row quarter of q, k, a
-// is padded by 16 bytes so that the four quarters sit on different banks); one block barrier per DA_U tokens.
+// grid (H, ceil(dv / 32)), block 128.  Thread (column pair, row eighth) holds R = dk_p / 8 rows of two columns as packed pairs of
+// rows, so that the state update and the read-out are two-wide fp32 instructions and a row of q, k, a is read from shared memory once for
+// two columns.  Operands of DA_U tokens at a time come DA_AHEAD - 1 stages ahead by cp.async (a row eighth is padded by 16 bytes: the eight
+// addresses of a warp's 16-byte reads sit on different banks); one block barrier per DA_U tokens, and no branch between the tokens of a
+// full stage, so that the next token's operands are read under the present one's arithmetic.
 #define DA_U 4
 #define DA_AHEAD 3
 __device__ __forceinline__ void da_cp16(void* dst, const void* src) {
@@ -130,22 +133,45 @@ __device__ __forceinline__ void da_cp16(void* dst, const void* src) {
 __device__ __forceinline__ void da_cp4(void* dst, const void* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
+typedef unsigned long long da_f2; // two fp32 values
+__device__ __forceinline__ da_f2 da_pack(float x, float y) {
+    da_f2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+    return r;
+}
+__device__ __forceinline__ float2 da_unpack(da_f2 v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ da_f2 da_fma2(da_f2 a, da_f2 b, da_f2 c) {
+    da_f2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ da_f2 da_mul2(da_f2 a, da_f2 b) {
+    da_f2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+struct __align__(16) da_quad { da_f2 lo, hi; }; // four consecutive rows
+
 template <int R>
 __device__ __forceinline__ void da_scan_body(const lb_decay_params2& p) {
-    constexpr int QS = R + 4, VEC = 4 * QS, TOK = 3 * VEC + DA_COLS; // floats: a row quarter, a vector, a token's operands
+    constexpr int QS = R + 4, VEC = 8 * QS, TOK = 3 * VEC + DA_COLS; // floats: a row eighth, a vector, a token's operands
     extern __shared__ __align__(16) float da_sm[];                   // [DA_AHEAD][DA_U][TOK]
-    const int h = blockIdx.x, t = threadIdx.x, q4 = t & 3, jl = t >> 2, j = blockIdx.y * DA_COLS + jl;
-    const bool live = j < p.dv;
-    float* S = p.state + ((size_t)h * p.dk + (size_t)q4 * R) * p.dv + j;
-    const int rows = min(R, p.dk - q4 * R);
+    const int h = blockIdx.x, t = threadIdx.x, e8 = t & 7, j = blockIdx.y * DA_COLS + 2 * (t >> 3);
+    const bool live0 = j < p.dv, live1 = j + 1 < p.dv;
+    float* S = p.state + ((size_t)h * p.dk + (size_t)e8 * R) * p.dv + j;
+    const int rows = min(R, p.dk - e8 * R);
     pdl_wait();
     const int n_st = (p.T + DA_U - 1) / DA_U;
     auto fetch = [&](int st) {
         float* dst = da_sm + (size_t)(st % DA_AHEAD) * (DA_U * TOK);
-        constexpr int PIECES = 3 * R; // 16-byte pieces of q, k, a (4 R floats each)
+        constexpr int PIECES = 3 * 2 * R; // 16-byte pieces of q, k, a (8 R floats each)
         for (int i = t; i < DA_U * PIECES; i += DA_THREADS) {
-            const int u = i / PIECES, c = i - u * PIECES, which = c / R, pc = c - which * R, tok = min(st * DA_U + u, p.T - 1);
-            const float* src = (which == 0 ? p.q : which == 1 ? p.k : p.a) + ((size_t)tok * p.H + h) * (4 * R) + pc * 4;
+            const int u = i / PIECES, c = i - u * PIECES, which = c / (2 * R), pc = c - which * (2 * R), tok = min(st * DA_U + u, p.T - 1);
+            const float* src = (which == 0 ? p.q : which == 1 ? p.k : p.a) + ((size_t)tok * p.H + h) * (8 * R) + pc * 4;
             da_cp16(dst + u * TOK + which * VEC + (pc / (R / 4)) * QS + (pc % (R / 4)) * 4, src);
         }
         { // DA_U x 32 values: one per thread
@@ -159,59 +185,83 @@ __device__ __forceinline__ void da_scan_body(const lb_decay_params2& p) {
         if (st < n_st) fetch(st);
         else asm volatile("cp.async.commit_group;" ::: "memory");
     }
-    float s[R];
+    da_f2 s0[R / 2], s1[R / 2]; // rows (2r, 2r + 1) of the two columns
 #pragma unroll
-    for (int r = 0; r < R; ++r) s[r] = live && r < rows ? S[(size_t)r * p.dv] : 0.f;
+    for (int r = 0; r < R; r += 2) {
+        auto at = [&](int rr, int c, bool on) { return on && rr < rows ? S[(size_t)rr * p.dv + c] : 0.f; };
+        s0[r / 2] = da_pack(at(r, 0, live0), at(r + 1, 0, live0));
+        s1[r / 2] = da_pack(at(r, 1, live1), at(r + 1, 1, live1));
+    }
+    auto step = [&](const float* tk, float& o0, float& o1) { // one token: state update, this thread's share of the two read-outs
+        const float2 v = *reinterpret_cast<const float2*>(tk + 3 * VEC + 2 * (t >> 3));
+        const da_f2 v0 = da_pack(v.x, v.x), v1 = da_pack(v.y, v.y);
+        const da_quad *qv = reinterpret_cast<const da_quad*>(tk + e8 * QS), *kv = reinterpret_cast<const da_quad*>(tk + VEC + e8 * QS),
+                      *av = reinterpret_cast<const da_quad*>(tk + 2 * VEC + e8 * QS);
+        da_f2 a0 = 0ull, a1 = 0ull, b0 = 0ull, b1 = 0ull;
+#pragma unroll
+        for (int c = 0; c < R / 4; ++c) {
+            const da_quad q = qv[c], k = kv[c], a = av[c];
+            s0[2 * c] = da_fma2(a.lo, s0[2 * c], da_mul2(k.lo, v0));
+            s1[2 * c] = da_fma2(a.lo, s1[2 * c], da_mul2(k.lo, v1));
+            s0[2 * c + 1] = da_fma2(a.hi, s0[2 * c + 1], da_mul2(k.hi, v0));
+            s1[2 * c + 1] = da_fma2(a.hi, s1[2 * c + 1], da_mul2(k.hi, v1));
+            a0 = da_fma2(s0[2 * c], q.lo, a0);
+            b0 = da_fma2(s1[2 * c], q.lo, b0);
+            a1 = da_fma2(s0[2 * c + 1], q.hi, a1);
+            b1 = da_fma2(s1[2 * c + 1], q.hi, b1);
+        }
+        const float2 x0 = da_unpack(a0), x1 = da_unpack(a1), y0 = da_unpack(b0), y1 = da_unpack(b1);
+        o0 = (x0.x + x0.y) + (x1.x + x1.y);
+        o1 = (y0.x + y0.y) + (y1.x + y1.y);
+    };
     for (int st = 0; st < n_st; ++st) {
         asm volatile("cp.async.wait_group %0;" ::"n"(DA_AHEAD - 2) : "memory");
         __syncthreads(); // everybody's pieces have landed, and everybody is done with the stage the next fetch fills
         if (st + DA_AHEAD - 1 < n_st) fetch(st + DA_AHEAD - 1);
         else asm volatile("cp.async.commit_group;" ::: "memory");
         const float* base = da_sm + (size_t)(st % DA_AHEAD) * (DA_U * TOK);
-        float o[DA_U];
+        float o[2 * DA_U]; // [token][column]
+        if ((st + 1) * DA_U <= p.T) {
 #pragma unroll
-        for (int u = 0; u < DA_U; ++u) {
-            const bool act = st * DA_U + u < p.T; // tokens past the chunk leave the state alone
-            const float* tk = base + u * TOK;
-            const float v = tk[3 * VEC + jl];
-            const float4 *qv = reinterpret_cast<const float4*>(tk + q4 * QS), *kv = reinterpret_cast<const float4*>(tk + VEC + q4 * QS),
-                         *av = reinterpret_cast<const float4*>(tk + 2 * VEC + q4 * QS);
-            float o0 = 0.f, o1 = 0.f;
-            if (act) {
+            for (int u = 0; u < DA_U; ++u) step(base + u * TOK, o[2 * u], o[2 * u + 1]);
+        } else { // the chunk ends inside this stage: tokens past it leave the state alone
 #pragma unroll
-                for (int c = 0; c < R / 4; ++c) {
-                    const float4 q = qv[c], k = kv[c], a = av[c];
-                    s[4 * c] = fmaf(a.x, s[4 * c], k.x * v);
-                    s[4 * c + 1] = fmaf(a.y, s[4 * c + 1], k.y * v);
-                    s[4 * c + 2] = fmaf(a.z, s[4 * c + 2], k.z * v);
-                    s[4 * c + 3] = fmaf(a.w, s[4 * c + 3], k.w * v);
-                    o0 = fmaf(s[4 * c], q.x, o0);
-                    o1 = fmaf(s[4 * c + 1], q.y, o1);
-                    o0 = fmaf(s[4 * c + 2], q.z, o0);
-                    o1 = fmaf(s[4 * c + 3], q.w, o1);
-                }
+            for (int u = 0; u < DA_U; ++u) {
+                o[2 * u] = o[2 * u + 1] = 0.f;
+                if (st * DA_U + u < p.T) step(base + u * TOK, o[2 * u], o[2 * u + 1]);
             }
-            o[u] = o0 + o1;
         }
+        // sums over the column's eight lanes: every exchange halves what a lane still holds, lane e8 ends with (token e8 / 2, column e8 & 1)
 #pragma unroll
-        for (int u = 0; u < DA_U; ++u) {
-            o[u] += __shfl_xor_sync(0xffffffffu, o[u], 1);
-            o[u] += __shfl_xor_sync(0xffffffffu, o[u], 2);
+        for (int half = 4; half >= 1; half >>= 1) {
+            const bool up = (e8 & half) != 0;
+#pragma unroll
+            for (int i = 0; i < half; ++i) {
+                const float give = up ? o[i] : o[i + half], keep = up ? o[i + half] : o[i];
+                o[i] = keep + __shfl_xor_sync(0xffffffffu, give, half);
+            }
         }
-        // lane q4 of a column stores token q4 of the four
-        const float mine = q4 == 0 ? o[0] : q4 == 1 ? o[1] : q4 == 2 ? o[2] : o[3];
-        const int tok = st * DA_U + q4;
-        if (live && tok < p.T) p.o[(size_t)tok * p.H * p.dv + (size_t)h * p.dv + j] = mine;
+        const int tok = st * DA_U + (e8 >> 1), col = j + (e8 & 1);
+        if (col < p.dv && tok < p.T) p.o[(size_t)tok * p.H * p.dv + (size_t)h * p.dv + col] = o[0];
     }
     pdl_launch_dependents();
 #pragma unroll
-    for (int r = 0; r < R; ++r)
-        if (live && r < rows) S[(size_t)r * p.dv] = s[r];
+    for (int r = 0; r < R; r += 2) {
+        const float2 x = da_unpack(s0[r / 2]), y = da_unpack(s1[r / 2]);
+        if (r < rows) {
+            if (live0) S[(size_t)r * p.dv] = x.x;
+            if (live1) S[(size_t)r * p.dv + 1] = y.x;
+        }
+        if (r + 1 < rows) {
+            if (live0) S[(size_t)(r + 1) * p.dv] = x.y;
+            if (live1) S[(size_t)(r + 1) * p.dv + 1] = y.y;
+        }
+    }
 }
-static_assert(DA_U == 4 && DA_THREADS == 32 * DA_U, "one value per thread and stage; one token per lane of a column");
-extern "C" __global__ void __launch_bounds__(DA_THREADS) da_scan_64(const __grid_constant__ lb_decay_params2 p) { da_scan_body<16>(p); }
-extern "C" __global__ void __launch_bounds__(DA_THREADS) da_scan_128(const __grid_constant__ lb_decay_params2 p) { da_scan_body<32>(p); }
-extern "C" __global__ void __launch_bounds__(DA_THREADS) da_scan_256(const __grid_constant__ lb_decay_params2 p) { da_scan_body<64>(p); }
+static_assert(DA_U == 4 && DA_THREADS == 32 * DA_U, "one value per thread and stage; two tokens' columns per lane of a column pair");
+extern "C" __global__ void __launch_bounds__(DA_THREADS) da_scan_64(const __grid_constant__ lb_decay_params2 p) { da_scan_body<8>(p); }
+extern "C" __global__ void __launch_bounds__(DA_THREADS) da_scan_128(const __grid_constant__ lb_decay_params2 p) { da_scan_body<16>(p); }
+extern "C" __global__ void __launch_bounds__(DA_THREADS) da_scan_256(const __grid_constant__ lb_decay_params2 p) { da_scan_body<32>(p); }
 
 // cat[t, h dv + i] = o / rms_head(o) * head_w[i] [ * silu(gate) ].  grid (T, ceil(H / 4)), block 128: one warp per (token, head)
 extern "C" __global__ void __launch_bounds__(128) da_finish(const __grid_constant__ lb_decay_params2 p) {

@@ -21,14 +21,16 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
     const int n_vec = p.x_mode == LB_RG_X_NORM ? p.n_mat : 1;
     unsigned char* ring = rg_sm;                                                              // [warps][S][2][SEG] bf16
     float* xsm = reinterpret_cast<float*>(ring + (size_t)LB_RG_WARPS * S * LB_RG_SEG * 4);     // [n_vec][K]
-    float* part = xsm + (size_t)n_vec * p.K;                                                   // [my_pairs * split][2]
+    float* gate_s = xsm + (size_t)n_vec * p.K;                                                 // [n_mix] when there is a gate
+    float* part = gate_s + (p.gate ? (p.n_mix + 3) & ~3 : 0);                                  // [my_pairs * split][2]
     const int max_pairs = (P + G - 1) / G;
     float* red = part + (size_t)2 * max_pairs * p.split;                                       // [40]
-    uint64_t* bars = reinterpret_cast<uint64_t*>(red + 40);                                    // [warps][S]
+    uint64_t* bars = reinterpret_cast<uint64_t*>(red + 40);                                    // [warps][S], the vector's
     if (lane == 0)
         for (int s = 0; s < S; ++s) mbar_init(&bars[warp * S + s], 1);
+    if (tid == 0) mbar_init(&bars[LB_RG_WARPS * S], 1);
     mbar_fence_init();
-    __syncwarp();
+    __syncthreads();
 
     // the warp's stages: items warp, warp + 8, ... (item = pair * split + piece), segments of the item in order
     const int items = my_pairs * p.split, spp = p.segs / p.split;
@@ -57,49 +59,101 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
     };
     for (int s = 0; s < S; ++s) request(); // weights are constants: asked for before the previous kernel has finished
 
+    // the norm weights are constants too: a thread's first 8 quads of them come in before the wait
+    const bool quads = (p.width & 3) == 0;
+    uint2 w_pre[2][8];
+    if (p.x_mode == LB_RG_X_NORM && quads) {
+#pragma unroll
+        for (int v = 0; v < 2; ++v)
+#pragma unroll
+            for (int u = 0; u < 8; ++u) {
+                const int i = 4 * (tid + u * LB_RG_THREADS);
+                w_pre[v][u] = v < n_vec && i < p.width ? __ldg(reinterpret_cast<const uint2*>(p.mat[v].norm_w + i)) : make_uint2(0u, 0u);
+            }
+    }
+    // the vector's parts come as bulk copies straight into its place (whole 16-byte pieces; what is left over by plain loads), so the
+    // launch waits for one trip to L2 and not for as many as a thread has loads in turn
+    uint64_t* xbar = bars + LB_RG_WARPS * S;
     pdl_wait();
     if (p.x_mode == LB_RG_X_NORM) {
+        const int n4 = p.width & ~3;
+        if (tid == 0) {
+            mbar_arrive_expect_tx(xbar, (uint32_t)n4 * 4u);
+            if (n4) bulk_g2s_plain(xsm, p.x, (uint32_t)n4 * 4u, xbar);
+        }
+        for (int i = n4 + tid; i < p.width; i += LB_RG_THREADS) xsm[i] = p.x[i];
+        for (int i = p.width + tid; i < p.K; i += LB_RG_THREADS) {
+            xsm[i] = 0.f;
+            if (n_vec > 1) xsm[p.K + i] = 0.f;
+        }
+        const bool here = mbar_wait(xbar, 0);
+        if (!here && p.status) atomicExch(p.status, LB_DEV_TIMEOUT_FULL);
+        __syncthreads();
         float ss = 0.f;
-#pragma unroll 4
-        for (int i = tid; i < p.K; i += LB_RG_THREADS) {
-            const float v = i < p.width ? p.x[i] : 0.f;
-            xsm[i] = v;
-            ss += v * v;
+        for (int i = tid; i < p.K / 4; i += LB_RG_THREADS) {
+            const float4 v = *reinterpret_cast<const float4*>(xsm + 4 * i);
+            ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
         }
         ss = block_sum(ss, red);
         const float rinv = 1.0f / sqrtf(ss / (float)p.width + p.eps);
-        const uint16_t *w0 = p.mat[0].norm_w, *w1 = n_vec > 1 ? p.mat[1].norm_w : nullptr;
-#pragma unroll 4
-        for (int i = tid; i < p.width; i += LB_RG_THREADS) {
-            const float v = xsm[i] * rinv;
-            xsm[i] = v * (1.0f + bf16_bits_to_f32(w0[i]));
-            if (w1) xsm[p.K + i] = v * (1.0f + bf16_bits_to_f32(w1[i]));
+        if (quads) {
+            auto apply = [&](int i, uint2 a, uint2 b) { // quad at i with the norm weights of the one or two vectors
+                float4 v = *reinterpret_cast<const float4*>(xsm + i);
+                v.x *= rinv; v.y *= rinv; v.z *= rinv; v.w *= rinv;
+                auto scaled = [&](uint2 w) {
+                    return make_float4(v.x * (1.0f + __uint_as_float(w.x << 16)), v.y * (1.0f + __uint_as_float(w.x & 0xffff0000u)),
+                                       v.z * (1.0f + __uint_as_float(w.y << 16)), v.w * (1.0f + __uint_as_float(w.y & 0xffff0000u)));
+                };
+                *reinterpret_cast<float4*>(xsm + i) = scaled(a);
+                if (n_vec > 1) *reinterpret_cast<float4*>(xsm + p.K + i) = scaled(b);
+            };
+#pragma unroll
+            for (int u = 0; u < 8; ++u) {
+                const int i = 4 * (tid + u * LB_RG_THREADS);
+                if (i < p.width) apply(i, w_pre[0][u], w_pre[1][u]);
+            }
+            for (int i = 4 * (tid + 8 * LB_RG_THREADS); i < p.width; i += 4 * LB_RG_THREADS)
+                apply(i, *reinterpret_cast<const uint2*>(p.mat[0].norm_w + i), n_vec > 1 ? *reinterpret_cast<const uint2*>(p.mat[1].norm_w + i) : make_uint2(0u, 0u));
+        } else {
+            for (int i = tid; i < p.width; i += LB_RG_THREADS) {
+                const float v = xsm[i] * rinv;
+                xsm[i] = v * (1.0f + bf16_bits_to_f32(p.mat[0].norm_w[i]));
+                if (n_vec > 1) xsm[p.K + i] = v * (1.0f + bf16_bits_to_f32(p.mat[1].norm_w[i]));
+            }
         }
-        if (w1)
-            for (int i = p.width + tid; i < p.K; i += LB_RG_THREADS) xsm[p.K + i] = 0.f;
     } else {
-#pragma unroll 4
-        for (int i = tid; i < p.n_act; i += LB_RG_THREADS) xsm[p.n_mix_pad + i] = p.act[i];
+        const int m4 = p.n_mix & ~3, a4 = p.n_act & ~3, g4 = p.gate && (reinterpret_cast<size_t>(p.gate) & 15) == 0 ? m4 : 0;
+        if (tid == 0) {
+            mbar_arrive_expect_tx(xbar, (uint32_t)(m4 + a4 + g4) * 4u);
+            if (m4) bulk_g2s_plain(xsm, p.mix, (uint32_t)m4 * 4u, xbar);
+            if (g4) bulk_g2s_plain(gate_s, p.gate, (uint32_t)g4 * 4u, xbar);
+            if (a4) bulk_g2s_plain(xsm + p.n_mix_pad, p.act, (uint32_t)a4 * 4u, xbar);
+        }
+        for (int i = m4 + tid; i < p.n_mix; i += LB_RG_THREADS) xsm[i] = p.mix[i];
+        if (p.gate)
+            for (int i = g4 + tid; i < p.n_mix; i += LB_RG_THREADS) gate_s[i] = p.gate[i];
+        for (int i = a4 + tid; i < p.n_act; i += LB_RG_THREADS) xsm[p.n_mix_pad + i] = p.act[i];
         for (int i = p.n_mix_pad + p.n_act + tid; i < p.K; i += LB_RG_THREADS) xsm[i] = 0.f;
         for (int i = p.n_mix + tid; i < p.n_mix_pad; i += LB_RG_THREADS) xsm[i] = 0.f;
+        const bool here = mbar_wait(xbar, 0);
+        if (!here && p.status) atomicExch(p.status, LB_DEV_TIMEOUT_FULL);
+        __syncthreads();
         if (p.head_w) {
             const int heads = p.n_mix / p.vdim;
             for (int h = warp; h < heads; h += LB_RG_WARPS) {
-                const float* src = p.mix + (size_t)h * p.vdim;
+                float* o = xsm + (size_t)h * p.vdim;
                 float ss = 0.f;
-                for (int i = lane; i < p.vdim; i += 32) ss += src[i] * src[i];
+                for (int i = lane; i < p.vdim; i += 32) ss += o[i] * o[i];
                 const float rinv = 1.0f / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
                 for (int i = lane; i < p.vdim; i += 32) {
-                    float v = src[i] * rinv * bf16_bits_to_f32(p.head_w[i]);
+                    float v = o[i] * rinv * bf16_bits_to_f32(__ldg(p.head_w + i));
                     if (p.gate) {
-                        const float g = p.gate[(size_t)h * p.vdim + i];
+                        const float g = gate_s[h * p.vdim + i];
                         v *= g * rg_sigmoid(g);
                     }
-                    xsm[h * p.vdim + i] = v;
+                    o[i] = v;
                 }
             }
-        } else {
-            for (int i = tid; i < p.n_mix; i += LB_RG_THREADS) xsm[i] = p.mix[i];
         }
     }
     __syncthreads();
