@@ -213,6 +213,15 @@ static int load_layer(lb_model* m, lb_weight_source* src, int i) {
 static int heads_per_cta(const lb_stack_layer* D) { const int G = D->heads / D->kv_heads; return G <= 2 ? 2 : G <= 4 ? 4 : 8; }
 static int head_groups(const lb_stack_layer* D) { const int G = D->heads / D->kv_heads, g = heads_per_cta(D); return (G + g - 1) / g; }
 
+static int rows_smem(int gh, int warps, int dim_p, int vdim_p, int esz) { /* as wattn_rows lays it out */
+    return gh * dim_p * 4 + warps * gh * vdim_p * 4 + (dim_p + vdim_p) * esz + warps * 32 * ((dim_p + vdim_p) * esz + 32);
+}
+static int rows_warps(const stack_t* S, const lb_stack_layer* D, int dim_p, int vdim_p) { /* 4, or as many as shared memory holds tiles for */
+    int w = 4;
+    while (w > 1 && rows_smem(heads_per_cta(D), w, dim_p, vdim_p, S->esz) > 200 * 1024) w--;
+    return w;
+}
+
 static void fill_wattn(const lb_model* m, int i, lb_wattn_params* p, CUdeviceptr proj) {
     const stack_t* S = S_of(m);
     const lb_stack_layer* D = &S->d.layer[i];
@@ -235,9 +244,10 @@ static int launch_wattn_rows(lb_model* m, int i, const lb_wattn_params* p) {
     const int gh = heads_per_cta(D), wide = p->vdim_p > 128, f32 = S->esz == 4;
     static const int k[2][2][3] = {{{LBK_wattn_rows_b2n2, LBK_wattn_rows_b4n2, LBK_wattn_rows_b8n2}, {LBK_wattn_rows_b2n4, LBK_wattn_rows_b4n4, LBK_wattn_rows_b8n4}},
                                    {{LBK_wattn_rows_f2n2, LBK_wattn_rows_f4n2, LBK_wattn_rows_f8n2}, {LBK_wattn_rows_f2n4, LBK_wattn_rows_f4n4, LBK_wattn_rows_f8n4}}};
-    const unsigned smem = (unsigned)(gh * p->dim_p * 4 + 8 * gh * p->vdim_p * 4 + (p->dim_p + p->vdim_p) * S->esz);
+    const int warps = rows_warps(S, D, p->dim_p, p->vdim_p);
+    const unsigned smem = (unsigned)rows_smem(gh, warps, p->dim_p, p->vdim_p, S->esz);
     void* params[] = {(void*)p};
-    return lb_launch(m->c, k[f32][wide][gh == 2 ? 0 : gh == 4 ? 1 : 2], (unsigned)(D->kv_heads * head_groups(D)), (unsigned)p->splits, (unsigned)p->T, 256, smem, params, 1);
+    return lb_launch(m->c, k[f32][wide][gh == 2 ? 0 : gh == 4 ? 1 : 2], (unsigned)(D->kv_heads * head_groups(D)), (unsigned)p->splits, (unsigned)p->T, (unsigned)(32 * warps), smem, params, 1);
 }
 
 static void fill_decay(const lb_model* m, int i, lb_decay_params2* p, CUdeviceptr proj) {
@@ -253,24 +263,33 @@ static void fill_decay(const lb_model* m, int i, lb_decay_params2* p, CUdevicept
     p->q_scale = (float)(1.0 / sqrt((double)D->dim)); p->inv_tau = D->decay == LB_DA_GLA ? (float)(1.0 / D->tau) : 0.f; p->eps = (float)S->d.eps;
 }
 
-/* one launch of rows_gemv: ring depth and row splitting from what shared memory holds */
+/* one launch of rows_gemv: ring depth and row splitting from what shared memory holds; two CTAs per row where one vector would leave the
+ * ring fewer than five stages (the mixer's part must lie in the first half) */
 static int launch_rows(lb_model* m, lb_rows_gemv_params* p) {
     lb_ctx* c = m->c;
     int P = 0;
     for (int i = 0; i < p->n_mat; i++) P += (p->mat[i].rows + 1) / 2;
-    const int max_pairs = (P + c->sm_count - 1) / c->sm_count, n_vec = p->x_mode == LB_RG_X_NORM ? p->n_mat : 1;
+    const int n_vec = p->x_mode == LB_RG_X_NORM ? p->n_mat : 1, limit = c->max_smem_optin - ((c->fn_static_smem[LBK_rows_gemv] + 1023) & ~1023);
     p->segs = (p->K + LB_RG_SEG - 1) / LB_RG_SEG;
-    p->split = max_pairs >= 64 ? 1 : p->segs;
     p->status = (uint32_t*)c->dev_status;
+    const int can_halve = p->x_mode == LB_RG_X_CAT && p->n_mix_pad <= p->segs / 2 * LB_RG_SEG && c->sm_count % 2 == 0;
     size_t smem = 0;
-    for (p->stages = 5; p->stages >= 1; p->stages--) {
-        smem = (size_t)LB_RG_WARPS * p->stages * LB_RG_SEG * 4 + (size_t)n_vec * p->K * 4 + (size_t)2 * max_pairs * p->split * 4 + 40 * 4 + ((size_t)LB_RG_WARPS * p->stages + 1) * 8 +
-               (p->gate ? (size_t)((p->n_mix + 3) & ~3) * 4 : 0);
-        if ((int)smem <= c->max_smem_optin - ((c->fn_static_smem[LBK_rows_gemv] + 1023) & ~1023)) break;
+    int ks = 1;
+    for (ks = 1; ks <= 1 + can_halve; ks++) {
+        const int ctas = c->sm_count / ks, max_pairs = (P + ctas - 1) / ctas, segs = (p->segs + ks - 1) / ks;
+        p->x_cols = ks == 1 ? p->K : segs * LB_RG_SEG;
+        p->split = max_pairs >= 64 ? 1 : segs;
+        for (p->stages = 5; p->stages >= 1; p->stages--) {
+            smem = (size_t)LB_RG_WARPS * p->stages * LB_RG_SEG * 4 + (size_t)n_vec * p->x_cols * 4 + (p->gate ? (size_t)((p->n_mix + 3) & ~3) * 4 : 0) +
+                   (size_t)2 * max_pairs * p->split * 4 + 40 * 4 + ((size_t)LB_RG_WARPS * p->stages + 1) * 8;
+            if ((int)smem <= limit) break;
+        }
+        if (p->stages == 5) break;
     }
+    if (ks > 1 + can_halve) ks = 1 + can_halve;
     if (p->stages < 1) return lb_fail(c, LB_ERR_INVALID, "model: a row of %d columns does not fit the decode step's shared memory", p->K);
     void* params[] = {p};
-    return lb_launch(c, LBK_rows_gemv, (unsigned)c->sm_count, 1, 1, LB_RG_THREADS, (unsigned)smem, params, 1);
+    return lb_launch_cluster(c, LBK_rows_gemv, (unsigned)(c->sm_count / ks), (unsigned)ks, 1, LB_RG_THREADS, (unsigned)smem, params, 1, (unsigned)ks);
 }
 
 /* one or two products Y = X W^T of a chunk (w[1] may be NULL) */
@@ -333,7 +352,7 @@ static int stack_step_layers(lb_model* m) {
             p.o = (float*)S->mix;
             void* params[] = {&p};
             LB_TRY(lb_launch(m->c, L->dk_p == 64 ? LBK_da_step_64 : L->dk_p == 128 ? LBK_da_step_128 : LBK_da_step_256, (unsigned)D->heads,
-                             (unsigned)((D->vdim + 31) / 32), 1, 128, 0, params, 1));
+                             (unsigned)((D->vdim + 31) / 32), 1, 128, D->decay == LB_DA_GLA ? (unsigned)(D->dim * D->rank * 2) : 0u, params, 1));
             g.head_w = (const uint16_t*)L->head_norm; g.vdim = D->vdim;
             if (L->g_off >= 0) g.gate = (const float*)(S->proj + (size_t)L->g_off * 4);
         }
@@ -512,9 +531,11 @@ static int stack_build(lb_model* m, const lb_stack_desc* d, lb_weight_source* sr
         MAX(S->max_in, L->in.rows); MAX(S->max_cat, L->out.K); MAX(S->max_mix, L->n_mix); MAX(S->max_ff, D->ff);
         if (D->mixer == LB_MIX_ATTENTION) {
             MAX(S->max_q, D->heads * L->dim_p);
-            /* slices of the decode attention: 256 rows (one block of 32 per warp) each, as many as keep one CTA per SM */
+            /* slices of the decode attention: one tile of 32 rows per warp each, as many as keep one CTA per SM */
             const int groups = D->kv_heads * head_groups(D), seen = D->block && D->block < d->max_ctx ? D->block : d->max_ctx;
-            L->splits = (seen + 255) / 256;
+            const int slice = 32 * rows_warps(S, D, L->dim_p, L->vdim_p);
+            L->splits = (seen + slice - 1) / slice;
+            if (L->splits > LB_WA_MAX_SPLITS) L->splits = LB_WA_MAX_SPLITS;
             if (L->splits * groups > c->sm_count) L->splits = c->sm_count / groups;
             if (L->splits < 1) L->splits = 1;
             const size_t n = (size_t)groups * L->splits * heads_per_cta(D) * (L->vdim_p + 2) * 4;

@@ -37,39 +37,49 @@ __device__ __forceinline__ float da_dot_rank(const uint16_t* w, const float* x, 
     return s;
 }
 
-// grid (H, ceil(dv / 32)), block 128
+// grid (H, ceil(dv / 32)), block 128; dynamic shared memory: GLA's W2 rows of the head, bf16 [dk][rank]
 template <int R>
 __device__ __forceinline__ void da_step_body(const lb_decay_params2& p) {
-    __shared__ float q_s[4 * R], k_s[4 * R], a_s[4 * R];
+    extern __shared__ __align__(16) uint16_t a2_s[];
+    __shared__ __align__(16) float q_s[4 * R], k_s[4 * R], a_s[4 * R], a1_s[256];
     const int h = blockIdx.x, t = threadIdx.x, q4 = t & 3, j = blockIdx.y * DA_COLS + (t >> 2);
-    const bool live = j < p.dv;
+    const bool live = j < p.dv, gla = p.kind == LB_DA_GLA;
     float* S = p.state + ((size_t)h * p.dk + (size_t)q4 * R) * p.dv + j;
     const int rows = min(R, p.dk - q4 * R);
+    // constants, and the state (written a whole step ago), need no wait
     float s[R];
 #pragma unroll
-    for (int r = 0; r < R; ++r) s[r] = live && r < rows ? S[(size_t)r * p.dv] : 0.f; // written a whole step ago: needs no wait
+    for (int r = 0; r < R; ++r) s[r] = live && r < rows ? S[(size_t)r * p.dv] : 0.f;
+    if (gla)
+        for (int i = t; i < p.dk * p.rank; i += DA_THREADS) a2_s[i] = __ldg(p.a2 + (size_t)h * p.dk * p.rank + i);
     pdl_wait();
+    const float v = live ? p.proj[p.v_off + (size_t)h * p.dv + j] : 0.f;
+    if (gla) {
+        for (int i = t; i < p.rank; i += DA_THREADS) a1_s[i] = p.proj[p.a1_off + i];
+        __syncthreads();
+    }
     for (int i = t; i < 4 * R; i += DA_THREADS) {
         float q = 0.f, k = 0.f, a = 0.f;
-        if (i < p.dk) {
-            const int ch = h * p.dk + i;
-            const float z2 = p.kind == LB_DA_GLA ? da_dot_rank(p.a2 + (size_t)ch * p.rank, p.proj + p.a1_off, p.rank) : 0.f;
-            da_channel(p, p.proj, ch, z2, q, k, a);
-        }
+        if (i < p.dk) da_channel(p, p.proj, h * p.dk + i, gla ? da_dot_rank(a2_s + i * p.rank, a1_s, p.rank) : 0.f, q, k, a);
         q_s[i] = q;
         k_s[i] = k;
         a_s[i] = a;
     }
-    const float v = live ? p.proj[p.v_off + (size_t)h * p.dv + j] : 0.f;
     __syncthreads();
     pdl_launch_dependents();
+    const float4 *qv = reinterpret_cast<const float4*>(q_s + q4 * R), *kv = reinterpret_cast<const float4*>(k_s + q4 * R), *av = reinterpret_cast<const float4*>(a_s + q4 * R);
     float o0 = 0.f, o1 = 0.f;
 #pragma unroll
-    for (int r = 0; r < R; r += 2) {
-        s[r] = fmaf(a_s[q4 * R + r], s[r], k_s[q4 * R + r] * v);
-        s[r + 1] = fmaf(a_s[q4 * R + r + 1], s[r + 1], k_s[q4 * R + r + 1] * v);
-        o0 = fmaf(s[r], q_s[q4 * R + r], o0);
-        o1 = fmaf(s[r + 1], q_s[q4 * R + r + 1], o1);
+    for (int c = 0; c < R / 4; ++c) {
+        const float4 q = qv[c], k = kv[c], a = av[c];
+        s[4 * c] = fmaf(a.x, s[4 * c], k.x * v);
+        s[4 * c + 1] = fmaf(a.y, s[4 * c + 1], k.y * v);
+        s[4 * c + 2] = fmaf(a.z, s[4 * c + 2], k.z * v);
+        s[4 * c + 3] = fmaf(a.w, s[4 * c + 3], k.w * v);
+        o0 = fmaf(s[4 * c], q.x, o0);
+        o1 = fmaf(s[4 * c + 1], q.y, o1);
+        o0 = fmaf(s[4 * c + 2], q.z, o0);
+        o1 = fmaf(s[4 * c + 3], q.w, o1);
     }
 #pragma unroll
     for (int r = 0; r < R; ++r)

@@ -228,24 +228,59 @@ extern "C" __global__ void __launch_bounds__(256) gemm_f32_simt(const __grid_con
     }
 }
 
-// h_i[t] = x[t] / sqrt(mean x^2 + eps) * (1 + w_i), columns width..ld are zero.  grid T, block 256
+// h_i[t] = x[t] / sqrt(mean x^2 + eps) * (1 + w_i), columns width..ld are zero.  grid T, block 256.  Rows of whole quads up to
+// 4 NR_Q x 256 columns stay in registers between the two passes.
+#define NR_Q 8
 extern "C" __global__ void __launch_bounds__(256) norm_rows2(const __grid_constant__ lb_norm2_params p) {
     __shared__ float red[40];
+    const int t = threadIdx.x;
+    const bool quads = (p.width & 3) == 0 && p.width <= 4 * NR_Q * 256;
     pdl_wait();
     const float* x = p.x + (size_t)blockIdx.x * p.width;
+    const size_t o = (size_t)blockIdx.x * p.ld;
+    float4 v[NR_Q];
     float ss = 0.f;
+    if (quads) {
+#pragma unroll
+        for (int u = 0; u < NR_Q; ++u) {
+            const int i = 4 * (t + 256 * u);
+            v[u] = i < p.width ? *reinterpret_cast<const float4*>(x + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int u = 0; u < NR_Q; ++u) ss += (v[u].x * v[u].x + v[u].y * v[u].y) + (v[u].z * v[u].z + v[u].w * v[u].w);
+    } else {
 #pragma unroll 4
-    for (int i = threadIdx.x; i < p.width; i += 256) ss += x[i] * x[i];
+        for (int i = t; i < p.width; i += 256) ss += x[i] * x[i];
+    }
     ss = block_sum(ss, red);
     const float rinv = 1.0f / sqrtf(ss / (float)p.width + p.eps);
     pdl_launch_dependents();
-    const size_t o = (size_t)blockIdx.x * p.ld;
-    for (int i = threadIdx.x; i < p.ld; i += 256) {
-        const float v = i < p.width ? x[i] * rinv : 0.f;
+    if (quads) {
+#pragma unroll
+        for (int u = 0; u < NR_Q; ++u) {
+            const int i = 4 * (t + 256 * u);
+            if (i >= p.width) continue;
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                if (!p.h[e]) continue;
+                const uint2 w = __ldg(reinterpret_cast<const uint2*>(p.w[e] + i));
+                const float a = v[u].x * rinv * (1.0f + __uint_as_float(w.x << 16)), b = v[u].y * rinv * (1.0f + __uint_as_float(w.x & 0xffff0000u)),
+                            c = v[u].z * rinv * (1.0f + __uint_as_float(w.y << 16)), d = v[u].w * rinv * (1.0f + __uint_as_float(w.y & 0xffff0000u));
+                if (p.f32) *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.h[e]) + o + i) = make_float4(a, b, c, d);
+                else {
+                    const __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
+                    *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(p.h[e]) + o + i) =
+                        make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+                }
+            }
+        }
+    }
+    for (int i = quads ? p.width + t : t; i < p.ld; i += 256) {
+        const float xv = i < p.width ? x[i] * rinv : 0.f;
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
             if (!p.h[e]) continue;
-            const float r = i < p.width ? v * (1.0f + bf16_bits_to_f32(p.w[e][i])) : 0.f;
+            const float r = i < p.width ? xv * (1.0f + bf16_bits_to_f32(p.w[e][i])) : 0.f;
             if (p.f32) reinterpret_cast<float*>(p.h[e])[o + i] = r;
             else reinterpret_cast<__nv_bfloat16*>(p.h[e])[o + i] = __float2bfloat16_rn(r);
         }

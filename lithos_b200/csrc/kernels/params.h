@@ -294,6 +294,7 @@ typedef struct {
     int32_t stages;         /* ring stages per warp */
     int32_t split;          /* pieces a row pair is cut into along K: 1, or one per stage segment */
     int32_t segs;           /* ceil(K / LB_RG_SEG) */
+    int32_t x_cols;         /* columns of a vector one CTA holds: K, or the longer half where two CTAs share a row */
     float eps, mult, cap;
 } lb_rows_gemv_params;
 
@@ -327,6 +328,7 @@ typedef struct {
 
 /* ---- attention over the current block of positions, general head sizes (window_attention.cu) ---------------- */
 #define LB_WA_MAX_DIM 256
+#define LB_WA_MAX_SPLITS 64 /* position slices of a decode step */
 typedef struct {
     const float* proj;   /* fp32 [T, ld]: q | k | v sections at the given offsets */
     void* k_cache;       /* bf16 (or fp32) [max_ctx, KV, dim_p]: rotated keys; padding columns are zero */

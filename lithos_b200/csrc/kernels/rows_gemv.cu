@@ -6,25 +6,41 @@
 // HBM-bound: one CTA per SM, every warp streams its own row segments with 1-D bulk copies through its own ring, so what is in flight
 // (ring bytes x 148) does not depend on registers.  Two rows share every read of the vector: shared memory moves 2 bytes of weights in,
 // 2 out and 2 bytes of vector per weight.  Narrow launches (few pairs per CTA, long rows) cut a pair into segments, one per warp turn;
-// the segments of a pair are added in order, so a result does not depend on the schedule.
+// the segments of a pair are added in order, so a result does not depend on the schedule.  Where the vector is so long that it would leave
+// the ring too shallow, two CTAs (a cluster) take half of K each: half the vector to gather and to hold, and the sums of the two halves are
+// added, in order, through distributed shared memory.
 #include "common.cuh"
 #include "params.h"
 
+__device__ __forceinline__ void rg_cluster_sync() {
+    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+__device__ __forceinline__ float2 rg_ld_cluster(const float* local_ptr, uint32_t rank) {
+    uint32_t remote;
+    float2 v;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(smem_u32(local_ptr)), "r"(rank));
+    asm volatile("ld.shared::cluster.v2.f32 {%0, %1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(remote) : "memory");
+    return v;
+}
 __device__ __forceinline__ float rg_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const __grid_constant__ lb_rows_gemv_params p) {
     extern __shared__ __align__(16) unsigned char rg_sm[];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int G = gridDim.x, c = blockIdx.x, S = p.stages;
+    // gridDim.y = 2 (a cluster along y): this CTA's half of the row segments, columns k_lo .. k_hi - 1
+    const int KS = gridDim.y, rank = blockIdx.y, seg_lo = rank * p.segs / KS, my_segs = (rank + 1) * p.segs / KS - seg_lo;
+    const int k_lo = seg_lo * LB_RG_SEG, k_hi = min(p.K, k_lo + my_segs * LB_RG_SEG);
+    const int split = p.split > 1 ? my_segs : 1, spp = p.split > 1 ? 1 : my_segs; // pieces of a row pair, segments of a piece
     const int pairs0 = (p.mat[0].rows + 1) >> 1, pairs1 = p.n_mat > 1 ? (p.mat[1].rows + 1) >> 1 : 0, P = pairs0 + pairs1;
     const int my_pairs = P > c ? (P - c + G - 1) / G : 0;
     const int n_vec = p.x_mode == LB_RG_X_NORM ? p.n_mat : 1;
     unsigned char* ring = rg_sm;                                                              // [warps][S][2][SEG] bf16
-    float* xsm = reinterpret_cast<float*>(ring + (size_t)LB_RG_WARPS * S * LB_RG_SEG * 4);     // [n_vec][K]
-    float* gate_s = xsm + (size_t)n_vec * p.K;                                                 // [n_mix] when there is a gate
+    float* xsm = reinterpret_cast<float*>(ring + (size_t)LB_RG_WARPS * S * LB_RG_SEG * 4);     // [n_vec][K] (its half)
+    float* gate_s = xsm + (size_t)n_vec * p.x_cols;                                                // [n_mix] when there is a gate
     float* part = gate_s + (p.gate ? (p.n_mix + 3) & ~3 : 0);                                  // [my_pairs * split][2]
     const int max_pairs = (P + G - 1) / G;
-    float* red = part + (size_t)2 * max_pairs * p.split;                                       // [40]
+    float* red = part + (size_t)2 * max_pairs * p.split;                                      // [40]
     uint64_t* bars = reinterpret_cast<uint64_t*>(red + 40);                                    // [warps][S], the vector's
     if (lane == 0)
         for (int s = 0; s < S; ++s) mbar_init(&bars[warp * S + s], 1);
@@ -33,7 +49,7 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
     __syncthreads();
 
     // the warp's stages: items warp, warp + 8, ... (item = pair * split + piece), segments of the item in order
-    const int items = my_pairs * p.split, spp = p.segs / p.split;
+    const int items = my_pairs * split;
     const uint64_t pol = l2_policy_evict_first();
     auto row_ptr = [&](int pair, int& mi) -> const uint16_t* {
         const int g = c + pair * G;
@@ -44,7 +60,7 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
     auto request = [&]() {
         if (r_item >= items) return;
         if (lane == 0) {
-            const int pair = r_item / p.split, seg = (r_item - pair * p.split) * spp + r_seg;
+            const int pair = split == 1 ? r_item : r_item / split, seg = seg_lo + (r_item - pair * split) * spp + r_seg;
             int mi;
             const uint16_t* w = row_ptr(pair, mi) + (size_t)seg * LB_RG_SEG;
             const uint32_t bytes = (uint32_t)min(LB_RG_SEG, p.K - seg * LB_RG_SEG) * 2u;
@@ -122,24 +138,27 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
             }
         }
     } else {
-        const int m4 = p.n_mix & ~3, a4 = p.n_act & ~3, g4 = p.gate && (reinterpret_cast<size_t>(p.gate) & 15) == 0 ? m4 : 0;
+        const int n_mix = rank == 0 ? p.n_mix : 0; // the whole mixer part lies in the first half
+        const int a_lo = max(0, k_lo - p.n_mix_pad), a_hi = min(p.n_act, max(0, k_hi - p.n_mix_pad)), n_act = max(0, a_hi - a_lo);
+        float* xa = xsm + (p.n_mix_pad + a_lo - k_lo);
+        const int m4 = n_mix & ~3, a4 = n_act & ~3, g4 = p.gate && (reinterpret_cast<size_t>(p.gate) & 15) == 0 ? m4 : 0;
         if (tid == 0) {
             mbar_arrive_expect_tx(xbar, (uint32_t)(m4 + a4 + g4) * 4u);
             if (m4) bulk_g2s_plain(xsm, p.mix, (uint32_t)m4 * 4u, xbar);
             if (g4) bulk_g2s_plain(gate_s, p.gate, (uint32_t)g4 * 4u, xbar);
-            if (a4) bulk_g2s_plain(xsm + p.n_mix_pad, p.act, (uint32_t)a4 * 4u, xbar);
+            if (a4) bulk_g2s_plain(xa, p.act + a_lo, (uint32_t)a4 * 4u, xbar);
         }
-        for (int i = m4 + tid; i < p.n_mix; i += LB_RG_THREADS) xsm[i] = p.mix[i];
+        for (int i = m4 + tid; i < n_mix; i += LB_RG_THREADS) xsm[i] = p.mix[i];
         if (p.gate)
-            for (int i = g4 + tid; i < p.n_mix; i += LB_RG_THREADS) gate_s[i] = p.gate[i];
-        for (int i = a4 + tid; i < p.n_act; i += LB_RG_THREADS) xsm[p.n_mix_pad + i] = p.act[i];
-        for (int i = p.n_mix_pad + p.n_act + tid; i < p.K; i += LB_RG_THREADS) xsm[i] = 0.f;
-        for (int i = p.n_mix + tid; i < p.n_mix_pad; i += LB_RG_THREADS) xsm[i] = 0.f;
+            for (int i = g4 + tid; i < n_mix; i += LB_RG_THREADS) gate_s[i] = p.gate[i];
+        for (int i = a4 + tid; i < n_act; i += LB_RG_THREADS) xa[i] = p.act[a_lo + i];
+        for (int i = max(p.n_mix_pad + p.n_act, k_lo) + tid; i < k_hi; i += LB_RG_THREADS) xsm[i - k_lo] = 0.f;
+        for (int i = n_mix + tid; rank == 0 && i < p.n_mix_pad; i += LB_RG_THREADS) xsm[i] = 0.f;
         const bool here = mbar_wait(xbar, 0);
         if (!here && p.status) atomicExch(p.status, LB_DEV_TIMEOUT_FULL);
         __syncthreads();
         if (p.head_w) {
-            const int heads = p.n_mix / p.vdim;
+            const int heads = n_mix / p.vdim;
             for (int h = warp; h < heads; h += LB_RG_WARPS) {
                 float* o = xsm + (size_t)h * p.vdim;
                 float ss = 0.f;
@@ -163,8 +182,8 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
     uint32_t phase = 0;
     bool ok = true;
     for (int item = warp; item < items && ok; item += LB_RG_WARPS) {
-        const int pair = item / p.split, seg0 = (item - pair * p.split) * spp;
-        const float* xv = xsm + ((n_vec > 1 && c + pair * G >= pairs0) ? p.K : 0);
+        const int pair = split == 1 ? item : item / split, seg0 = seg_lo + (item - pair * split) * spp;
+        const float* xv = xsm + ((n_vec > 1 && c + pair * G >= pairs0) ? p.K : 0) - k_lo;
         float a0 = 0.f, a1 = 0.f, b0 = 0.f, b1 = 0.f;
         for (int s = 0; s < spp; ++s) {
             if (!__all_sync(0xffffffffu, mbar_wait(&bars[warp * S + slot], phase))) { // bounded: the rows left keep their old result
@@ -203,15 +222,37 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
         const float ya = warp_sum(a0 + a1), yb = warp_sum(b0 + b1);
         if (lane == 0) { part[2 * item] = ya; part[2 * item + 1] = yb; }
     }
-    const bool all_ok = __syncthreads_and(ok ? 1 : 0) != 0;
+    bool all_ok = __syncthreads_and(ok ? 1 : 0) != 0;
+    if (KS > 1) { // this half's sums where the other CTA finds them
+        for (int m = tid; m < my_pairs; m += LB_RG_THREADS) {
+            float2 r = make_float2(0.f, 0.f);
+            for (int q = 0; q < split; ++q) {
+                r.x += part[2 * (m * split + q)];
+                r.y += part[2 * (m * split + q) + 1];
+            }
+            *reinterpret_cast<float2*>(part + 2 * m * split) = r; // read and written by this thread alone
+        }
+        if (tid == 0) red[36] = all_ok ? 1.f : 0.f;
+        if (tid == 0) red[37] = (float)split;
+        rg_cluster_sync();
+        all_ok = rg_ld_cluster(red + 36, rank ^ 1).x != 0.f && all_ok;
+    }
+    const int other_split = KS > 1 ? (int)rg_ld_cluster(red + 36, rank ^ 1).y : 0;
 
     float best_v = -INFINITY;
     int best_i = 0x7fffffff;
     for (int m = tid; m < my_pairs && all_ok; m += LB_RG_THREADS) {
         float r[2] = {0.f, 0.f};
-        for (int q = 0; q < p.split; ++q) {
-            r[0] += part[2 * (m * p.split + q)];
-            r[1] += part[2 * (m * p.split + q) + 1];
+        if (KS > 1) {
+            if ((m & 1) != rank) continue; // the two CTAs finish every other pair each
+            const float2 mine = *reinterpret_cast<const float2*>(part + 2 * m * split), his = rg_ld_cluster(part + 2 * m * other_split, rank ^ 1);
+            r[0] = rank == 0 ? mine.x + his.x : his.x + mine.x;
+            r[1] = rank == 0 ? mine.y + his.y : his.y + mine.y;
+        } else {
+            for (int q = 0; q < split; ++q) {
+                r[0] += part[2 * (m * split + q)];
+                r[1] += part[2 * (m * split + q) + 1];
+            }
         }
         const int g = c + m * G, mi = g >= pairs0, n = 2 * (mi ? g - pairs0 : g);
         const lb_rg_mat& M = p.mat[mi];
@@ -246,4 +287,5 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
             p.part_idx[c] = best_i;
         }
     }
+    if (KS > 1) rg_cluster_sync(); // nobody leaves while the other CTA still reads its sums
 }

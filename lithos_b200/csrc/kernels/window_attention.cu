@@ -36,6 +36,9 @@ template <> struct wa_t<float> {
     static __device__ __forceinline__ float from(float v) { return v; }
 };
 
+__device__ __forceinline__ void wa_cp16(uint32_t dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
 struct wa_angles { // cosines and sines of a position: key / query pairs and value pairs
     float ck[LB_WA_MAX_DIM / 2], sk[LB_WA_MAX_DIM / 2], cv[LB_WA_MAX_DIM / 2], sv[LB_WA_MAX_DIM / 2];
 };
@@ -73,49 +76,76 @@ __device__ __forceinline__ void wa_warp_value(const lb_wattn_params& p, const fl
     wa_warp_rotate(src, dst, p.vdim, p.freq_v ? p.vdim : 0, A.cv, A.sv, r);
 }
 
-#define WR_WARPS 8
-// grid (KV * groups, splits, tokens), block 256; GH query heads per CTA, NV pairs of value features per lane (64 NV >= vdim).
-// dynamic shared memory: q [GH][dim_p] fp32 | accumulators [8][GH][vdim_p] fp32 | new key, value row in the cache's format
+#define WR_MAX_WARPS 4
+// grid (KV * groups, splits, tokens), block 32 x warps (1..4); GH query heads per CTA, NV pairs of value features per lane (64 NV >= vdim).
+// A warp takes tiles of 32 cache rows: the tile's K and V rows come to shared memory in one go, a lane scores one row for all heads of the
+// CTA (no exchange between lanes), then lanes own value features.  In the decode step everything that does not depend on this step's
+// projections -- position, angles, the first tile (rows of earlier positions, written by kernels that have long finished) -- is under way
+// before the wait for the previous kernel.
+// dynamic shared memory: q [GH][dim_p] fp32 | accumulators [warps][GH][vdim_p] fp32 | new key, value row in the cache's format |
+// tiles [warps][32][K row + 16 B, V row + 16 B]
 template <typename TC, int GH, int NV>
 __device__ __forceinline__ void wattn_rows_body(const lb_wattn_params& p) {
     extern __shared__ __align__(16) unsigned char wr_sm[];
     __shared__ wa_angles A;
-    __shared__ float pw[WR_WARPS][32][GH];
-    __shared__ float ml[WR_WARPS][GH][2];
+    __shared__ __align__(16) float pw[WR_MAX_WARPS][32][GH];
+    __shared__ float ml[WR_MAX_WARPS][GH][2];
+    __shared__ float fw[LB_WA_MAX_SPLITS][GH]; // weight of each slice (or warp) in the merged sum, denominators divided in
     __shared__ int last_flag;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nw = blockDim.x >> 5;
     const int G = p.H / p.KV, groups = (G + GH - 1) / GH;
     const int kv = blockIdx.x / groups, hg = blockIdx.x - kv * groups, h0 = kv * G + hg * GH, nh = min(GH, G - hg * GH);
     float* q_s = reinterpret_cast<float*>(wr_sm);
     float* acc_s = q_s + GH * p.dim_p;
-    TC* kn = reinterpret_cast<TC*>(acc_s + WR_WARPS * GH * p.vdim_p);
+    TC* kn = reinterpret_cast<TC*>(acc_s + nw * GH * p.vdim_p);
     TC* vn = kn + p.dim_p;
-    pdl_wait();
+    const int ks_t = p.dim_p + 16 / (int)sizeof(TC), vs_t = p.vdim_p + 16 / (int)sizeof(TC); // tile row strides: 16 bytes of padding
+    TC* kt = vn + p.vdim_p + (size_t)warp * 32 * (ks_t + vs_t);
+    TC* vt = kt + 32 * ks_t;
+    const bool early = p.pos_ptr != nullptr; // decode step
+    if (!early) pdl_wait();
     const int s = blockIdx.z, pos = (p.pos_ptr ? p.pos_ptr[0] : p.pos0) + s;
     if (pos < 0 || pos >= p.max_ctx) { // refused before anything is read or written (the same for every CTA)
         if (tid == 0 && p.status) atomicExch(p.status, LB_DEV_POS_RANGE);
+        if (early) pdl_wait();
         return;
     }
     const float* row = p.proj + (size_t)s * p.ld;
     const int w0 = p.block > 0 ? pos / p.block * p.block : 0, n = pos - w0 + 1;
-    const int per = ((n + p.splits - 1) / p.splits + 31) & ~31;
-    const int r0 = w0 + blockIdx.y * per, r1 = min(r0 + per, pos + 1); // this CTA's rows (none when r0 >= r1)
+    const int per = ((n + p.splits - 1) / p.splits + 31) & ~31, used = (n + per - 1) / per; // rows per slice; slices that have rows
+    if ((int)blockIdx.y >= used) return;
+    const int r0 = w0 + blockIdx.y * per, r1 = min(r0 + per, pos + 1); // this CTA's rows
     const bool own = p.k_off >= 0; // the newest row is made here
+    TC* kc = reinterpret_cast<TC*>(p.k_cache) + (size_t)kv * p.dim_p;
+    TC* vc = reinterpret_cast<TC*>(p.v_cache) + (size_t)kv * p.vdim_p;
+    const size_t ks = (size_t)p.KV * p.dim_p, vs = (size_t)p.KV * p.vdim_p;
+    auto stage = [&](int b) { // rows b .. b + 31 (those past the slice repeat its last one; the newest row's place is not used)
+        constexpr int E = 16 / (int)sizeof(TC);
+        const int kq = p.dim_p / E, vq = p.vdim_p / E;
+        for (int i = lane; i < 32 * kq; i += 32) {
+            const int r = i / kq, c = i - r * kq;
+            wa_cp16(smem_u32(kt + r * ks_t + c * E), kc + (size_t)min(b + r, r1 - 1) * ks + c * E);
+        }
+        for (int i = lane; i < 32 * vq; i += 32) {
+            const int r = i / vq, c = i - r * vq;
+            wa_cp16(smem_u32(vt + r * vs_t + c * E), vc + (size_t)min(b + r, r1 - 1) * vs + c * E);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    if (r0 + warp * 32 < r1) stage(r0 + warp * 32);
     wa_fill_angles(p, pos, A);
     __syncthreads();
-    for (int g = warp; g < GH; g += WR_WARPS) {
+    if (early) pdl_wait();
+    for (int g = warp; g < GH; g += nw) {
         float* dst = q_s + g * p.dim_p;
         if (g < nh) wa_warp_rotate(row + p.q_off + (size_t)(h0 + g) * p.dim, dst, p.dim, p.rot_dims, A.ck, A.sk, p.scale);
         for (int i = lane; i < p.dim_p; i += 32)
             if (g >= nh || i >= p.dim) dst[i] = 0.f;
     }
-    TC* kc = reinterpret_cast<TC*>(p.k_cache) + (size_t)kv * p.dim_p;
-    TC* vc = reinterpret_cast<TC*>(p.v_cache) + (size_t)kv * p.vdim_p;
-    const size_t ks = (size_t)p.KV * p.dim_p, vs = (size_t)p.KV * p.vdim_p;
-    const bool has_new = own && r0 <= pos && pos < r1;
+    const bool has_new = own && pos < r1;
     if (has_new) {
-        if (warp == WR_WARPS - 1) wa_warp_rotate(row + p.k_off + (size_t)kv * p.dim, kn, p.dim, p.rot_dims, A.ck, A.sk, 1.f);
-        if (warp == WR_WARPS - 2) wa_warp_value(p, row + p.v_off + (size_t)kv * p.vdim, vn, A);
+        if (warp == nw - 1) wa_warp_rotate(row + p.k_off + (size_t)kv * p.dim, kn, p.dim, p.rot_dims, A.ck, A.sk, 1.f);
+        if (warp == (nw > 1 ? nw - 2 : 0)) wa_warp_value(p, row + p.v_off + (size_t)kv * p.vdim, vn, A);
         for (int i = tid; i < p.dim_p; i += blockDim.x)
             if (i >= p.dim) kn[i] = wa_t<TC>::from(0.f);
         for (int i = tid; i < p.vdim_p; i += blockDim.x)
@@ -136,9 +166,11 @@ __device__ __forceinline__ void wattn_rows_body(const lb_wattn_params& p) {
 #pragma unroll
         for (int i = 0; i < 2 * NV; ++i) acc[g][i] = 0.f;
     }
-    for (int b = r0 + warp * 32; b < r1; b += WR_WARPS * 32) {
-        const int r = min(b + lane, r1 - 1);
-        const TC* kr = own && r == pos ? kn : kc + (size_t)r * ks;
+    for (int b = r0 + warp * 32; b < r1; b += nw * 32) {
+        if (b != r0 + warp * 32) stage(b);
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncwarp();
+        const TC* kr = own && b + lane == pos ? kn : kt + lane * ks_t;
         float sc[GH];
 #pragma unroll
         for (int g = 0; g < GH; ++g) sc[g] = 0.f;
@@ -160,22 +192,33 @@ __device__ __forceinline__ void wattn_rows_body(const lb_wattn_params& p) {
             }
         }
         const int cnt = min(32, r1 - b);
+        float mx[GH], ps[GH];
+#pragma unroll
+        for (int g = 0; g < GH; ++g) mx[g] = lane < cnt ? sc[g] : -INFINITY;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+            for (int g = 0; g < GH; ++g) mx[g] = fmaxf(mx[g], __shfl_xor_sync(0xffffffffu, mx[g], o));
 #pragma unroll
         for (int g = 0; g < GH; ++g) {
-            float v = lane < cnt ? sc[g] : -INFINITY, mx = v;
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-            const float mn = fmaxf(m[g], mx), corr = expf(m[g] - mn), e = expf(v - mn);
-            l[g] = fmaf(l[g], corr, warp_sum(e));
+            const float mn = fmaxf(m[g], mx[g]), corr = expf(m[g] - mn), e = lane < cnt ? expf(sc[g] - mn) : 0.f;
             m[g] = mn;
+            l[g] *= corr;
+            ps[g] = e;
             pw[warp][lane][g] = e;
 #pragma unroll
             for (int i = 0; i < 2 * NV; ++i) acc[g][i] *= corr;
         }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+            for (int g = 0; g < GH; ++g) ps[g] += __shfl_xor_sync(0xffffffffu, ps[g], o);
+#pragma unroll
+        for (int g = 0; g < GH; ++g) l[g] += ps[g];
         __syncwarp();
 #pragma unroll 4
         for (int j = 0; j < cnt; ++j) {
-            const TC* vr = own && b + j == pos ? vn : vc + (size_t)(b + j) * vs;
+            const TC* vr = own && b + j == pos ? vn : vt + j * vs_t;
             float2 vv[NV];
 #pragma unroll
             for (int i = 0; i < NV; ++i) {
@@ -207,13 +250,13 @@ __device__ __forceinline__ void wattn_rows_body(const lb_wattn_params& p) {
     __syncthreads();
     const int rec = p.vdim_p + 2;
     float* scr = p.scratch + ((size_t)blockIdx.x * p.splits) * GH * rec;
-    if (p.splits > 1) {
+    if (used > 1) {
         float* mine = scr + (size_t)blockIdx.y * GH * rec;
         for (int i = tid; i < nh * p.vdim_p; i += blockDim.x) {
             const int g = i / p.vdim_p, d = i - g * p.vdim_p;
             float M = -1e30f, a = 0.f, L = 0.f;
-            for (int w = 0; w < WR_WARPS; ++w) M = fmaxf(M, ml[w][g][0]);
-            for (int w = 0; w < WR_WARPS; ++w) {
+            for (int w = 0; w < nw; ++w) M = fmaxf(M, ml[w][g][0]);
+            for (int w = 0; w < nw; ++w) {
                 const float f = expf(ml[w][g][0] - M);
                 a = fmaf(f, acc_s[(w * GH + g) * p.vdim_p + d], a);
                 L = fmaf(f, ml[w][g][1], L);
@@ -225,42 +268,47 @@ __device__ __forceinline__ void wattn_rows_body(const lb_wattn_params& p) {
         __syncthreads();
         if (tid == 0) {
             const uint32_t old = atomicAdd(p.counters + blockIdx.x, 1u);
-            last_flag = old == (uint32_t)p.splits - 1u;
+            last_flag = old == (uint32_t)used - 1u;
             if (last_flag) p.counters[blockIdx.x] = 0u; // everybody has arrived: ready for the next launch
         }
         __syncthreads();
         if (!last_flag) return;
         __threadfence();
     }
-    // the whole sum of each head (slices in order), the sink, back-rotation by this position
-    const float M0 = p.sink ? 0.f : -1e30f;
+    // the whole sum of each head (slices in order, or the warps of the only one), the sink, back-rotation by this position
+    const int parts = used > 1 ? used : nw;
+    if (tid < nh) {
+        const int g = tid;
+        float M = p.sink ? 0.f : -1e30f;
+#pragma unroll 4
+        for (int q = 0; q < parts; ++q) M = fmaxf(M, used > 1 ? __ldcg(scr + ((size_t)q * GH + g) * rec + p.vdim_p) : ml[q][g][0]);
+        float L = p.sink ? expf(-M) : 0.f;
+#pragma unroll 4
+        for (int q = 0; q < parts; ++q) {
+            const float f = expf((used > 1 ? __ldcg(scr + ((size_t)q * GH + g) * rec + p.vdim_p) : ml[q][g][0]) - M);
+            L = fmaf(f, used > 1 ? __ldcg(scr + ((size_t)q * GH + g) * rec + p.vdim_p + 1) : ml[q][g][1], L);
+            fw[q][g] = f;
+        }
+        for (int q = 0; q < parts; ++q) fw[q][g] /= L;
+    }
+    __syncthreads();
     for (int i = tid; i < nh * (p.vdim_p / 2); i += blockDim.x) {
         const int g = i / (p.vdim_p / 2), d = 2 * (i - g * (p.vdim_p / 2));
         if (d >= p.vdim) continue;
-        float M = M0, L, u = 0.f, v = 0.f;
-        if (p.splits > 1) {
-            for (int q = 0; q < p.splits; ++q) M = fmaxf(M, __ldcg(scr + ((size_t)q * GH + g) * rec + p.vdim_p));
-            L = p.sink ? expf(-M) : 0.f;
-            for (int q = 0; q < p.splits; ++q) {
-                const float* R = scr + ((size_t)q * GH + g) * rec;
-                const float f = expf(__ldcg(R + p.vdim_p) - M);
-                L = fmaf(f, __ldcg(R + p.vdim_p + 1), L);
-                u = fmaf(f, __ldcg(R + d), u);
-                v = fmaf(f, __ldcg(R + d + 1), v);
+        float u = 0.f, v = 0.f;
+        if (used > 1) {
+#pragma unroll 8
+            for (int q = 0; q < parts; ++q) {
+                const float2 x = __ldcg(reinterpret_cast<const float2*>(scr + ((size_t)q * GH + g) * rec + d));
+                u = fmaf(fw[q][g], x.x, u);
+                v = fmaf(fw[q][g], x.y, v);
             }
         } else {
-            for (int w = 0; w < WR_WARPS; ++w) M = fmaxf(M, ml[w][g][0]);
-            L = p.sink ? expf(-M) : 0.f;
-            for (int w = 0; w < WR_WARPS; ++w) {
-                const float f = expf(ml[w][g][0] - M);
-                L = fmaf(f, ml[w][g][1], L);
-                u = fmaf(f, acc_s[(w * GH + g) * p.vdim_p + d], u);
-                v = fmaf(f, acc_s[(w * GH + g) * p.vdim_p + d + 1], v);
+            for (int q = 0; q < parts; ++q) {
+                u = fmaf(fw[q][g], acc_s[(q * GH + g) * p.vdim_p + d], u);
+                v = fmaf(fw[q][g], acc_s[(q * GH + g) * p.vdim_p + d + 1], v);
             }
         }
-        const float inv = 1.0f / L;
-        u *= inv;
-        v *= inv;
         if (p.freq_v) {
             const float c = A.cv[d / 2], sn = A.sv[d / 2], a = u * c + v * sn;
             v = v * c - u * sn;
@@ -278,7 +326,7 @@ __device__ __forceinline__ void wattn_rows_body(const lb_wattn_params& p) {
     }
 }
 #define WR_KERNEL(name, TC, GH, NV)                                                                                      \
-    extern "C" __global__ void __launch_bounds__(WR_WARPS * 32) name(const __grid_constant__ lb_wattn_params p) {        \
+    extern "C" __global__ void __launch_bounds__(WR_MAX_WARPS * 32) name(const __grid_constant__ lb_wattn_params p) {        \
         wattn_rows_body<TC, GH, NV>(p);                                                                                  \
     }
 WR_KERNEL(wattn_rows_b2n2, __nv_bfloat16, 2, 2)
@@ -339,9 +387,6 @@ __device__ __forceinline__ void wa_ldsm(uint32_t addr, uint32_t& r0, uint32_t& r
 }
 __device__ __forceinline__ void wa_ldsm_t(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void wa_cp16(uint32_t dst, const void* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
 }
 __device__ __forceinline__ void wa_split(float x, float y, uint32_t& hi, uint32_t& lo) {
     const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
