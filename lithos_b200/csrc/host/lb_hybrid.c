@@ -29,6 +29,8 @@ extern unsigned lb_attn_mma_smem(int G);
 
 static int is_fa(const lb_model_cfg* c, int l) { return (l % c->fa_period) == c->fa_period - 1; }
 
+#define PF_CHUNK 256 /* tokens per prompt chunk: what one lb_gemm_int4 call takes */
+
 static const lb_arch k_hybrid;
 
 LB_API int lb_model_create(lb_ctx* c, const lb_model_cfg* cfg, int tp_rank, int tp_size, lb_model** out) {
@@ -45,7 +47,7 @@ LB_API int lb_model_create(lb_ctx* c, const lb_model_cfg* cfg, int tp_rank, int 
         return lb_fail(c, LB_ERR_INVALID, "model: heads / intermediate size / vocabulary do not split %d ways", tp_size);
     lb_model* m = (lb_model*)calloc(1, sizeof *m);
     if (!m) return LB_ERR_NOMEM;
-    m->c = c; m->arch = &k_hybrid; m->cfg = *cfg; m->tp_rank = tp_rank; m->tp_size = tp_size;
+    m->c = c; m->arch = &k_hybrid; m->pf_chunk = PF_CHUNK; m->cfg = *cfg; m->tp_rank = tp_rank; m->tp_size = tp_size;
     m->use_chain = 1;
     m->HV = cfg->dn_v_heads / tp_size; m->HK = cfg->dn_k_heads / tp_size; m->HQ = cfg->fa_q_heads / tp_size;
     m->HKV = cfg->fa_kv_heads >= tp_size ? cfg->fa_kv_heads / tp_size : 1; /* fewer KV heads than GPUs: replicated */
@@ -616,7 +618,6 @@ static void hybrid_destroy(lb_model* m) {
 }
 
 /* ---- a prompt chunk ---------------------------------------------------------------------- */
-#define PF_CHUNK 256
 static unsigned blocks_for(long long n) {
     long long b = (n + 255) / 256;
     return (unsigned)(b > 4096 ? 4096 : b < 1 ? 1 : b);
@@ -716,5 +717,5 @@ static void hybrid_pf_sizes(const lb_model* m, size_t bytes[LB_PF_MAX_BUFS]) {
     memcpy(bytes, b, sizeof b); /* in the order of pf_set.hy */
 }
 
-static const lb_arch k_hybrid = {"hybrid", PF_CHUNK, 4, hybrid_reset_state, hybrid_snapshot, hybrid_state_ptr, hybrid_step_layers, hybrid_head,
+static const lb_arch k_hybrid = {"hybrid", 4, hybrid_reset_state, hybrid_snapshot, hybrid_state_ptr, hybrid_step_layers, hybrid_head,
                                  hybrid_head_ctas, hybrid_head_rows, hybrid_pf_sizes, hybrid_pf_layer, hybrid_destroy};

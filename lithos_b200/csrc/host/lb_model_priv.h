@@ -45,14 +45,14 @@ typedef union {
  * streams of the prompt pass, sampling and the generation loop. */
 typedef struct lb_arch {
     const char* name;
-    int pf_chunk, pf_streams;                          /* prompt pass: tokens per chunk, chunks in flight (<= LB_PF_MAX_STREAMS) */
+    int pf_streams;                                     /* prompt pass: chunks in flight (<= LB_PF_MAX_STREAMS) */
     int (*reset_state)(lb_model* m);                    /* caches and recurrent states of the sequence back to empty (stream-ordered) */
     int (*snapshot)(lb_model* m, int restore);          /* checkpoint / rollback of the recurrent states */
     int (*state_ptr)(lb_model* m, int layer, int which, uint64_t* dptr, size_t* bytes);
     int (*step_layers)(lb_model* m);                    /* one token: m->X (its embedding) through every layer; position in m->d_pos */
     int (*head)(lb_model* m, CUdeviceptr x_row);        /* final norm + LM head of one row -> m->logits, arg-max candidates */
     int (*head_ctas)(lb_model* m);                      /* how many candidates head leaves */
-    int (*head_rows)(lb_model* m, CUdeviceptr rows, int n, CUdeviceptr logits); /* the same for n <= pf_chunk rows, no candidates */
+    int (*head_rows)(lb_model* m, CUdeviceptr rows, int n, CUdeviceptr logits); /* the same for n <= lb_model.pf_chunk rows, no candidates */
     void (*pf_sizes)(const lb_model* m, size_t bytes[LB_PF_MAX_BUFS]);          /* bytes of each buffer of a chunk (0 = unused) */
     int (*pf_layer)(lb_model* m, pf_set* w, int l, int pos0, int T);           /* one layer over a chunk; on c->stream */
     void (*destroy)(lb_model* m);
@@ -64,6 +64,7 @@ struct lb_model {
     const lb_arch* arch;
     void* impl;       /* lb_stack.c: its own description and weights */
     lb_model_cfg cfg; /* n_layers, hidden, vocab, max_ctx and eps hold for every architecture, the rest for the hybrid */
+    int pf_chunk;     /* prompt pass: tokens per chunk, set by the architecture */
     int tp_rank, tp_size;
     /* per-shard sizes */
     int HV, HK, HQ, HKV, inter_s; /* heads / intermediate columns on this shard */

@@ -1,4 +1,4 @@
-/* The prompt pass: runs n tokens through the model in chunks (lb_arch.pf_chunk tokens each) and leaves the state a
+/* The prompt pass: runs n tokens through the model in chunks (lb_model.pf_chunk tokens each) and leaves the state a
  * token-by-token decode of the same tokens leaves, then the sampled next token (lb_model_prefill) or the logits of chosen
  * tokens (lb_model_forward).  The layer order is that of compiler/megakernel-link.ls:281-525; what a layer does to a chunk is
  * the architecture's pf_layer: every projection is one matrix product per chunk (weights read once), recurrences walk the
@@ -101,7 +101,7 @@ static int run_chunks(lb_model* m, const int* tokens, int n, int pos0, const int
     lb_ctx* c = m->c;
     const lb_model_cfg* cfg = &m->cfg;
     lb_prefill_ws* ws = m->ws;
-    const int H = cfg->hidden, CH = m->arch->pf_chunk, NS = m->arch->pf_streams;
+    const int H = cfg->hidden, CH = m->pf_chunk, NS = m->arch->pf_streams;
     CUstream main_stream = c->stream;
     LB_CU(c, lb_drv.MemcpyHtoDAsync(ws->tokens, tokens, (size_t)n * 4, main_stream));
     LB_CU(c, lb_drv.StreamSynchronize(main_stream)); /* the caller's token array may be pageable */
@@ -184,8 +184,8 @@ LB_API int lb_model_forward(lb_model* m, const int* tokens, int n, int pos0, con
         LB_TRY(rows_reserve(m, n_want));
         lb_prefill_ws* ws = m->ws;
         LB_TRY(run_chunks(m, tokens, n, pos0, want, n_want, ws->rows));
-        for (int r = 0; r < n_want; r += m->arch->pf_chunk) {
-            const int k = n_want - r < m->arch->pf_chunk ? n_want - r : m->arch->pf_chunk;
+        for (int r = 0; r < n_want; r += m->pf_chunk) {
+            const int k = n_want - r < m->pf_chunk ? n_want - r : m->pf_chunk;
             LB_TRY(m->arch->head_rows(m, ws->rows + (size_t)r * m->cfg.hidden * 4, k, ws->row_logits + (size_t)r * m->cfg.vocab * 4));
         }
         src = ws->row_logits;

@@ -17,7 +17,7 @@
 #include "lb_stack.h"
 #include <math.h>
 
-#define ST_CHUNK 512
+#define ST_CHUNK 1024 /* largest chunk of a prompt; stack_chunk picks the model's */
 #define ST_STREAMS 4
 
 typedef struct {
@@ -292,6 +292,19 @@ static int launch_rows(lb_model* m, lb_rows_gemv_params* p) {
     return lb_launch_cluster(c, LBK_rows_gemv, (unsigned)(c->sm_count / ks), (unsigned)ks, 1, LB_RG_THREADS, (unsigned)smem, params, 1, (unsigned)ks);
 }
 
+/* Tokens per product tile, and what a product then costs in units of one wave of 256-token tiles: fewer tokens per tile make more tiles
+ * for narrow matrices, at a lower rate per tile (measured: the operands' trip through shared memory bounds small tiles). */
+static double product_cost(const lb_ctx* c, int row_tiles, int T, int* nt_out) {
+    static const struct { int nt; double cost; } k[] = {{256, 1.0}, {128, 0.55}, {64, 0.38}, {32, 0.34}, {16, 0.33}};
+    double best = 1e30;
+    for (int i = 0; i < 5; i++) {
+        const int tiles = row_tiles * ((T + k[i].nt - 1) / k[i].nt);
+        const double v = (double)((tiles + c->sm_count - 1) / c->sm_count) * k[i].cost;
+        if (v < best) { best = v; *nt_out = k[i].nt; }
+    }
+    return best;
+}
+
 /* one or two products Y = X W^T of a chunk (w[1] may be NULL) */
 typedef struct { const st_mat* w; CUdeviceptr x; CUdeviceptr y; int y_mode, ld_y; } st_prod;
 static int launch_products(lb_model* m, const st_prod* pr, int n, int T) {
@@ -302,13 +315,13 @@ static int launch_products(lb_model* m, const st_prod* pr, int n, int T) {
     p.T = T; p.K = pr[0].w->K; p.ld_x = p.K;
     p.mult = (float)S->d.residual_mult; p.cap = (float)S->d.logit_softcap;
     p.status = (uint32_t*)c->dev_status;
-    p.NT = T > 128 ? 256 : T > 64 ? 128 : T > 32 ? 64 : T > 16 ? 32 : 16;
-    p.t_tiles = (T + p.NT - 1) / p.NT;
     for (int i = 0; i < n; i++) {
         p.rows[i] = pr[i].w->rows; p.w[i] = (const uint16_t*)pr[i].w->w; p.x[i] = (const void*)pr[i].x;
         p.y[i] = (void*)pr[i].y; p.y_mode[i] = pr[i].y_mode; p.ld_y[i] = pr[i].ld_y; p.y_f32[i] = S->esz == 4;
         p.tiles[i] = (p.rows[i] + LB_DG_ROWS - 1) / LB_DG_ROWS;
     }
+    product_cost(c, p.tiles[0] + p.tiles[1], T, &p.NT);
+    p.t_tiles = (T + p.NT - 1) / p.NT;
     void* params[] = {&p};
     if (S->esz == 4)
         return lb_launch(c, LBK_gemm_f32_simt, (unsigned)((p.rows[0] + 63) / 64 + (p.rows[1] + 63) / 64), (unsigned)((T + 63) / 64), 1, 256, 0, params, 1);
@@ -421,8 +434,8 @@ static int stack_pf_layer(lb_model* m, pf_set* w, int i, int pos0, int T) {
         p.cat = (void*)w->st.cat; p.cat_ld = L->out.K; p.cat_f32 = f32;
         void* params[] = {&p};
         LB_TRY(lb_launch(c, LBK_da_inputs, (unsigned)((D->heads * L->dk_p + 255) / 256), (unsigned)((T + 7) / 8), 1, 256, (unsigned)(8 * (D->rank > 0 ? D->rank : 1) * 4), params, 1));
-        const int tok = 3 * (L->dk_p + 8 * 4) + 32; /* floats a token's operands take in a stage */
-        LB_TRY(lb_launch(c, L->dk_p == 64 ? LBK_da_scan_64 : L->dk_p == 128 ? LBK_da_scan_128 : LBK_da_scan_256, (unsigned)D->heads, (unsigned)((D->vdim + 31) / 32), 1, 128,
+        const int part = L->dk_p / 16, tok = 3 * 16 * (part == 4 ? 4 : part + 4) + 32; /* floats a token's operands take in a stage */
+        LB_TRY(lb_launch(c, L->dk_p == 64 ? LBK_da_scan_64 : L->dk_p == 128 ? LBK_da_scan_128 : LBK_da_scan_256, (unsigned)D->heads, (unsigned)((D->vdim + 31) / 32), 1, 256,
                          (unsigned)(3 * 4 * tok * 4), params, 1));
         LB_TRY(lb_launch(c, LBK_da_finish, (unsigned)T, (unsigned)((D->heads + 3) / 4), 1, 128, 0, params, 1));
     }
@@ -440,7 +453,7 @@ static int stack_head_rows(lb_model* m, CUdeviceptr rows, int n, CUdeviceptr log
 
 static void stack_pf_sizes(const lb_model* m, size_t bytes[LB_PF_MAX_BUFS]) {
     const stack_t* S = S_of(m);
-    const size_t T = ST_CHUNK, e = (size_t)S->esz, q = (size_t)S->max_dk * 4 > (size_t)S->max_q * 2 ? (size_t)S->max_dk * 4 : (size_t)S->max_q * 2;
+    const size_t T = (size_t)m->pf_chunk, e = (size_t)S->esz, q = (size_t)S->max_dk * 4 > (size_t)S->max_q * 2 ? (size_t)S->max_dk * 4 : (size_t)S->max_q * 2;
     const size_t b[] = {T * (size_t)S->d.width * 4, T * (size_t)S->Kw * e, T * (size_t)S->Kw * e, T * (size_t)S->max_in * 4, T * (size_t)S->max_cat * e,
                         T * q, T * q, T * (size_t)S->max_dk * 4, T * (size_t)S->max_o * 4};
     memcpy(bytes, b, sizeof b); /* in the order of pf_set.st */
@@ -503,8 +516,28 @@ static void stack_destroy(lb_model* m) {
     S->d.layer = NULL;
 }
 
-static const lb_arch k_stack = {"stack", ST_CHUNK, ST_STREAMS, stack_reset_state, stack_snapshot, stack_state_ptr, stack_step_layers, stack_head,
+static const lb_arch k_stack = {"stack", ST_STREAMS, stack_reset_state, stack_snapshot, stack_state_ptr, stack_step_layers, stack_head,
                                 stack_head_ctas, stack_head_rows, stack_pf_sizes, stack_pf_layer, stack_destroy};
+
+/* tokens per prompt chunk: the multiple of 256 whose products fill whole waves of SMs best */
+static int stack_chunk(const lb_model* m) {
+    const stack_t* S = S_of(m);
+    double best = 1e30;
+    int chunk = 256;
+    for (int T = 256; T <= ST_CHUNK; T += 256) {
+        double cost = 0;
+        for (int i = 0; i < S->d.n_layers; i++) {
+            const st_layer* L = &S->L[i];
+            int nt;
+            cost += L->in.K * product_cost(m->c, (L->in.rows + LB_DG_ROWS - 1) / LB_DG_ROWS + (L->ff.rows + LB_DG_ROWS - 1) / LB_DG_ROWS, T, &nt) +
+                    L->out.K * product_cost(m->c, (L->out.rows + LB_DG_ROWS - 1) / LB_DG_ROWS, T, &nt);
+        }
+        cost /= T;
+        if (T < 512) cost *= 1.05; /* weights read once per chunk */
+        if (cost < best * 0.999) { best = cost; chunk = T; }
+    }
+    return chunk;
+}
 
 static int stack_build(lb_model* m, const lb_stack_desc* d, lb_weight_source* src) {
     lb_ctx* c = m->c;
@@ -563,6 +596,7 @@ static int stack_build(lb_model* m, const lb_stack_desc* d, lb_weight_source* sr
     LB_TRY(lb_dalloc(m, &S->counters, (size_t)groups_max * 4));
     LB_CU(c, lb_drv.MemsetD8Async(S->counters, 0, (size_t)groups_max * 4, c->stream));
     m->globals_loaded = 1;
+    m->pf_chunk = stack_chunk(m);
     return lb_model_reset_state(m);
 }
 

@@ -130,13 +130,15 @@ extern "C" __global__ void __launch_bounds__(256) da_inputs(const __grid_constan
     pdl_launch_dependents();
 }
 
-// grid (H, ceil(dv / 32)), block 128.  Thread (column pair, row eighth) holds R = dk_p / 8 rows of two columns as packed pairs of
+// grid (H, ceil(dv / 32)), block 256.  Thread (column pair, row sixteenth) holds R = dk_p / 16 rows of two columns as packed pairs of
 // rows, so that the state update and the read-out are two-wide fp32 instructions and a row of q, k, a is read from shared memory once for
-// two columns.  Operands of DA_U tokens at a time come DA_AHEAD - 1 stages ahead by cp.async (a row eighth is padded by 16 bytes: the eight
-// addresses of a warp's 16-byte reads sit on different banks); one block barrier per DA_U tokens, and no branch between the tokens of a
-// full stage, so that the next token's operands are read under the present one's arithmetic.
+// two columns.  A step is a chain of latencies: what counts is how many warps a scheduler has to choose from, hence few rows per thread.
+// Operands of DA_U tokens at a time come DA_AHEAD - 1 stages ahead by cp.async (a row part is padded so that eight neighbouring lanes'
+// 16-byte reads sit on different banks); one block barrier per DA_U tokens, and no branch between the tokens of a full stage, so that the
+// next token's operands are read under the present one's arithmetic.
 #define DA_U 4
 #define DA_AHEAD 3
+#define DA_SCAN_THREADS 256
 __device__ __forceinline__ void da_cp16(void* dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
@@ -168,23 +170,23 @@ struct __align__(16) da_quad { da_f2 lo, hi; }; // four consecutive rows
 
 template <int R>
 __device__ __forceinline__ void da_scan_body(const lb_decay_params2& p) {
-    constexpr int QS = R + 4, VEC = 8 * QS, TOK = 3 * VEC + DA_COLS; // floats: a row eighth, a vector, a token's operands
+    constexpr int QS = R == 4 ? 4 : R + 4, VEC = 16 * QS, TOK = 3 * VEC + DA_COLS; // floats: a row part, a vector, a token's operands
     extern __shared__ __align__(16) float da_sm[];                   // [DA_AHEAD][DA_U][TOK]
-    const int h = blockIdx.x, t = threadIdx.x, e8 = t & 7, j = blockIdx.y * DA_COLS + 2 * (t >> 3);
+    const int h = blockIdx.x, t = threadIdx.x, e = t & 15, j = blockIdx.y * DA_COLS + 2 * (t >> 4);
     const bool live0 = j < p.dv, live1 = j + 1 < p.dv;
-    float* S = p.state + ((size_t)h * p.dk + (size_t)e8 * R) * p.dv + j;
-    const int rows = min(R, p.dk - e8 * R);
+    float* S = p.state + ((size_t)h * p.dk + (size_t)e * R) * p.dv + j;
+    const int rows = min(R, p.dk - e * R);
     pdl_wait();
     const int n_st = (p.T + DA_U - 1) / DA_U;
     auto fetch = [&](int st) {
         float* dst = da_sm + (size_t)(st % DA_AHEAD) * (DA_U * TOK);
-        constexpr int PIECES = 3 * 2 * R; // 16-byte pieces of q, k, a (8 R floats each)
-        for (int i = t; i < DA_U * PIECES; i += DA_THREADS) {
-            const int u = i / PIECES, c = i - u * PIECES, which = c / (2 * R), pc = c - which * (2 * R), tok = min(st * DA_U + u, p.T - 1);
-            const float* src = (which == 0 ? p.q : which == 1 ? p.k : p.a) + ((size_t)tok * p.H + h) * (8 * R) + pc * 4;
+        constexpr int PIECES = 3 * 4 * R; // 16-byte pieces of q, k, a (16 R floats each)
+        for (int i = t; i < DA_U * PIECES; i += DA_SCAN_THREADS) {
+            const int u = i / PIECES, c = i - u * PIECES, which = c / (4 * R), pc = c - which * (4 * R), tok = min(st * DA_U + u, p.T - 1);
+            const float* src = (which == 0 ? p.q : which == 1 ? p.k : p.a) + ((size_t)tok * p.H + h) * (16 * R) + pc * 4;
             da_cp16(dst + u * TOK + which * VEC + (pc / (R / 4)) * QS + (pc % (R / 4)) * 4, src);
         }
-        { // DA_U x 32 values: one per thread
+        if (t < DA_U * 32) { // DA_U x 32 values
             const int u = t >> 5, cc = t & 31, tok = min(st * DA_U + u, p.T - 1), col = min(blockIdx.y * DA_COLS + cc, p.dv - 1);
             da_cp4(dst + u * TOK + 3 * VEC + cc, p.proj + (size_t)tok * p.ld + p.v_off + (size_t)h * p.dv + col);
         }
@@ -203,10 +205,10 @@ __device__ __forceinline__ void da_scan_body(const lb_decay_params2& p) {
         s1[r / 2] = da_pack(at(r, 1, live1), at(r + 1, 1, live1));
     }
     auto step = [&](const float* tk, float& o0, float& o1) { // one token: state update, this thread's share of the two read-outs
-        const float2 v = *reinterpret_cast<const float2*>(tk + 3 * VEC + 2 * (t >> 3));
+        const float2 v = *reinterpret_cast<const float2*>(tk + 3 * VEC + 2 * (t >> 4));
         const da_f2 v0 = da_pack(v.x, v.x), v1 = da_pack(v.y, v.y);
-        const da_quad *qv = reinterpret_cast<const da_quad*>(tk + e8 * QS), *kv = reinterpret_cast<const da_quad*>(tk + VEC + e8 * QS),
-                      *av = reinterpret_cast<const da_quad*>(tk + 2 * VEC + e8 * QS);
+        const da_quad *qv = reinterpret_cast<const da_quad*>(tk + e * QS), *kv = reinterpret_cast<const da_quad*>(tk + VEC + e * QS),
+                      *av = reinterpret_cast<const da_quad*>(tk + 2 * VEC + e * QS);
         da_f2 a0 = 0ull, a1 = 0ull, b0 = 0ull, b1 = 0ull;
 #pragma unroll
         for (int c = 0; c < R / 4; ++c) {
@@ -241,17 +243,20 @@ __device__ __forceinline__ void da_scan_body(const lb_decay_params2& p) {
                 if (st * DA_U + u < p.T) step(base + u * TOK, o[2 * u], o[2 * u + 1]);
             }
         }
-        // sums over the column's eight lanes: every exchange halves what a lane still holds, lane e8 ends with (token e8 / 2, column e8 & 1)
+        // sums over the column's 16 lanes: the first three exchanges each halve what a lane still holds, the last adds two lanes: lanes
+        // e and e ^ 1 end with token e / 4, column (e / 2) & 1
 #pragma unroll
         for (int half = 4; half >= 1; half >>= 1) {
-            const bool up = (e8 & half) != 0;
+            const bool up = (e & (2 * half)) != 0;
 #pragma unroll
             for (int i = 0; i < half; ++i) {
                 const float give = up ? o[i] : o[i + half], keep = up ? o[i + half] : o[i];
-                o[i] = keep + __shfl_xor_sync(0xffffffffu, give, half);
+                o[i] = keep + __shfl_xor_sync(0xffffffffu, give, 2 * half);
             }
         }
-        const int tok = st * DA_U + (e8 >> 1), col = j + (e8 & 1);
+        o[0] += __shfl_xor_sync(0xffffffffu, o[0], 1);
+        const int tok = st * DA_U + (e >> 2), col = j + ((e >> 1) & 1);
+        if (e & 1) continue;
         if (col < p.dv && tok < p.T) p.o[(size_t)tok * p.H * p.dv + (size_t)h * p.dv + col] = o[0];
     }
     pdl_launch_dependents();
@@ -268,10 +273,10 @@ __device__ __forceinline__ void da_scan_body(const lb_decay_params2& p) {
         }
     }
 }
-static_assert(DA_U == 4 && DA_THREADS == 32 * DA_U, "one value per thread and stage; two tokens' columns per lane of a column pair");
-extern "C" __global__ void __launch_bounds__(DA_THREADS) da_scan_64(const __grid_constant__ lb_decay_params2 p) { da_scan_body<8>(p); }
-extern "C" __global__ void __launch_bounds__(DA_THREADS) da_scan_128(const __grid_constant__ lb_decay_params2 p) { da_scan_body<16>(p); }
-extern "C" __global__ void __launch_bounds__(DA_THREADS) da_scan_256(const __grid_constant__ lb_decay_params2 p) { da_scan_body<32>(p); }
+static_assert(DA_U == 4, "four tokens of two columns are what three halvings leave one of");
+extern "C" __global__ void __launch_bounds__(DA_SCAN_THREADS) da_scan_64(const __grid_constant__ lb_decay_params2 p) { da_scan_body<4>(p); }
+extern "C" __global__ void __launch_bounds__(DA_SCAN_THREADS) da_scan_128(const __grid_constant__ lb_decay_params2 p) { da_scan_body<8>(p); }
+extern "C" __global__ void __launch_bounds__(DA_SCAN_THREADS) da_scan_256(const __grid_constant__ lb_decay_params2 p) { da_scan_body<16>(p); }
 
 // cat[t, h dv + i] = o / rms_head(o) * head_w[i] [ * silu(gate) ].  grid (T, ceil(H / 4)), block 128: one warp per (token, head)
 extern "C" __global__ void __launch_bounds__(128) da_finish(const __grid_constant__ lb_decay_params2 p) {
