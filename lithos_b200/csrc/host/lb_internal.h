@@ -144,6 +144,9 @@ int lb_driver_load(char* err, size_t errlen); /* LB_OK or LB_ERR_NO_DRIVER */
     X(da_step_128)                    \
     X(da_step_256)                    \
     X(da_inputs)                      \
+    X(da_local_64)                    \
+    X(da_local_128)                   \
+    X(da_local_256)                   \
     X(da_scan_64)                     \
     X(da_scan_128)                    \
     X(da_scan_256)                    \

@@ -38,7 +38,7 @@ typedef struct {
 typedef union {
     CUdeviceptr b[LB_PF_MAX_BUFS];
     struct { CUdeviceptr X, xn16, proj, q, k, v, g, beta, mix, mix16, y, gu, act16; } hy; /* lb_hybrid.c */
-    struct { CUdeviceptr X, h1, h2, proj, cat, q, k, a, o; } st;                            /* lb_stack.c */
+    struct { CUdeviceptr X, h1, h2, proj, cat, q, k, a, o, seg_state, seg_decay; } st;                        /* lb_stack.c */
 } pf_set;
 
 /* What an architecture supplies.  The runtime owns embedding, order of calls, positions, graph capture, chunking and

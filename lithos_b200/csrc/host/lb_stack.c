@@ -19,6 +19,7 @@
 
 #define ST_CHUNK 1024 /* largest chunk of a prompt; stack_chunk picks the model's */
 #define ST_STREAMS 4
+#define ST_SEG 128     /* tokens of a chunk a recurrence walks one after the other; segments run side by side */
 
 typedef struct {
     CUdeviceptr w;
@@ -44,10 +45,12 @@ typedef struct {
     int Kw; /* width padded to 64 columns */
     int esz; /* bytes of an activation / cache element: 2 (bf16) or 4 (fp32) */
     int max_in, max_cat, max_mix, max_ff, max_q, max_dk, max_o;
+    size_t max_state;
     CUdeviceptr proj, mix, act;        /* decode step: fp32 */
     CUdeviceptr scratch, counters;
 } stack_t;
 
+static size_t state_bytes(const lb_stack_layer* D) { return (size_t)D->heads * D->dim * D->vdim * 4; }
 static int pad_to(int n, int m) { return (n + m - 1) / m * m; }
 static stack_t* S_of(const lb_model* m) { return (stack_t*)m->impl; }
 
@@ -434,9 +437,13 @@ static int stack_pf_layer(lb_model* m, pf_set* w, int i, int pos0, int T) {
         p.cat = (void*)w->st.cat; p.cat_ld = L->out.K; p.cat_f32 = f32;
         void* params[] = {&p};
         LB_TRY(lb_launch(c, LBK_da_inputs, (unsigned)((D->heads * L->dk_p + 255) / 256), (unsigned)((T + 7) / 8), 1, 256, (unsigned)(8 * (D->rank > 0 ? D->rank : 1) * 4), params, 1));
-        const int part = L->dk_p / 16, tok = 3 * 16 * (part == 4 ? 4 : part + 4) + 32; /* floats a token's operands take in a stage */
-        LB_TRY(lb_launch(c, L->dk_p == 64 ? LBK_da_scan_64 : L->dk_p == 128 ? LBK_da_scan_128 : LBK_da_scan_256, (unsigned)D->heads, (unsigned)((D->vdim + 31) / 32), 1, 256,
-                         (unsigned)(3 * 4 * tok * 4), params, 1));
+        const int part = L->dk_p / 16, tok = 3 * 16 * (part == 4 ? 4 : part + 4) + 64; /* floats a token's operands take in a stage */
+        const int dki = L->dk_p == 64 ? 0 : L->dk_p == 128 ? 1 : 2;
+        static const int k_scan[3] = {LBK_da_scan_64, LBK_da_scan_128, LBK_da_scan_256}, k_local[3] = {LBK_da_local_64, LBK_da_local_128, LBK_da_local_256};
+        const unsigned slabs = (unsigned)((D->vdim + 63) / 64), threads = dki == 2 ? 256 : 128, smem = (unsigned)(3 * 4 * tok * 4), segs = (unsigned)((T + ST_SEG - 1) / ST_SEG);
+        p.seg = ST_SEG; p.seg_state = (float*)w->st.seg_state; p.seg_decay = (float*)w->st.seg_decay;
+        if (segs > 1) LB_TRY(lb_launch(c, k_local[dki], (unsigned)D->heads, slabs, segs, threads, smem, params, 1));
+        LB_TRY(lb_launch(c, k_scan[dki], (unsigned)D->heads, slabs, segs, threads, smem, params, 1));
         LB_TRY(lb_launch(c, LBK_da_finish, (unsigned)T, (unsigned)((D->heads + 3) / 4), 1, 128, 0, params, 1));
     }
     const st_prod out = {&L->out, w->st.cat, w->st.X, LB_DY_RESIDUAL, S->d.width};
@@ -455,13 +462,12 @@ static void stack_pf_sizes(const lb_model* m, size_t bytes[LB_PF_MAX_BUFS]) {
     const stack_t* S = S_of(m);
     const size_t T = (size_t)m->pf_chunk, e = (size_t)S->esz, q = (size_t)S->max_dk * 4 > (size_t)S->max_q * 2 ? (size_t)S->max_dk * 4 : (size_t)S->max_q * 2;
     const size_t b[] = {T * (size_t)S->d.width * 4, T * (size_t)S->Kw * e, T * (size_t)S->Kw * e, T * (size_t)S->max_in * 4, T * (size_t)S->max_cat * e,
-                        T * q, T * q, T * (size_t)S->max_dk * 4, T * (size_t)S->max_o * 4};
+                        T * q, T * q, T * (size_t)S->max_dk * 4, T * (size_t)S->max_o * 4,
+                        (T + ST_SEG - 1) / ST_SEG * S->max_state, (T + ST_SEG - 1) / ST_SEG * (size_t)S->max_dk * 4};
     memcpy(bytes, b, sizeof b); /* in the order of pf_set.st */
 }
 
 /* ---- state ---------------------------------------------------------------------------------------------------------------- */
-static size_t state_bytes(const lb_stack_layer* D) { return (size_t)D->heads * D->dim * D->vdim * 4; }
-
 static int stack_reset_state(lb_model* m) { /* cache rows past the position are never read: only the recurrent states start over */
     const stack_t* S = S_of(m);
     for (int i = 0; i < S->d.n_layers; i++)
@@ -576,6 +582,7 @@ static int stack_build(lb_model* m, const lb_stack_desc* d, lb_weight_source* sr
             MAX(groups_max, groups);
         } else {
             MAX(S->max_dk, D->heads * L->dk_p);
+            MAX(S->max_state, state_bytes(D));
             MAX(S->max_o, D->heads * D->vdim);
         }
 #undef MAX

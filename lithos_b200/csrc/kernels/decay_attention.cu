@@ -5,7 +5,8 @@
 // row part) has R rows of its column (rows past dk stay zero), the sum over rows is local terms and a few shuffles.
 //   da_step_*   one token (decode): makes q, k, a of its head from the projections, state read and written once
 //   da_inputs   a prompt chunk's q, k, a
-//   da_scan_*   a prompt chunk through the recurrence, the state on chip for all of it
+//   da_scan_*   a prompt chunk through the recurrence, the state on chip; a long chunk in two passes over segments of it, so that the
+//               segments run side by side: da_local_* carries every segment from a zero state, da_scan_* starts each from its true state
 //   da_finish   per-head norm (and output gate) of the chunk's read-outs
 #include "common.cuh"
 #include "params.h"
@@ -130,15 +131,14 @@ extern "C" __global__ void __launch_bounds__(256) da_inputs(const __grid_constan
     pdl_launch_dependents();
 }
 
-// grid (H, ceil(dv / 32)), block 256.  Thread (column pair, row sixteenth) holds R = dk_p / 16 rows of two columns as packed pairs of
-// rows, so that the state update and the read-out are two-wide fp32 instructions and a row of q, k, a is read from shared memory once for
-// two columns.  A step is a chain of latencies: what counts is how many warps a scheduler has to choose from, hence few rows per thread.
-// Operands of DA_U tokens at a time come DA_AHEAD - 1 stages ahead by cp.async (a row part is padded so that eight neighbouring lanes'
-// 16-byte reads sit on different banks); one block barrier per DA_U tokens, and no branch between the tokens of a full stage, so that the
-// next token's operands are read under the present one's arithmetic.
+// grid (H, ceil(dv / 64), segments), block 16 x 64 / C.  Thread (C columns, row sixteenth) holds R = dk_p / 16 rows of C columns as packed
+// pairs of rows, so that the state update and the read-out are two-wide fp32 instructions and a row of q, k, a is read from shared memory
+// once for C columns (with two columns those reads bounded the kernel).  Operands of DA_U tokens at a time come DA_AHEAD - 1 stages ahead by
+// cp.async (a row part is padded so that eight neighbouring lanes' 16-byte reads sit on different banks); one block barrier per DA_U tokens,
+// and no branch between the tokens of a full stage, so that the next token's operands are read under the present one's arithmetic.
 #define DA_U 4
 #define DA_AHEAD 3
-#define DA_SCAN_THREADS 256
+#define DA_SLAB 64 /* columns per CTA */
 __device__ __forceinline__ void da_cp16(void* dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
@@ -168,115 +168,192 @@ __device__ __forceinline__ da_f2 da_mul2(da_f2 a, da_f2 b) {
 }
 struct __align__(16) da_quad { da_f2 lo, hi; }; // four consecutive rows
 
-template <int R>
+// Segments (gridDim.z = P > 1; segment g is tokens g * seg .. of the chunk).  The state after a segment is diag(b) S_in + L, b the product
+// of its decays and L what it makes of a zero state.  LOCAL (first launch): every segment leaves L and b in the workspace; segment 0 starts
+// from the sequence's state, so its L is a true state.  Second launch: segment g makes its S_in from the L and b of those before it, then runs
+// with read-outs; segment 0, the only one that touches the sequence's state, replaces it by the state after the last segment.
+template <int R, int C, bool LOCAL>
 __device__ __forceinline__ void da_scan_body(const lb_decay_params2& p) {
-    constexpr int QS = R == 4 ? 4 : R + 4, VEC = 16 * QS, TOK = 3 * VEC + DA_COLS; // floats: a row part, a vector, a token's operands
-    extern __shared__ __align__(16) float da_sm[];                   // [DA_AHEAD][DA_U][TOK]
-    const int h = blockIdx.x, t = threadIdx.x, e = t & 15, j = blockIdx.y * DA_COLS + 2 * (t >> 4);
-    const bool live0 = j < p.dv, live1 = j + 1 < p.dv;
-    float* S = p.state + ((size_t)h * p.dk + (size_t)e * R) * p.dv + j;
-    const int rows = min(R, p.dk - e * R);
+    constexpr int DA_SCAN_THREADS = 16 * DA_SLAB / C;
+    constexpr int QS = R == 4 ? 4 : R + 4, VEC = 16 * QS, TOK = 3 * VEC + DA_SLAB; // floats: a row part, a vector, a token's operands
+    constexpr int PV = 4 * R, PIECES = (LOCAL ? 2 : 3) * PV;                         // 16-byte pieces of a vector; of a token (no q for LOCAL)
+    constexpr int NI = (DA_U * PIECES + DA_SCAN_THREADS - 1) / DA_SCAN_THREADS;
+    extern __shared__ __align__(16) float da_sm[]; // [DA_AHEAD][DA_U][TOK]
+    const int h = blockIdx.x, t = threadIdx.x, e = t & 15, cg = t >> 4, j = blockIdx.y * DA_SLAB + C * cg;
+    const int g = blockIdx.z, P = gridDim.z, tok0 = g * p.seg, n_tok = min(p.seg, p.T - tok0), n_st = (n_tok + DA_U - 1) / DA_U;
+    const int rows = min(R, p.dk - e * R), cols = min(C, p.dv - j); // what of this thread's tile exists
+    const size_t head_off = ((size_t)h * p.dk + (size_t)e * R) * p.dv + j, all = (size_t)p.H * p.dk * p.dv; // this thread's corner of a state
     pdl_wait();
-    const int n_st = (p.T + DA_U - 1) / DA_U;
-    auto fetch = [&](int st) {
-        float* dst = da_sm + (size_t)(st % DA_AHEAD) * (DA_U * TOK);
-        constexpr int PIECES = 3 * 4 * R; // 16-byte pieces of q, k, a (16 R floats each)
-        for (int i = t; i < DA_U * PIECES; i += DA_SCAN_THREADS) {
-            const int u = i / PIECES, c = i - u * PIECES, which = c / (4 * R), pc = c - which * (4 * R), tok = min(st * DA_U + u, p.T - 1);
-            const float* src = (which == 0 ? p.q : which == 1 ? p.k : p.a) + ((size_t)tok * p.H + h) * (16 * R) + pc * 4;
-            da_cp16(dst + u * TOK + which * VEC + (pc / (R / 4)) * QS + (pc % (R / 4)) * 4, src);
+    // operands: a thread copies the same pieces of every stage, so only the source moves on.  A last stage reads past the chunk's tokens
+    // (the buffers hold a whole number of stages); what it reads there is not used.
+    const float* src[NI];
+    int dst[NI];
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+        const int idx = t + i * DA_SCAN_THREADS, u = idx / PIECES, c = idx - u * PIECES, which = c / PV + (LOCAL ? 1 : 0), pc = c % PV;
+        src[i] = (which == 0 ? p.q : which == 1 ? p.k : p.a) + ((size_t)(tok0 + u) * p.H + h) * (16 * R) + pc * 4;
+        dst[i] = u * TOK + which * VEC + (pc / (R / 4)) * QS + (pc % (R / 4)) * 4;
+    }
+    const float* vsrc = p.proj + (size_t)(tok0 + t / DA_SLAB) * p.ld + p.v_off + (size_t)h * p.dv + min(blockIdx.y * DA_SLAB + t % DA_SLAB, (unsigned)p.dv - 1u);
+    const size_t step_qka = (size_t)DA_U * p.H * (16 * R), step_v = (size_t)DA_U * p.ld;
+    int f_slot = 0;
+    auto fetch = [&]() {
+        float* d = da_sm + f_slot * (DA_U * TOK);
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            if ((i + 1) * DA_SCAN_THREADS <= DA_U * PIECES || t + i * DA_SCAN_THREADS < DA_U * PIECES) da_cp16(d + dst[i], src[i]);
+            src[i] += step_qka;
         }
-        if (t < DA_U * 32) { // DA_U x 32 values
-            const int u = t >> 5, cc = t & 31, tok = min(st * DA_U + u, p.T - 1), col = min(blockIdx.y * DA_COLS + cc, p.dv - 1);
-            da_cp4(dst + u * TOK + 3 * VEC + cc, p.proj + (size_t)tok * p.ld + p.v_off + (size_t)h * p.dv + col);
-        }
+#pragma unroll
+        for (int u = 0; u < DA_U; u += DA_SCAN_THREADS / DA_SLAB)
+            da_cp4(d + (u + t / DA_SLAB) * TOK + 3 * VEC + t % DA_SLAB, vsrc + (size_t)u * p.ld);
+        vsrc += step_v;
+        if (++f_slot == DA_AHEAD) f_slot = 0;
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
 #pragma unroll
     for (int st = 0; st < DA_AHEAD - 1; ++st) {
-        if (st < n_st) fetch(st);
+        if (st < n_st) fetch();
         else asm volatile("cp.async.commit_group;" ::: "memory");
     }
-    da_f2 s0[R / 2], s1[R / 2]; // rows (2r, 2r + 1) of the two columns
+    // the tile as pairs of rows (2r, 2r + 1), column by column
+    da_f2 s[C][R / 2];
+    auto load = [&](const float* S) {
 #pragma unroll
-    for (int r = 0; r < R; r += 2) {
-        auto at = [&](int rr, int c, bool on) { return on && rr < rows ? S[(size_t)rr * p.dv + c] : 0.f; };
-        s0[r / 2] = da_pack(at(r, 0, live0), at(r + 1, 0, live0));
-        s1[r / 2] = da_pack(at(r, 1, live1), at(r + 1, 1, live1));
+        for (int r = 0; r < R; r += 2)
+#pragma unroll
+            for (int c = 0; c < C; ++c)
+                s[c][r / 2] = da_pack(c < cols && r < rows ? S[(size_t)r * p.dv + c] : 0.f, c < cols && r + 1 < rows ? S[(size_t)(r + 1) * p.dv + c] : 0.f);
+    };
+    auto store = [&](float* S) {
+#pragma unroll
+        for (int r = 0; r < R; r += 2)
+#pragma unroll
+            for (int c = 0; c < C; ++c) {
+                const float2 x = da_unpack(s[c][r / 2]);
+                if (c < cols && r < rows) S[(size_t)r * p.dv + c] = x.x;
+                if (c < cols && r + 1 < rows) S[(size_t)(r + 1) * p.dv + c] = x.y;
+            }
+    };
+    auto advance = [&](int seg) { // the state through a whole segment: S <- diag(b) S + L
+        const float* L = p.seg_state + (size_t)seg * all + head_off;
+        const float* b = p.seg_decay + ((size_t)seg * p.H + h) * (16 * R) + e * R;
+#pragma unroll
+        for (int r = 0; r < R; r += 2) {
+            const da_f2 bb = da_pack(b[r], b[r + 1]);
+#pragma unroll
+            for (int c = 0; c < C; ++c)
+                s[c][r / 2] = da_fma2(bb, s[c][r / 2], da_pack(c < cols && r < rows ? L[(size_t)r * p.dv + c] : 0.f, c < cols && r + 1 < rows ? L[(size_t)(r + 1) * p.dv + c] : 0.f));
+        }
+    };
+    if (LOCAL ? g > 0 : false) {
+#pragma unroll
+        for (int c = 0; c < C; ++c)
+#pragma unroll
+            for (int r = 0; r < R / 2; ++r) s[c][r] = 0ull;
+    } else if (LOCAL || g == 0) {
+        load(p.state + head_off);
+    } else {
+        load(p.seg_state + head_off);
+        for (int q = 1; q < g; ++q) advance(q);
     }
-    auto step = [&](const float* tk, float& o0, float& o1) { // one token: state update, this thread's share of the two read-outs
-        const float2 v = *reinterpret_cast<const float2*>(tk + 3 * VEC + 2 * (t >> 4));
-        const da_f2 v0 = da_pack(v.x, v.x), v1 = da_pack(v.y, v.y);
+    da_f2 dec[R / 2]; // LOCAL: product of the segment's decays
+#pragma unroll
+    for (int r = 0; r < R / 2; ++r) dec[r] = da_pack(1.f, 1.f);
+
+    auto step = [&](const float* tk, int tok) { // one token: state update, read-out
+        float v[C];
+#pragma unroll
+        for (int c = 0; c < C; c += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(tk + 3 * VEC + C * cg + c);
+            v[c] = x.x; v[c + 1] = x.y; v[c + 2] = x.z; v[c + 3] = x.w;
+        }
         const da_quad *qv = reinterpret_cast<const da_quad*>(tk + e * QS), *kv = reinterpret_cast<const da_quad*>(tk + VEC + e * QS),
                       *av = reinterpret_cast<const da_quad*>(tk + 2 * VEC + e * QS);
-        da_f2 a0 = 0ull, a1 = 0ull, b0 = 0ull, b1 = 0ull;
+        da_f2 acc[C];
 #pragma unroll
-        for (int c = 0; c < R / 4; ++c) {
-            const da_quad q = qv[c], k = kv[c], a = av[c];
-            s0[2 * c] = da_fma2(a.lo, s0[2 * c], da_mul2(k.lo, v0));
-            s1[2 * c] = da_fma2(a.lo, s1[2 * c], da_mul2(k.lo, v1));
-            s0[2 * c + 1] = da_fma2(a.hi, s0[2 * c + 1], da_mul2(k.hi, v0));
-            s1[2 * c + 1] = da_fma2(a.hi, s1[2 * c + 1], da_mul2(k.hi, v1));
-            a0 = da_fma2(s0[2 * c], q.lo, a0);
-            b0 = da_fma2(s1[2 * c], q.lo, b0);
-            a1 = da_fma2(s0[2 * c + 1], q.hi, a1);
-            b1 = da_fma2(s1[2 * c + 1], q.hi, b1);
-        }
-        const float2 x0 = da_unpack(a0), x1 = da_unpack(a1), y0 = da_unpack(b0), y1 = da_unpack(b1);
-        o0 = (x0.x + x0.y) + (x1.x + x1.y);
-        o1 = (y0.x + y0.y) + (y1.x + y1.y);
-    };
-    for (int st = 0; st < n_st; ++st) {
-        asm volatile("cp.async.wait_group %0;" ::"n"(DA_AHEAD - 2) : "memory");
-        __syncthreads(); // everybody's pieces have landed, and everybody is done with the stage the next fetch fills
-        if (st + DA_AHEAD - 1 < n_st) fetch(st + DA_AHEAD - 1);
-        else asm volatile("cp.async.commit_group;" ::: "memory");
-        const float* base = da_sm + (size_t)(st % DA_AHEAD) * (DA_U * TOK);
-        float o[2 * DA_U]; // [token][column]
-        if ((st + 1) * DA_U <= p.T) {
+        for (int c = 0; c < C; ++c) acc[c] = 0ull;
 #pragma unroll
-            for (int u = 0; u < DA_U; ++u) step(base + u * TOK, o[2 * u], o[2 * u + 1]);
-        } else { // the chunk ends inside this stage: tokens past it leave the state alone
+        for (int i = 0; i < R / 4; ++i) {
+            const da_quad k = kv[i], a = av[i];
+            da_quad q;
+            if (!LOCAL) q = qv[i];
 #pragma unroll
-            for (int u = 0; u < DA_U; ++u) {
-                o[2 * u] = o[2 * u + 1] = 0.f;
-                if (st * DA_U + u < p.T) step(base + u * TOK, o[2 * u], o[2 * u + 1]);
+            for (int c = 0; c < C; ++c) {
+                const da_f2 vv = da_pack(v[c], v[c]);
+                s[c][2 * i] = da_fma2(a.lo, s[c][2 * i], da_mul2(k.lo, vv));
+                s[c][2 * i + 1] = da_fma2(a.hi, s[c][2 * i + 1], da_mul2(k.hi, vv));
+                if (!LOCAL) acc[c] = da_fma2(s[c][2 * i + 1], q.hi, da_fma2(s[c][2 * i], q.lo, acc[c]));
+            }
+            if (LOCAL) {
+                dec[2 * i] = da_mul2(dec[2 * i], a.lo);
+                dec[2 * i + 1] = da_mul2(dec[2 * i + 1], a.hi);
             }
         }
-        // sums over the column's 16 lanes: the first three exchanges each halve what a lane still holds, the last adds two lanes: lanes
-        // e and e ^ 1 end with token e / 4, column (e / 2) & 1
+        if (LOCAL) return;
+        float o[C];
 #pragma unroll
-        for (int half = 4; half >= 1; half >>= 1) {
-            const bool up = (e & (2 * half)) != 0;
+        for (int c = 0; c < C; ++c) {
+            const float2 x = da_unpack(acc[c]);
+            o[c] = x.x + x.y;
+        }
+        // sums over the 16 row parts: each of the first exchanges halves what a lane still holds, the others add two lanes
+        int bit = 8;
+#pragma unroll
+        for (int half = C / 2; half >= 1; half >>= 1, bit >>= 1) {
+            const bool up = (e & bit) != 0;
 #pragma unroll
             for (int i = 0; i < half; ++i) {
                 const float give = up ? o[i] : o[i + half], keep = up ? o[i + half] : o[i];
-                o[i] = keep + __shfl_xor_sync(0xffffffffu, give, 2 * half);
+                o[i] = keep + __shfl_xor_sync(0xffffffffu, give, bit);
             }
         }
-        o[0] += __shfl_xor_sync(0xffffffffu, o[0], 1);
-        const int tok = st * DA_U + (e >> 2), col = j + ((e >> 1) & 1);
-        if (e & 1) continue;
-        if (col < p.dv && tok < p.T) p.o[(size_t)tok * p.H * p.dv + (size_t)h * p.dv + col] = o[0];
+#pragma unroll
+        for (; bit >= 1; bit >>= 1) o[0] += __shfl_xor_sync(0xffffffffu, o[0], bit);
+        const int col = e / (16 / C);
+        if (e % (16 / C) == 0 && col < cols) p.o[((size_t)(tok0 + tok) * p.H + h) * p.dv + j + col] = o[0];
+    };
+    int slot = 0;
+    for (int st = 0; st < n_st; ++st) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(DA_AHEAD - 2) : "memory");
+        __syncthreads(); // everybody's pieces have landed, and everybody is done with the stage the next fetch fills
+        if (st + DA_AHEAD - 1 < n_st) fetch();
+        else asm volatile("cp.async.commit_group;" ::: "memory");
+        const float* base = da_sm + slot * (DA_U * TOK);
+        if (++slot == DA_AHEAD) slot = 0;
+        if ((st + 1) * DA_U <= n_tok) {
+#pragma unroll
+            for (int u = 0; u < DA_U; ++u) step(base + u * TOK, st * DA_U + u);
+        } else { // the segment ends inside this stage: tokens past it leave the state alone
+            for (int u = 0; st * DA_U + u < n_tok; ++u) step(base + u * TOK, st * DA_U + u);
+        }
     }
     pdl_launch_dependents();
+    if (LOCAL) {
+        store(p.seg_state + (size_t)g * all + head_off);
+        if (blockIdx.y == 0 && t < 16) {
+            float* b = p.seg_decay + ((size_t)g * p.H + h) * (16 * R) + e * R;
 #pragma unroll
-    for (int r = 0; r < R; r += 2) {
-        const float2 x = da_unpack(s0[r / 2]), y = da_unpack(s1[r / 2]);
-        if (r < rows) {
-            if (live0) S[(size_t)r * p.dv] = x.x;
-            if (live1) S[(size_t)r * p.dv + 1] = y.x;
+            for (int r = 0; r < R / 2; ++r) {
+                const float2 x = da_unpack(dec[r]);
+                b[2 * r] = x.x;
+                b[2 * r + 1] = x.y;
+            }
         }
-        if (r + 1 < rows) {
-            if (live0) S[(size_t)(r + 1) * p.dv] = x.y;
-            if (live1) S[(size_t)(r + 1) * p.dv + 1] = y.y;
-        }
+    } else if (P == 1) {
+        store(p.state + head_off);
+    } else if (g == 0) {
+        load(p.seg_state + head_off);
+        for (int q = 1; q < P; ++q) advance(q);
+        store(p.state + head_off);
     }
 }
-static_assert(DA_U == 4, "four tokens of two columns are what three halvings leave one of");
-extern "C" __global__ void __launch_bounds__(DA_SCAN_THREADS) da_scan_64(const __grid_constant__ lb_decay_params2 p) { da_scan_body<4>(p); }
-extern "C" __global__ void __launch_bounds__(DA_SCAN_THREADS) da_scan_128(const __grid_constant__ lb_decay_params2 p) { da_scan_body<8>(p); }
-extern "C" __global__ void __launch_bounds__(DA_SCAN_THREADS) da_scan_256(const __grid_constant__ lb_decay_params2 p) { da_scan_body<16>(p); }
+#define DA_SCAN_KERNELS(dk, R, C)                                                                                                                                          \
+    extern "C" __global__ void __launch_bounds__(16 * DA_SLAB / C) da_scan_##dk(const __grid_constant__ lb_decay_params2 p) { da_scan_body<R, C, false>(p); } \
+    extern "C" __global__ void __launch_bounds__(16 * DA_SLAB / C) da_local_##dk(const __grid_constant__ lb_decay_params2 p) { da_scan_body<R, C, true>(p); }
+DA_SCAN_KERNELS(64, 4, 8)
+DA_SCAN_KERNELS(128, 8, 8)
+DA_SCAN_KERNELS(256, 16, 4)
 
 // cat[t, h dv + i] = o / rms_head(o) * head_w[i] [ * silu(gate) ].  grid (T, ceil(H / 4)), block 128: one warp per (token, head)
 extern "C" __global__ void __launch_bounds__(128) da_finish(const __grid_constant__ lb_decay_params2 p) {

@@ -370,9 +370,12 @@ typedef struct {
     float* a;
     float* o;             /* fp32 [T, H * dv] */
     void* cat;            /* prompt: bf16 / fp32 rows [T, cat_ld] */
+    float* seg_state;     /* prompt in segments: fp32 [segments, H, dk, dv] and ... */
+    float* seg_decay;     /* ... [segments, H, dk_p] */
     int32_t kind, ld, q_off, k_off, v_off, g_off; /* k_off: HGRN2 the gate's section; g_off < 0: no output gate */
     int32_t a1_off, rank; /* GLA: section of the low-rank pre-activation */
     int32_t H, dk, dv, dk_p, T, cat_ld, cat_f32;
+    int32_t seg;          /* prompt: tokens per segment, a multiple of 4 (T or more: one segment) */
     float q_scale, inv_tau, eps;
 } lb_decay_params2;
 
