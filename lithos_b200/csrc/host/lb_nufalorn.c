@@ -26,8 +26,9 @@ int lb_nufalorn_describe(lb_ctx* c, const lb_json* cfg, const lb_weight_source* 
     LB_TRY(need_int(c, cfg, "width", 1, 1 << 20, -1, &d->width));
     LB_TRY(need_int(c, cfg, "vocab", 1, 1 << 28, -1, &d->vocab));
     LB_TRY(need_num(c, lb_json_get(cfg, "norm"), "eps", -1, &d->eps));
-    LB_TRY(need_num(c, cfg, "residual_mult", -1, &d->residual_mult));
-    LB_TRY(need_num(c, cfg, "logit_softcap", -1, &d->logit_softcap));
+    d->residual_mult = 1.0;
+    if (lb_json_has(cfg, "residual_mult")) LB_TRY(need_num(c, cfg, "residual_mult", -1, &d->residual_mult));
+    if (lb_json_has(cfg, "logit_softcap")) LB_TRY(need_num(c, cfg, "logit_softcap", -1, &d->logit_softcap)); /* else 0: no cap */
     snprintf(d->embed, sizeof d->embed, "embed");
     snprintf(d->head, sizeof d->head, "head");
     snprintf(d->final_norm, sizeof d->final_norm, "final.norm");
@@ -51,10 +52,11 @@ int lb_nufalorn_describe(lb_ctx* c, const lb_json* cfg, const lb_weight_source* 
             const lb_json *rot = lb_json_get(m, "rot"), *mask = lb_json_get(m, "mask");
             L->mixer = LB_MIX_ATTENTION;
             L->v_norm = L->v_rot = L->sink = 1;
-            LB_TRY(need_int(c, m, "kv_heads", 1, L->heads, i, &L->kv_heads));
-            LB_TRY(need_int(c, rot, "dims", 0, L->dim, i, &L->rot_dims));
+            if (lb_json_has(m, "kv_heads")) LB_TRY(need_int(c, m, "kv_heads", 1, L->heads, i, &L->kv_heads));
+            L->rot_dims = L->dim;
+            if (lb_json_has(rot, "dims")) LB_TRY(need_int(c, rot, "dims", 0, L->dim, i, &L->rot_dims));
             LB_TRY(need_num(c, rot, "base", i, &L->rot_base));
-            LB_TRY(need_int(c, mask, "size", 1, 1 << 30, i, &L->block));
+            if (mask && mask->type == LB_JSON_OBJECT) LB_TRY(need_int(c, mask, "size", 1, 1 << 30, i, &L->block)); /* else 0: every earlier position */
             LB_TRY(need_num(c, m, "scale", i, &L->scale));
             if (lb_json_has(m, "kv_from")) LB_TRY(need_int(c, m, "kv_from", 0, i - 1, i, &L->kv_from));
             if (L->kv_from < 0) {
