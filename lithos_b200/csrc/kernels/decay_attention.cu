@@ -1,7 +1,7 @@
 // Linear attention whose state decays per key channel:  S <- diag(a_t) S + k_t v_t^T,  o_t = S^T q_t  per head, fp32 throughout.
 //   HGRN2: f = l + (1 - l) sigmoid(z + b), a = f, k = 1 - f, q = silu(zq)
 //   GLA:   a = sigmoid(W2 (W1 h) + b)^(1/tau), k = zk, q = dk^-1/2 zq
-// A column j of a head's state needs only v_j, so a CTA owns a 32-column slab of one head and holds it in registers: thread (column,
+// A column j of a head's state needs only v_j, so a CTA owns a slab of columns of one head and holds it in registers: thread (column,
 // row part) has R rows of its column (rows past dk stay zero), the sum over rows is local terms and a few shuffles.
 //   da_step_*   one token (decode): makes q, k, a of its head from the projections, state read and written once
 //   da_inputs   a prompt chunk's q, k, a
