@@ -128,7 +128,8 @@ static int load_cubin(lb_ctx* c, const char* dir, const char* file) {
 }
 
 static const char* const k_cubins[] = {"gemv.cubin", "chain.cubin", "batched.cubin", "batched_tc.cubin", "deltanet.cubin", "attention.cubin", "attention_mma.cubin", "small.cubin", "comm.cubin", "prefill.cubin",
-                                       "rows_gemv.cubin", "dense_gemm.cubin", "window_attention.cubin", "decay_attention.cubin"};
+                                       "rows_gemv.cubin", "dense_gemm.cubin", "window_attention.cubin", "decay_attention.cubin",
+                                       "latent_attention.cubin", "ssm.cubin"};
 
 LB_API int lb_init(int device, const char* kernel_dir, lb_ctx** out) { return lb_init_images(device, kernel_dir, NULL, out); }
 

@@ -104,6 +104,7 @@ int lb_driver_load(char* err, size_t errlen); /* LB_OK or LB_ERR_NO_DRIVER */
     X(attn_decode_split)              \
     X(attn_decode_mma)                \
     X(embed_bf16)                     \
+    X(embed_bigram)                   \
     X(argmax_f32)                     \
     X(topk_sample_f32)                \
     X(rmsnorm_f32)                    \
@@ -123,6 +124,7 @@ int lb_driver_load(char* err, size_t errlen); /* LB_OK or LB_ERR_NO_DRIVER */
     X(gemm_bf16_tc)                   \
     X(gemm_f32_simt)                  \
     X(norm_rows2)                     \
+    X(moe_plan)                       \
     X(wattn_rows_b2n2)                \
     X(wattn_rows_b4n2)                \
     X(wattn_rows_b8n2)                \
@@ -151,6 +153,26 @@ int lb_driver_load(char* err, size_t errlen); /* LB_OK or LB_ERR_NO_DRIVER */
     X(da_scan_128)                    \
     X(da_scan_256)                    \
     X(da_finish)                      \
+    X(lat_query_bf16)                 \
+    X(lat_query_f32)                  \
+    X(lat_rows_128)                   \
+    X(lat_rows_256)                   \
+    X(lat_rows_512)                   \
+    X(lat_rows_f32)                   \
+    X(lat_out_bf16)                   \
+    X(lat_out_f32)                    \
+    X(lat_prepare)                    \
+    X(ssm_step_64)                    \
+    X(ssm_step_128)                   \
+    X(ssm_step_256)                   \
+    X(ssm_conv)                       \
+    X(ssm_chunk_64)                   \
+    X(ssm_chunk_128)                  \
+    X(ssm_chunk_256)                  \
+    X(ssm_scan_f32_64)                \
+    X(ssm_scan_f32_128)               \
+    X(ssm_scan_f32_256)               \
+    X(ssm_finish)                     \
     X(l2_flush)
 
 enum {

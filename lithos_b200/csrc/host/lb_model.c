@@ -27,6 +27,7 @@ int lb_model_alloc_common(lb_model* m) {
     LB_TRY(lb_dalloc(m, &m->d_token, 16));
     LB_TRY(lb_dalloc(m, &m->d_pos, 16));
     LB_TRY(lb_dalloc(m, &m->d_next, 16));
+    LB_TRY(lb_dalloc(m, &m->d_tokens, (size_t)m->cfg.max_ctx * 4));
     LB_TRY(lb_dalloc(m, &m->cand_val, (size_t)m->arch->head_ctas(m) * 4));
     LB_TRY(lb_dalloc(m, &m->cand_idx, (size_t)m->arch->head_ctas(m) * 4));
     LB_CU(m->c, lb_drv.MemHostAlloc((void**)&m->h_next, 64, 0));
@@ -83,11 +84,19 @@ int lb_model_launch_sampler(lb_model* m) {
     return LB_OK;
 }
 
+/* n tokens' embeddings with the pair embedding: one token (given, its position in device memory), or the tokens already in m->d_tokens from pos0 on */
+int lb_model_embed_bigram(lb_model* m, CUdeviceptr token, CUdeviceptr pos_ptr, int pos0, int n, CUdeviceptr out) {
+    const int H = m->cfg.hidden;
+    void* params[] = {&m->embed, &m->bigram, &token, &pos_ptr, &pos0, &m->d_tokens, &out, (void*)&H, &m->bigram_buckets, &m->bigram_mul_prev, &m->bigram_mul_cur};
+    return lb_launch(m->c, LBK_embed_bigram, (unsigned)((H + 1023) / 1024), (unsigned)n, 1, 256, 0, params, 1);
+}
+
 static int issue_step(lb_model* m) {
     lb_ctx* c = m->c;
     const int H = m->cfg.hidden;
     uint64_t launches0 = c->launches;
-    {
+    if (m->bigram) LB_TRY(lb_model_embed_bigram(m, m->d_token, m->d_pos, 0, 1, m->X));
+    else {
         void* params[] = {&m->embed, &m->d_token, &m->X, (void*)&H};
         LB_TRY(lb_launch(c, LBK_embed_bf16, (unsigned)((H + 1023) / 1024), 1, 1, 256, 0, params, 1));
     }
@@ -220,7 +229,7 @@ LB_API void lb_model_destroy(lb_model* m) {
         lb_drv.StreamSynchronize(c->stream);
         if (m->graph) lb_graph_destroy(c, m->graph);
         if (m->arch) m->arch->destroy(m);
-        CUdeviceptr g[] = {m->embed, m->lm_head, m->final_norm, m->X, m->logits, m->d_token, m->d_pos, m->d_next, m->cand_val, m->cand_idx};
+        CUdeviceptr g[] = {m->embed, m->lm_head, m->final_norm, m->X, m->logits, m->d_token, m->d_pos, m->d_next, m->cand_val, m->cand_idx, m->bigram, m->d_tokens};
         for (size_t i = 0; i < sizeof g / sizeof g[0]; i++) if (g[i]) lb_drv.MemFree(g[i]);
         lb_prefill_ws_free(m);
         if (m->h_next) lb_drv.MemFreeHost(m->h_next);

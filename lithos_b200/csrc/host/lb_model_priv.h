@@ -34,11 +34,11 @@ typedef struct {
 } layer_t;
 
 /* the activations of one prompt chunk: an architecture names the buffers it uses; the residual stream comes first */
-#define LB_PF_MAX_BUFS 16
+#define LB_PF_MAX_BUFS 24
 typedef union {
     CUdeviceptr b[LB_PF_MAX_BUFS];
     struct { CUdeviceptr X, xn16, proj, q, k, v, g, beta, mix, mix16, y, gu, act16; } hy; /* lb_hybrid.c */
-    struct { CUdeviceptr X, h1, h2, proj, cat, q, k, a, o, seg_state, seg_decay; } st;                        /* lb_stack.c */
+    struct { CUdeviceptr X, h1, h2, proj, cat, q, k, a, o, seg_state, seg_decay, lq, kx, vx, lat_q, lat_part, xbc, dt, act, xg, ye, plan; } st; /* lb_stack.c */
 } pf_set;
 
 /* What an architecture supplies.  The runtime owns embedding, order of calls, positions, graph capture, chunking and
@@ -71,6 +71,9 @@ struct lb_model {
     int C_s;                      /* conv channels on this shard: 2*HK*128 + HV*128 */
     layer_t* L;
     CUdeviceptr embed, lm_head, final_norm;
+    CUdeviceptr bigram; /* embedding of (previous, current) token pairs, added to the token's own; 0: none */
+    int bigram_buckets, bigram_mul_prev, bigram_mul_cur;
+    CUdeviceptr d_tokens; /* the sequence's token ids by position [max_ctx] (decode steps enter theirs only where the embedding needs them) */
     int globals_loaded;
     /* activations */
     CUdeviceptr X, xn, in_out, mix_out, mlp_m, logits, d_token, d_pos, d_next, cand_val, cand_idx;
@@ -96,6 +99,7 @@ typedef struct lb_prefill_ws lb_prefill_ws;
 
 int lb_model_is_fa(const lb_model_cfg* c, int l);
 int lb_model_launch_sampler(lb_model* m);
+int lb_model_embed_bigram(lb_model* m, CUdeviceptr token, CUdeviceptr pos_ptr, int pos0, int n, CUdeviceptr out);
 int lb_model_alloc_common(lb_model* m); /* the buffers every architecture uses; cfg and vocab_s must be set */
 pf_set* lb_prefill_set(lb_model* m, int s);    /* buffers of prompt stream s (after a prompt pass) */
 int lb_dalloc(lb_model* m, CUdeviceptr* p, size_t bytes);

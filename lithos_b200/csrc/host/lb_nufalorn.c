@@ -6,29 +6,17 @@
 #include "../kernels/params.h"
 #include <math.h>
 
-static int need_int(lb_ctx* c, const lb_json* j, const char* key, int lo, int hi, int layer, int* out) {
-    const double v = lb_json_num(j, key, NAN);
-    if (!(v >= lo && v <= hi) || v != floor(v)) return lb_fail(c, LB_ERR_INVALID, "config: layer %d: '%s' is missing or not an integer in [%d, %d]", layer, key, lo, hi);
-    *out = (int)v;
-    return LB_OK;
-}
-static int need_num(lb_ctx* c, const lb_json* j, const char* key, int layer, double* out) {
-    *out = lb_json_num(j, key, NAN);
-    if (!isfinite(*out)) return lb_fail(c, LB_ERR_INVALID, "config: layer %d: '%s' is missing or not a number", layer, key);
-    return LB_OK;
-}
-
 int lb_nufalorn_describe(lb_ctx* c, const lb_json* cfg, const lb_weight_source* src, lb_stack_desc* d) {
     const lb_json* layers = lb_json_get(cfg, "layers");
     if (!layers || layers->type != LB_JSON_ARRAY || layers->n < 1) return lb_fail(c, LB_ERR_INVALID, "config: 'layers' is not a list of layers");
     d->design = "Nufalorn";
     d->n_layers = layers->n;
-    LB_TRY(need_int(c, cfg, "width", 1, 1 << 20, -1, &d->width));
-    LB_TRY(need_int(c, cfg, "vocab", 1, 1 << 28, -1, &d->vocab));
-    LB_TRY(need_num(c, lb_json_get(cfg, "norm"), "eps", -1, &d->eps));
+    LB_TRY(lb_cfg_int(c, cfg, "width", 1, 1 << 20, -1, &d->width));
+    LB_TRY(lb_cfg_int(c, cfg, "vocab", 1, 1 << 28, -1, &d->vocab));
+    LB_TRY(lb_cfg_num(c, lb_json_get(cfg, "norm"), "eps", -1, &d->eps));
     d->residual_mult = 1.0;
-    if (lb_json_has(cfg, "residual_mult")) LB_TRY(need_num(c, cfg, "residual_mult", -1, &d->residual_mult));
-    if (lb_json_has(cfg, "logit_softcap")) LB_TRY(need_num(c, cfg, "logit_softcap", -1, &d->logit_softcap)); /* else 0: no cap */
+    if (lb_json_has(cfg, "residual_mult")) LB_TRY(lb_cfg_num(c, cfg, "residual_mult", -1, &d->residual_mult));
+    if (lb_json_has(cfg, "logit_softcap")) LB_TRY(lb_cfg_num(c, cfg, "logit_softcap", -1, &d->logit_softcap)); /* else 0: no cap */
     snprintf(d->embed, sizeof d->embed, "embed");
     snprintf(d->head, sizeof d->head, "head");
     snprintf(d->final_norm, sizeof d->final_norm, "final.norm");
@@ -41,9 +29,9 @@ int lb_nufalorn_describe(lb_ctx* c, const lb_json* cfg, const lb_weight_source* 
 #define NAME(role, ...) snprintf(L->tensor[role], sizeof L->tensor[role], __VA_ARGS__)
         if (!type || !m) return lb_fail(c, LB_ERR_INVALID, "config: layer %d has no type or no mixer", i);
         L->kv_from = -1;
-        LB_TRY(need_int(c, m, "heads", 1, 65536, i, &L->heads));
-        LB_TRY(need_int(c, m, "dim", 1, 65536, i, &L->dim));
-        LB_TRY(need_int(c, m, "vdim", 1, 65536, i, &L->vdim));
+        LB_TRY(lb_cfg_int(c, m, "heads", 1, 65536, i, &L->heads));
+        LB_TRY(lb_cfg_int(c, m, "dim", 1, 65536, i, &L->dim));
+        LB_TRY(lb_cfg_int(c, m, "vdim", 1, 65536, i, &L->vdim));
         L->kv_heads = L->heads;
         NAME(LB_T_NORM1, "l%d.norm1", i);
         NAME(LB_T_Q, "l%d.mix.q", i);
@@ -52,13 +40,13 @@ int lb_nufalorn_describe(lb_ctx* c, const lb_json* cfg, const lb_weight_source* 
             const lb_json *rot = lb_json_get(m, "rot"), *mask = lb_json_get(m, "mask");
             L->mixer = LB_MIX_ATTENTION;
             L->v_norm = L->v_rot = L->sink = 1;
-            if (lb_json_has(m, "kv_heads")) LB_TRY(need_int(c, m, "kv_heads", 1, L->heads, i, &L->kv_heads));
+            if (lb_json_has(m, "kv_heads")) LB_TRY(lb_cfg_int(c, m, "kv_heads", 1, L->heads, i, &L->kv_heads));
             L->rot_dims = L->dim;
-            if (lb_json_has(rot, "dims")) LB_TRY(need_int(c, rot, "dims", 0, L->dim, i, &L->rot_dims));
-            LB_TRY(need_num(c, rot, "base", i, &L->rot_base));
-            if (mask && mask->type == LB_JSON_OBJECT) LB_TRY(need_int(c, mask, "size", 1, 1 << 30, i, &L->block)); /* else 0: every earlier position */
-            LB_TRY(need_num(c, m, "scale", i, &L->scale));
-            if (lb_json_has(m, "kv_from")) LB_TRY(need_int(c, m, "kv_from", 0, i - 1, i, &L->kv_from));
+            if (lb_json_has(rot, "dims")) LB_TRY(lb_cfg_int(c, rot, "dims", 0, L->dim, i, &L->rot_dims));
+            LB_TRY(lb_cfg_num(c, rot, "base", i, &L->rot_base));
+            if (mask && mask->type == LB_JSON_OBJECT) LB_TRY(lb_cfg_int(c, mask, "size", 1, 1 << 30, i, &L->block)); /* else 0: every earlier position */
+            LB_TRY(lb_cfg_num(c, m, "scale", i, &L->scale));
+            if (lb_json_has(m, "kv_from")) LB_TRY(lb_cfg_int(c, m, "kv_from", 0, i - 1, i, &L->kv_from));
             if (L->kv_from < 0) {
                 NAME(LB_T_K, "l%d.mix.k", i);
                 NAME(LB_T_V, "l%d.mix.v", i);
@@ -74,7 +62,7 @@ int lb_nufalorn_describe(lb_ctx* c, const lb_json* cfg, const lb_weight_source* 
                 NAME(LB_T_LOWER, "l%d.mix.lower", i);
             } else {
                 L->decay = LB_DA_GLA;
-                LB_TRY(need_num(c, m, "tau", i, &L->tau));
+                LB_TRY(lb_cfg_num(c, m, "tau", i, &L->tau));
                 NAME(LB_T_K, "l%d.mix.k", i);
                 NAME(LB_T_G, "l%d.mix.g", i);
                 NAME(LB_T_A1, "l%d.mix.a1", i);
@@ -91,7 +79,7 @@ int lb_nufalorn_describe(lb_ctx* c, const lb_json* cfg, const lb_weight_source* 
         if (f && f->type == LB_JSON_OBJECT) {
             const char* kind = lb_json_str(f, "kind");
             if (kind && strcmp(kind, "dense")) return lb_fail(c, LB_ERR_INVALID, "config: layer %d: unknown feed-forward '%s'", i, kind);
-            LB_TRY(need_int(c, f, "ff", 1, 1 << 24, i, &L->ff));
+            LB_TRY(lb_cfg_int(c, f, "ff", 1, 1 << 24, i, &L->ff));
             NAME(LB_T_NORM2, "l%d.norm2", i);
             NAME(LB_T_FF_GATE, "l%d.mlp.gate", i);
             NAME(LB_T_FF_UP, "l%d.mlp.up", i);

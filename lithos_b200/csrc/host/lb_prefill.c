@@ -14,7 +14,6 @@
 
 struct lb_prefill_ws {
     pf_set set[LB_PF_MAX_STREAMS]; /* one per stream */
-    CUdeviceptr tokens;            /* the whole prompt's token ids [max_ctx] */
     CUdeviceptr rows, row_logits;  /* residual rows whose logits are wanted, and those logits; grown on demand */
     int rows_cap;
     CUstream stream[LB_PF_MAX_STREAMS];
@@ -32,7 +31,6 @@ static int ws_fill(lb_model* m) {
     const lb_model_cfg* c = &m->cfg;
     size_t bytes[LB_PF_MAX_BUFS] = {0};
     m->arch->pf_sizes(m, bytes);
-    LB_TRY(lb_dalloc(m, &ws->tokens, (size_t)c->max_ctx * 4));
     for (int s = 0; s < m->arch->pf_streams; s++) {
         for (int i = 0; i < LB_PF_MAX_BUFS; i++) {
             if (!bytes[i]) continue;
@@ -88,7 +86,6 @@ void lb_prefill_ws_free(lb_model* m) {
         if (ws->stream[s]) lb_drv.StreamDestroy(ws->stream[s]);
     }
     if (ws->fork) lb_drv.EventDestroy(ws->fork);
-    if (ws->tokens) lb_drv.MemFree(ws->tokens);
     if (ws->rows) lb_drv.MemFree(ws->rows);
     if (ws->row_logits) lb_drv.MemFree(ws->row_logits);
     free(ws);
@@ -103,7 +100,7 @@ static int run_chunks(lb_model* m, const int* tokens, int n, int pos0, const int
     lb_prefill_ws* ws = m->ws;
     const int H = cfg->hidden, CH = m->pf_chunk, NS = m->arch->pf_streams;
     CUstream main_stream = c->stream;
-    LB_CU(c, lb_drv.MemcpyHtoDAsync(ws->tokens, tokens, (size_t)n * 4, main_stream));
+    LB_CU(c, lb_drv.MemcpyHtoDAsync(m->d_tokens + (size_t)pos0 * 4, tokens, (size_t)n * 4, main_stream));
     LB_CU(c, lb_drv.StreamSynchronize(main_stream)); /* the caller's token array may be pageable */
     /* the chunk streams start behind what the caller's stream holds so far (an earlier decode step, the token copy) */
     LB_CU(c, lb_drv.EventRecord(ws->fork, main_stream));
@@ -113,9 +110,9 @@ static int run_chunks(lb_model* m, const int* tokens, int n, int pos0, const int
         const int T = n - c0 < CH ? n - c0 : CH, s = chunk % NS, prev = (chunk + NS - 1) % NS;
         pf_set* w = &ws->set[s];
         c->stream = ws->stream[s]; /* every launch below goes to this chunk's stream */
-        CUdeviceptr toks = ws->tokens + (size_t)c0 * 4;
+        CUdeviceptr toks = m->d_tokens + (size_t)(pos0 + c0) * 4;
         void* params[] = {&m->embed, &toks, &w->b[0], (void*)&H};
-        st = lb_launch(c, LBK_pf_embed, (unsigned)T, 1, 1, 256, 0, params, 1);
+        st = m->bigram ? lb_model_embed_bigram(m, 0, 0, pos0 + c0, T, w->b[0]) : lb_launch(c, LBK_pf_embed, (unsigned)T, 1, 1, 256, 0, params, 1);
         for (int l = 0; l < cfg->n_layers && st == LB_OK; l++) {
             /* layer l's state, ring and cache rows come from the previous chunk's layer l (on the stream before this one) */
             if (chunk > 0 && lb_drv.StreamWaitEvent(c->stream, ws->layer_done[prev][l], 0) != CUDA_SUCCESS) st = LB_ERR_CUDA;

@@ -32,6 +32,10 @@ static int open_nufalorn(lb_ctx* c, const lb_json* cfg, const char* dir, int max
     return open_stack(c, cfg, dir, max_ctx, dtype, seed, out, lb_nufalorn_describe);
 }
 
+static int open_vobunex(lb_ctx* c, const lb_json* cfg, const char* dir, int max_ctx, int dtype, uint64_t seed, lb_model** out) {
+    return open_stack(c, cfg, dir, max_ctx, dtype, seed, out, lb_vobunex_describe);
+}
+
 /* the int4 hybrid: config.json with the fields of lb_model_cfg; weights through weight_index.bin, which is written over the
  * directory's safetensors files when it is not there yet */
 static int open_hybrid(lb_ctx* c, const lb_json* cfg, const char* dir, int max_ctx, int dtype, uint64_t seed, lb_model** out) {
@@ -60,6 +64,7 @@ static int open_hybrid(lb_ctx* c, const lb_json* cfg, const char* dir, int max_c
 
 static const struct { const char* architecture; open_fn open; const char* images; } k_registry[] = {
     {"Nufalorn", open_nufalorn, "small prefill rows_gemv dense_gemm window_attention decay_attention"},
+    {"Vobunex", open_vobunex, "small prefill rows_gemv dense_gemm window_attention latent_attention ssm"},
     {"Qwen3.5-hybrid", open_hybrid, "gemv chain batched batched_tc deltanet attention attention_mma small comm prefill"},
 };
 

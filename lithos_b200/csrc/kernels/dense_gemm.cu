@@ -6,6 +6,7 @@
 // lane issues products, four warps read accumulators (lane = weight row, column = token) and finish them.  Two accumulators, so the
 // epilogue of a tile runs beside the products of the next.  Weight rows are the lanes, so 32 neighbouring outputs of a token are one
 // coalesced store and a (gate, up) pair sits in neighbouring lanes.  Every wait is bounded and reports through the status word.
+// With experts the chunk's (token, expert) assignments come sorted by expert (moe_plan) and every token tile belongs to one of them.
 // gemm_f32_simt: the same products in fp32 throughout (fp32 activations, weights exact in fp32, fp32 fused multiply-adds).
 #include "tcgen05.cuh"
 #include "params.h"
@@ -20,6 +21,33 @@ __device__ __forceinline__ void dg_tma(uint32_t dst_smem, const void* tmap, int 
                  : "memory");
 }
 
+// tile t of a launch: product m, weight rows from row (row in its matrix: n0), tokens tok .. end - 1.  With experts a token tile is an entry
+// of the plan and the expert's rows are rows of the stack.
+struct dg_tile { int m, row, n0, tok, end; };
+__device__ __forceinline__ dg_tile dg_find(const lb_dgemm_params& p, int t) {
+    dg_tile d;
+    if (p.plan_tiles) {
+        const int tt = t / p.tiles[0];
+        const int4 e = __ldg(reinterpret_cast<const int4*>(p.plan_tiles) + tt);
+        d.m = 0;
+        d.n0 = (t - tt * p.tiles[0]) * LB_DG_ROWS;
+        d.row = e.x * p.expert_rows + d.n0;
+        d.tok = e.y;
+        d.end = e.z;
+    } else {
+        const int rt = t / p.t_tiles, tt = t - rt * p.t_tiles;
+        d.m = rt >= p.tiles[0];
+        d.row = d.n0 = (d.m ? rt - p.tiles[0] : rt) * LB_DG_ROWS;
+        d.tok = tt * p.NT;
+        d.end = p.T;
+    }
+    return d;
+}
+__device__ __forceinline__ float dg_clamp_glu(float gate, float up, float limit, float alpha) {
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+    return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+}
+
 extern "C" __global__ void __launch_bounds__(LB_DG_THREADS, 1) gemm_bf16_tc(const __grid_constant__ lb_dgemm_params p) {
     extern __shared__ __align__(1024) unsigned char dg_sm[];
     __shared__ __align__(8) uint64_t bar_full[LB_DG_MAX_STAGES], bar_empty[LB_DG_MAX_STAGES], bar_acc[2], bar_free[2];
@@ -27,7 +55,7 @@ extern "C" __global__ void __launch_bounds__(LB_DG_THREADS, 1) gemm_bf16_tc(cons
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int S = p.stages, NT = p.NT;
     const uint32_t a_bytes = LB_DG_ROWS * LB_DG_KB * 2, b_bytes = (uint32_t)NT * LB_DG_KB * 2, stage_bytes = a_bytes + b_bytes;
-    const int ksteps = p.K / LB_DG_KB, n_tiles = (p.tiles[0] + p.tiles[1]) * p.t_tiles;
+    const int ksteps = p.K / LB_DG_KB;
     if (tid == 0) {
         for (int s = 0; s < S; ++s) {
             mbar_init(&bar_full[s], 1);
@@ -45,6 +73,7 @@ extern "C" __global__ void __launch_bounds__(LB_DG_THREADS, 1) gemm_bf16_tc(cons
     tc_fence_after();
     const uint32_t tmem = tmem_slot;
     pdl_wait();
+    const int n_tiles = p.plan_tiles ? p.plan_n[0] * p.tiles[0] : (p.tiles[0] + p.tiles[1]) * p.t_tiles;
 
     if (warp == 0 && lane == 0) {
         // ---------------- operands ----------------
@@ -52,8 +81,7 @@ extern "C" __global__ void __launch_bounds__(LB_DG_THREADS, 1) gemm_bf16_tc(cons
         uint32_t ph = 0;
         bool ok = true;
         for (int tile = blockIdx.x; tile < n_tiles && ok; tile += gridDim.x) {
-            const int rt = tile / p.t_tiles, tt = tile - rt * p.t_tiles, m = rt >= p.tiles[0];
-            const int row = (m ? rt - p.tiles[0] : rt) * LB_DG_ROWS, tok = tt * NT;
+            const dg_tile d = dg_find(p, tile);
             for (int k = 0; k < ksteps; ++k) {
                 if (issued >= S && !tc_wait(&bar_empty[s], ph ^ 1u)) {
                     ok = false;
@@ -62,14 +90,14 @@ extern "C" __global__ void __launch_bounds__(LB_DG_THREADS, 1) gemm_bf16_tc(cons
                 }
                 mbar_arrive_expect_tx(&bar_full[s], stage_bytes);
                 const uint32_t dst = smem_u32(dg_sm) + (uint32_t)s * stage_bytes;
-                dg_tma(dst, p.tmap_w[m], k * LB_DG_KB, row, &bar_full[s]);
-                dg_tma(dst + a_bytes, p.tmap_x[m], k * LB_DG_KB, tok, &bar_full[s]);
+                dg_tma(dst, p.tmap_w[d.m], k * LB_DG_KB, d.row, &bar_full[s]);
+                dg_tma(dst + a_bytes, p.tmap_x[d.m], k * LB_DG_KB, d.tok, &bar_full[s]);
                 ++issued;
                 if (++s == S) { s = 0; ph ^= 1u; }
             }
         }
         if (!ok) // nothing may still be on its way into this CTA's shared memory when it ends
-            for (int d = 0; d < S && d < issued; ++d) {
+            for (int i = 0; i < S && i < issued; ++i) {
                 if (--s < 0) { s = S - 1; ph ^= 1u; }
                 tc_wait(&bar_full[s], ph);
             }
@@ -111,25 +139,36 @@ extern "C" __global__ void __launch_bounds__(LB_DG_THREADS, 1) gemm_bf16_tc(cons
         int it = 0;
         for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x, ++it) {
             const int b = it & 1;
-            const int rt = tile / p.t_tiles, tt = tile - rt * p.t_tiles, m = rt >= p.tiles[0];
-            const int n = (m ? rt - p.tiles[0] : rt) * LB_DG_ROWS + quad * 32 + lane, t0 = tt * NT;
+            const dg_tile d = dg_find(p, tile);
+            const int m = d.m, n = d.n0 + quad * 32 + lane, t0 = d.tok;
             const bool got = tc_wait(&bar_acc[b], (uint32_t)(it >> 1) & 1u);
             if (!__all_sync(0xffffffffu, got)) {
                 if (lane == 0 && p.status) atomicExch(p.status, DG_FAIL_ACC);
                 break;
             }
             tc_fence_after();
-            const int mode = p.y_mode[m], ld = p.ld_y[m], n_t = min(NT, p.T - t0);
+            const int mode = p.y_mode[m], ld = p.ld_y[m], n_t = min(NT, d.end - t0);
             const bool live = n < p.rows[m];
+            const int hn = mode == LB_DY_HEADS ? n / p.head[m] : 0, hcol = hn * p.head_p[m] + (n - hn * p.head[m]);
             for (int c = 0; c < n_t; c += 16) {
                 uint32_t r[16];
                 tmem_ld16(tmem + ((uint32_t)(32 * quad) << 16) + (uint32_t)(b * NT + c), r);
                 tmem_ld_wait();
-                if (mode == LB_DY_RELU_GLU) {
+                if (mode == LB_DY_HEADS || mode == LB_DY_RELU2) {
+#pragma unroll
+                    for (int j = 0; j < 16; ++j) {
+                        if (!live || c + j >= n_t) continue;
+                        const float v = __uint_as_float(r[j]), v0 = fmaxf(v, 0.f);
+                        const size_t o = (size_t)(t0 + c + j) * ld + (mode == LB_DY_HEADS ? hcol : n);
+                        if (mode == LB_DY_RELU2 && p.y_f32[m]) reinterpret_cast<float*>(p.y[m])[o] = v0 * v0;
+                        else reinterpret_cast<__nv_bfloat16*>(p.y[m])[o] = __float2bfloat16_rn(mode == LB_DY_HEADS ? v : v0 * v0);
+                    }
+                } else if (mode == LB_DY_RELU_GLU || mode == LB_DY_CLAMP_GLU) {
                     const bool st = live && !(lane & 1);
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
-                        const float up = __uint_as_float(__shfl_xor_sync(0xffffffffu, r[j], 1)), v = fmaxf(__uint_as_float(r[j]), 0.f) * up;
+                        const float ga = __uint_as_float(r[j]), up = __uint_as_float(__shfl_xor_sync(0xffffffffu, r[j], 1));
+                        const float v = mode == LB_DY_RELU_GLU ? fmaxf(ga, 0.f) * up : dg_clamp_glu(ga, up, p.limit, p.alpha);
                         if (st && c + j < n_t) {
                             const size_t o = (size_t)(t0 + c + j) * ld + (n >> 1);
                             if (p.y_f32[m]) reinterpret_cast<float*>(p.y[m])[o] = v;
@@ -175,8 +214,16 @@ extern "C" __global__ void __launch_bounds__(256) gemm_f32_simt(const __grid_con
     pdl_wait();
     const int tid = threadIdx.x, tn = tid & 15, tt = tid >> 4;
     const int nt0 = (p.rows[0] + SG_TN - 1) / SG_TN, m = (int)blockIdx.x >= nt0;
-    const int row0 = ((int)blockIdx.x - (m ? nt0 : 0)) * SG_TN, t0 = blockIdx.y * SG_TT;
+    const int row0 = ((int)blockIdx.x - (m ? nt0 : 0)) * SG_TN;
+    int t0 = blockIdx.y * SG_TT, end = p.T;
     const uint16_t* W = p.w[m];
+    if (p.plan_tiles) {
+        if ((int)blockIdx.y >= p.plan_n[0]) return;
+        const int4 e = reinterpret_cast<const int4*>(p.plan_tiles)[blockIdx.y];
+        W += (size_t)e.x * p.expert_rows * p.K;
+        t0 = e.y;
+        end = e.z;
+    }
     const float* X = reinterpret_cast<const float*>(p.x[m]);
     float acc[4][4] = {};
     const int lr = tid >> 2, lk = (tid & 3) * 4; // load: row / token of the tile, 4 k
@@ -184,7 +231,7 @@ extern "C" __global__ void __launch_bounds__(256) gemm_f32_simt(const __grid_con
         uint2 w = make_uint2(0u, 0u);
         float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
         if (row0 + lr < p.rows[m]) w = *reinterpret_cast<const uint2*>(W + (size_t)(row0 + lr) * p.K + k0 + lk);
-        if (t0 + lr < p.T) x = *reinterpret_cast<const float4*>(X + (size_t)(t0 + lr) * p.ld_x + k0 + lk);
+        if (t0 + lr < end) x = *reinterpret_cast<const float4*>(X + (size_t)(t0 + lr) * p.ld_x + k0 + lk);
         __syncthreads();
         ws[lk][lr] = __uint_as_float(w.x << 16);
         ws[lk + 1][lr] = __uint_as_float(w.x & 0xffff0000u);
@@ -210,7 +257,7 @@ extern "C" __global__ void __launch_bounds__(256) gemm_f32_simt(const __grid_con
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
         const int t = t0 + tt * 4 + j;
-        if (t >= p.T) continue;
+        if (t >= end) continue;
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
             const int n = row0 + tn * 4 + i;
@@ -222,39 +269,100 @@ extern "C" __global__ void __launch_bounds__(256) gemm_f32_simt(const __grid_con
                 v = fmaxf(v, 0.f) * acc[i | 1][j];
                 if (p.y_f32[m]) y[n >> 1] = v;
                 else reinterpret_cast<__nv_bfloat16*>(p.y[m])[(size_t)t * ld + (n >> 1)] = __float2bfloat16_rn(v);
-            } else if (mode == LB_DY_RESIDUAL) y[n] = fmaf(p.mult, v, y[n]);
+            } else if (mode == LB_DY_CLAMP_GLU) {
+                if (!(i & 1)) y[n >> 1] = dg_clamp_glu(v, acc[i | 1][j], p.limit, p.alpha);
+            } else if (mode == LB_DY_RELU2) y[n] = fmaxf(v, 0.f) * fmaxf(v, 0.f);
+            else if (mode == LB_DY_RESIDUAL) y[n] = fmaf(p.mult, v, y[n]);
             else y[n] = mode == LB_DY_SOFTCAP && p.cap > 0.f ? p.cap * tanhf(v / p.cap) : v;
         }
     }
 }
 
-// h_i[t] = x[t] / sqrt(mean x^2 + eps) * (1 + w_i), columns width..ld are zero.  grid T, block 256.  Rows of whole quads up to
-// 4 NR_Q x 256 columns stay in registers between the two passes.
+// norm of a chunk's rows (lb_norm2_params), columns width..ld are zero.  grid T, block 256.  Rows of whole quads up to
+// 4 NR_Q x 256 columns stay in registers between the passes.
 #define NR_Q 8
-extern "C" __global__ void __launch_bounds__(256) norm_rows2(const __grid_constant__ lb_norm2_params p) {
+__device__ __forceinline__ float4 nr_quad(const uint16_t* w, int i) {
+    const uint2 u = __ldg(reinterpret_cast<const uint2*>(w + i));
+    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
+}
+__device__ __forceinline__ float nr_added(const lb_norm2_params& p, int t, int i) { // sum of the token's rows of y, in the order of its parts
+    float s = 0.f;
+    for (int k = 0; k < p.y_top; ++k) {
+        const size_t o = (size_t)p.y_place[(size_t)t * p.y_top + k] * p.ld_y + i;
+        s += p.f32 ? reinterpret_cast<const float*>(p.y)[o] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.y)[o]);
+    }
+    return s;
+}
+__device__ __forceinline__ void nr_store4(const lb_norm2_params& p, void* h, size_t o, float4 r) {
+    if (p.f32) *reinterpret_cast<float4*>(reinterpret_cast<float*>(h) + o) = r;
+    else {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(r.x, r.y), hi = __floats2bfloat162_rn(r.z, r.w);
+        *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(h) + o) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+    }
+}
+__device__ __forceinline__ void nr_store1(const lb_norm2_params& p, void* h, size_t o, float r) {
+    if (p.f32) reinterpret_cast<float*>(h)[o] = r;
+    else reinterpret_cast<__nv_bfloat16*>(h)[o] = __float2bfloat16_rn(r);
+}
+extern "C" __global__ void __launch_bounds__(256, 4) norm_rows2(const __grid_constant__ lb_norm2_params p) {
     __shared__ float red[40];
-    const int t = threadIdx.x;
-    const bool quads = (p.width & 3) == 0 && p.width <= 4 * NR_Q * 256;
+    const int t = threadIdx.x, tok = blockIdx.x;
+    const bool quads = (p.width & 3) == 0 && (p.ld_x & 3) == 0 && (p.ld_y & 3) == 0 && p.width <= 4 * NR_Q * 256;
+    const float one = p.norm == LB_NORM_RMS_1P ? 1.0f : 0.0f;
     pdl_wait();
-    const float* x = p.x + (size_t)blockIdx.x * p.width;
-    const size_t o = (size_t)blockIdx.x * p.ld;
+    float* x = p.x + (size_t)tok * p.ld_x;
     float4 v[NR_Q];
-    float ss = 0.f;
+    float mean = 0.f, ss = 0.f;
     if (quads) {
 #pragma unroll
         for (int u = 0; u < NR_Q; ++u) {
             const int i = 4 * (t + 256 * u);
             v[u] = i < p.width ? *reinterpret_cast<const float4*>(x + i) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
+        if (p.y) {
+#pragma unroll
+            for (int u = 0; u < NR_Q; ++u) {
+                const int i = 4 * (t + 256 * u);
+                if (i >= p.width) continue;
+                float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+                for (int k = 0; k < p.y_top; ++k) {
+                    const size_t o = (size_t)p.y_place[(size_t)tok * p.y_top + k] * p.ld_y + i;
+                    const float4 a = p.f32 ? *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.y) + o) : nr_quad(reinterpret_cast<const uint16_t*>(p.y) + o, 0);
+                    s.x += a.x; s.y += a.y; s.z += a.z; s.w += a.w;
+                }
+                v[u].x = fmaf(p.y_mult, s.x, v[u].x); v[u].y = fmaf(p.y_mult, s.y, v[u].y);
+                v[u].z = fmaf(p.y_mult, s.z, v[u].z); v[u].w = fmaf(p.y_mult, s.w, v[u].w);
+                *reinterpret_cast<float4*>(x + i) = v[u];
+            }
+        }
+        if (p.norm == LB_NORM_LAYER) {
+#pragma unroll
+            for (int u = 0; u < NR_Q; ++u) mean += (v[u].x + v[u].y) + (v[u].z + v[u].w);
+            mean = block_sum(mean, red) / (float)p.width;
+#pragma unroll
+            for (int u = 0; u < NR_Q; ++u)
+                if (4 * (t + 256 * u) < p.width) { v[u].x -= mean; v[u].y -= mean; v[u].z -= mean; v[u].w -= mean; }
+        }
 #pragma unroll
         for (int u = 0; u < NR_Q; ++u) ss += (v[u].x * v[u].x + v[u].y * v[u].y) + (v[u].z * v[u].z + v[u].w * v[u].w);
     } else {
+        if (p.y)
+            for (int i = t; i < p.width; i += 256) x[i] = fmaf(p.y_mult, nr_added(p, tok, i), x[i]); // read again by this thread alone
+        if (p.norm == LB_NORM_LAYER) {
+            for (int i = t; i < p.width; i += 256) mean += x[i];
+            mean = block_sum(mean, red) / (float)p.width;
+        }
 #pragma unroll 4
-        for (int i = t; i < p.width; i += 256) ss += x[i] * x[i];
+        for (int i = t; i < p.width; i += 256) {
+            const float d = x[i] - mean;
+            ss += d * d;
+        }
     }
     ss = block_sum(ss, red);
     const float rinv = 1.0f / sqrtf(ss / (float)p.width + p.eps);
     pdl_launch_dependents();
+    if (!p.h[0]) return; // only the sum was asked for
+    const int copies = p.scatter ? p.top : 1;
     if (quads) {
 #pragma unroll
         for (int u = 0; u < NR_Q; ++u) {
@@ -263,26 +371,55 @@ extern "C" __global__ void __launch_bounds__(256) norm_rows2(const __grid_consta
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 if (!p.h[e]) continue;
-                const uint2 w = __ldg(reinterpret_cast<const uint2*>(p.w[e] + i));
-                const float a = v[u].x * rinv * (1.0f + __uint_as_float(w.x << 16)), b = v[u].y * rinv * (1.0f + __uint_as_float(w.x & 0xffff0000u)),
-                            c = v[u].z * rinv * (1.0f + __uint_as_float(w.y << 16)), d = v[u].w * rinv * (1.0f + __uint_as_float(w.y & 0xffff0000u));
-                if (p.f32) *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.h[e]) + o + i) = make_float4(a, b, c, d);
-                else {
-                    const __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
-                    *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(p.h[e]) + o + i) =
-                        make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+                const float4 w = nr_quad(p.w[e], i);
+                float4 r = make_float4(v[u].x * rinv * (one + w.x), v[u].y * rinv * (one + w.y), v[u].z * rinv * (one + w.z), v[u].w * rinv * (one + w.w));
+                if (p.norm == LB_NORM_LAYER) {
+                    const float4 b = nr_quad(p.b[e], i);
+                    r.x += b.x; r.y += b.y; r.z += b.z; r.w += b.w;
                 }
+                for (int k = 0; k < copies; ++k) nr_store4(p, p.h[e], (size_t)(p.scatter ? p.scatter[(size_t)tok * p.top + k] : tok) * p.ld + i, r);
             }
         }
     }
     for (int i = quads ? p.width + t : t; i < p.ld; i += 256) {
-        const float xv = i < p.width ? x[i] * rinv : 0.f;
+        const float xv = i < p.width ? (x[i] - mean) * rinv : 0.f;
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
             if (!p.h[e]) continue;
-            const float r = i < p.width ? xv * (1.0f + bf16_bits_to_f32(p.w[e][i])) : 0.f;
-            if (p.f32) reinterpret_cast<float*>(p.h[e])[o + i] = r;
-            else reinterpret_cast<__nv_bfloat16*>(p.h[e])[o + i] = __float2bfloat16_rn(r);
+            float r = i < p.width ? xv * (one + bf16_bits_to_f32(p.w[e][i])) : 0.f;
+            if (p.norm == LB_NORM_LAYER && i < p.width) r += bf16_bits_to_f32(p.b[e][i]);
+            for (int k = 0; k < copies; ++k) nr_store1(p, p.h[e], (size_t)(p.scatter ? p.scatter[(size_t)tok * p.top + k] : tok) * p.ld + i, r);
         }
     }
+}
+
+// The chunk's (token, expert) assignments sorted by expert: the row of every assignment, and the token tiles (of at most NT assignments of one
+// expert).  One CTA of 1024 threads per launch.
+extern "C" __global__ void __launch_bounds__(1024) moe_plan(const __grid_constant__ lb_moe_plan_params p) {
+    __shared__ int count[LB_MOE_MAX_EXPERTS], first[LB_MOE_MAX_EXPERTS], tile0[LB_MOE_MAX_EXPERTS], wsum[2][32];
+    const int t = threadIdx.x, n = p.T * p.top, lane = t & 31, warp = t >> 5;
+    count[t] = 0;
+    __syncthreads();
+    pdl_wait(); // the buffers written here may still be read by the kernels before
+    for (int a = t; a < n; a += 1024) p.place[a] = atomicAdd(&count[p.table[(size_t)p.tokens[a / p.top] * p.top + a % p.top]], 1);
+    __syncthreads();
+    // exclusive sums over experts of assignments and of tiles
+    const int c = t < p.experts ? count[t] : 0, nt = (c + p.NT - 1) / p.NT;
+    int ic = c, it = nt;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const int a = __shfl_up_sync(0xffffffffu, ic, o), b = __shfl_up_sync(0xffffffffu, it, o);
+        if (lane >= o) { ic += a; it += b; }
+    }
+    if (lane == 31) { wsum[0][warp] = ic; wsum[1][warp] = it; }
+    __syncthreads();
+    int bc = 0, bt = 0;
+    for (int w = 0; w < warp; ++w) { bc += wsum[0][w]; bt += wsum[1][w]; }
+    first[t] = bc + ic - c;
+    tile0[t] = bt + it - nt;
+    if (t == 1023) p.n_tiles[0] = bt + it;
+    for (int k = 0; k < nt; ++k) reinterpret_cast<int4*>(p.tiles)[tile0[t] + k] = make_int4(t, first[t] + k * p.NT, first[t] + c, 0);
+    __syncthreads();
+    for (int a = t; a < n; a += 1024) p.place[a] += first[p.table[(size_t)p.tokens[a / p.top] * p.top + a % p.top]];
+    pdl_launch_dependents();
 }

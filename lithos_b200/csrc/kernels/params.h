@@ -265,16 +265,24 @@ typedef struct {
 #define LB_RG_THREADS 256
 #define LB_RG_WARPS 8
 #define LB_RG_SEG 1024 /* elements of one row in a pipeline stage */
-enum { LB_RG_X_NORM = 0, /* vector of matrix i = rmsnorm(x) * (1 + norm_w[i]) */
-       LB_RG_X_CAT = 1   /* one vector: the mixer's output (per-head norm and gate applied here), then the feed-forward's activations */ };
+enum { LB_RG_X_NORM = 0, /* vector of matrix i = norm(x) with that matrix's weights */
+       LB_RG_X_CAT = 1   /* one vector: the mixer's output (norm of its parts and gate applied here), then the feed-forward's activations */ };
+/* norms in front of a product */
+enum { LB_NORM_RMS_1P = 0, /* x / rms(x) * (1 + w) */
+       LB_NORM_RMS = 1,    /* x / rms(x) * w */
+       LB_NORM_LAYER = 2   /* (x - mean) / sd * w + b */ };
 /* epilogues, shared with the matrix products of a prompt chunk (lb_dgemm_params) */
 enum { LB_DY_STORE = 0,    /* y[n] = r */
        LB_DY_RELU_GLU = 1, /* rows come as (gate, up) pairs: y[pair] = relu(gate) * up */
        LB_DY_RESIDUAL = 2, /* y[n] += mult * r */
-       LB_DY_SOFTCAP = 3   /* y[n] = cap * tanh(r / cap), cap 0: y[n] = r; with part_val: arg-max candidates */ };
+       LB_DY_SOFTCAP = 3,  /* y[n] = cap * tanh(r / cap), cap 0: y[n] = r; with part_val: arg-max candidates */
+       LB_DY_RELU2 = 4,    /* y[n] = max(r, 0)^2 */
+       LB_DY_CLAMP_GLU = 5, /* (gate, up) pairs: g = min(gate, limit), u = clamp(up, -limit, limit), y[pair] = g sigmoid(alpha g) (u + 1) */
+       LB_DY_HEADS = 6     /* prompt: bf16 y[n / head * head_p + n % head] */ };
 typedef struct {
     const uint16_t* w;      /* bf16 [rows, K] */
     const uint16_t* norm_w; /* bf16 [width] (LB_RG_X_NORM) */
+    const uint16_t* norm_b; /* bf16 [width] (LB_NORM_LAYER) */
     float* y;
     int32_t rows;           /* rows with a result (the allocation holds an even number) */
     int32_t y_mode;
@@ -284,7 +292,7 @@ typedef struct {
     const float* x;         /* LB_RG_X_NORM: fp32 [width] */
     const float* mix;       /* LB_RG_X_CAT: fp32 [n_mix] */
     const float* gate;      /* fp32 [n_mix]: mix *= silu(gate); NULL = no gate */
-    const uint16_t* head_w; /* bf16 [vdim]: mix = per-head rmsnorm * head_w first; NULL = none */
+    const uint16_t* head_w; /* mix = rmsnorm of each part of vdim values * head_w first (bf16 [vdim]; [n_mix] with gate_first); NULL = none */
     const float* act;       /* fp32 [n_act] */
     float* part_val;        /* [gridDim.x] arg-max candidates (LB_DY_SOFTCAP), or NULL */
     int32_t* part_idx;
@@ -295,8 +303,20 @@ typedef struct {
     int32_t split;          /* pieces a row pair is cut into along K: 1, or one per stage segment */
     int32_t segs;           /* ceil(K / LB_RG_SEG) */
     int32_t x_cols;         /* columns of a vector one CTA holds: K, or the longer half where two CTAs share a row */
+    int32_t norm;           /* LB_NORM_* (LB_RG_X_NORM) */
+    int32_t gate_first;     /* mix is gated before its norm, not after */
+    /* experts: a matrix is a stack of `experts`; sel[0..parts) (a row of a table, row *sel_row) names the ones this token uses */
+    const int32_t* sel;     /* NULL: no experts */
+    const int32_t* sel_row; /* row of sel; written well before the launch in front of this one has started */
+    int32_t parts;          /* experts per token (1 without experts) */
+    int32_t sel_rows;       /* LB_RG_X_NORM: rows of one expert; mat.rows = parts * sel_rows, results of part i start at y[i * y_part] */
+    int32_t y_part;
+    int32_t k_part;         /* LB_RG_X_CAT: columns of one expert; K = parts * k_part, expert e is [rows padded to even][k_part].  Else K */
+    int32_t segs_part;      /* ceil(k_part / LB_RG_SEG); segs = parts * segs_part */
+    float limit, alpha;     /* LB_DY_CLAMP_GLU */
     float eps, mult, cap;
 } lb_rows_gemv_params;
+#define LB_RG_MAX_PARTS 32
 
 /* ---- dense products of a prompt chunk: Y[T, N] = X[T, K] W[N, K]^T, one or two of them in one launch --------- */
 #define LB_DG_ROWS 128  /* weight rows per tile = M of the product */
@@ -313,17 +333,42 @@ typedef struct {
     int32_t tiles[2];     /* row tiles of each product (tiles[1] = 0: one product) */
     int32_t y_f32[2];     /* LB_DY_RELU_GLU: y is fp32 (else bf16) */
     int32_t T, NT, t_tiles, K, ld_x, stages, tmem_cols;
-    float mult, cap;
+    int32_t head[2], head_p[2]; /* LB_DY_HEADS */
+    float mult, cap, limit, alpha;
     uint32_t* status;
+    /* experts (one product): w is a stack of experts, x and y have the chunk's (token, expert) assignments sorted by
+     * expert; a token tile is plan_tiles[i] = (expert, first assignment, end of the expert's assignments, 0), i < *plan_n */
+    const int32_t* plan_tiles; /* NULL: no experts */
+    const int32_t* plan_n;
+    int32_t expert_rows; /* rows of the stack from one expert to the next */
 } lb_dgemm_params;
 
-/* rmsnorm of a chunk with up to two weights: h_i[t] = rmsnorm(x[t]) * (1 + w_i) */
+/* a chunk's (token, expert) assignments sorted by expert (moe_plan) */
 typedef struct {
-    const float* x;      /* fp32 [T, width] */
+    const int32_t* tokens; /* [T] */
+    const int32_t* table;  /* [vocab, top]: the experts of a token id */
+    int32_t* place;        /* [T, top]: row of the assignment in sorted order */
+    int32_t* tiles;        /* as lb_dgemm_params.plan_tiles */
+    int32_t* n_tiles;
+    int32_t T, top, experts, NT;
+} lb_moe_plan_params;
+#define LB_MOE_MAX_EXPERTS 1024
+
+/* norm of a chunk's rows with up to two weights: h_i[t] = norm(x[t]) with w_i (and b_i).  Before it, optionally, x[t] += mult * the sum of the
+ * token's rows of y (place: a layer's expert outputs); after it, optionally, the row goes to `scatter` places instead of place t */
+typedef struct {
+    float* x;            /* fp32 [T, ld_x] */
     const uint16_t* w[2];
+    const uint16_t* b[2]; /* LB_NORM_LAYER */
     void* h[2];          /* bf16 (or fp32) [T, ld]; h[1] may be NULL */
-    int32_t width, ld, f32;
+    int32_t width, ld, ld_x, f32, norm;
     float eps;
+    const void* y;       /* NULL: nothing to add; bf16 (or fp32) [assignments, ld_y] */
+    const int32_t* y_place; /* [T, y_top] */
+    int32_t y_top, ld_y;
+    float y_mult;
+    const int32_t* scatter; /* NULL, or [T, top]: h_0[scatter[t, i]] = row */
+    int32_t top;
 } lb_norm2_params;
 
 /* ---- attention over the current block of positions, general head sizes (window_attention.cu) ---------------- */
@@ -350,6 +395,10 @@ typedef struct {
     int32_t sink;        /* 1 is added to the soft-max denominator */
     int32_t pos0, T, max_ctx, splits, cat_ld;
     float scale, eps;
+    /* prompt, bf16: the last tail_p of a key's dim_p values are shared by all heads: k_tail rows (of tail_ld values), k_cache rows without them */
+    const uint16_t* k_tail;
+    int32_t tail_p, tail_ld;
+    const uint16_t* sink_w; /* bf16 [H]: exp(sink_w) is added to the denominator instead of 1 */
 } lb_wattn_params;
 /* wattn_chunk_*: query rows per CTA (16 per warp), keys per staged block */
 #define LB_WA_ROWS 64
@@ -378,6 +427,61 @@ typedef struct {
     int32_t seg;          /* prompt: tokens per segment, a multiple of 4 (T or more: one segment) */
     float q_scale, inv_tau, eps;
 } lb_decay_params2;
+
+/* ---- attention over a cached latent (latent_attention.cu) ---------------------------------------------------
+ * A position is cached as one row [latent c (rank_p) | rotated key part shared by all heads (rot_p)]; a head's key is [W_uk c | that part],
+ * its value W_uv c. */
+#define LB_LA_MAX_RANK 512
+#define LB_LA_MAX_ROT 128
+#define LB_LA_MAX_SPLITS 64
+#define LB_LA_TOKENS 8 /* tokens a CTA of lat_query / lat_out walks with one read of its weights */
+#define LB_LA_KEYS 64  /* lat_rows_bf16: cache rows per staged block */
+typedef struct {
+    const float* proj;     /* fp32 [T, ld]: at kv_off the latent (rank) and the shared key part (rot), before norm and rotation */
+    const float* q;        /* fp32 [T, H * (dim + rot)] */
+    const uint16_t* uk;    /* bf16 [H * dim, rank_p] */
+    const uint16_t* uv;    /* bf16 [H * vdim, rank_p] */
+    const uint16_t* c_norm; /* bf16 [rank] */
+    const uint16_t* sink;  /* bf16 [H]: exp(sink) joins the denominator; NULL: none */
+    const double* freq;    /* [rot / 2] radians per position */
+    void* cache;           /* bf16 (or fp32) [max_ctx, rank_p + rot_p]; padding columns are zero */
+    float* ql;             /* fp32 [T, H, rank_p + rot_p]: (W_uk^T q | rotated q) * scale */
+    float* part;           /* fp32 [T * H][splits][rank_p + 2]: weighted sum of latents, maximum, denominator of a slice of positions */
+    float* out;            /* fp32 [H * vdim] of one token (decode) ... */
+    void* cat;             /* ... or, when not NULL, rows [T, cat_ld] of bf16 / fp32 */
+    uint16_t* qh;          /* lat_prepare: queries x scale x log2(e) as two bf16 terms [T, H, dim_p + rot_p]; NULL: cache rows only */
+    uint16_t* ql16;
+    const int32_t* pos_ptr; /* position of token 0 in device memory, or NULL: pos0 */
+    uint32_t* status;
+    int32_t ld, kv_off, H, dim, dim_p, vdim, rank, rank_p, rot, rot_p;
+    int32_t pos0, T, max_ctx, splits, cat_ld, stages;
+    float rot_mul, scale, eps;
+} lb_latent_params;
+
+/* ---- state-space recurrence with a scalar decay per head (ssm.cu) -------------------------------------------- */
+#define LB_SSM_MAX_TAPS 8
+#define LB_SSM_MAX_STATE 256
+#define LB_SSM_SEG 64  /* tokens per block of ssm_chunk_* */
+#define LB_SSM_COLS 32 /* value columns per CTA */
+typedef struct {
+    const float* proj;      /* fp32 [T, ld]: z [H V] | x [H V] | B [G N] | C [G N] | dt [H] */
+    const uint16_t* conv_w; /* bf16 [channels, taps], last column = the current token */
+    const uint16_t* conv_b; /* bf16 [channels] */
+    const uint16_t* dt_bias; /* bf16 [H] */
+    const uint16_t* a_log;
+    const uint16_t* d;
+    const uint16_t* norm_w; /* bf16 [H V] */
+    float* state;           /* fp32 [H, N, V] */
+    float* ring;            /* fp32 [taps, channels]: slot position % taps holds that position's values before the convolution */
+    float* y;               /* fp32 [T, H V] */
+    void* xbc;              /* prompt: x [H, V_p] | B [G, N_p] | C [G, N_p] after the convolution, bf16 (or fp32), padding zero, rows of ld_xbc */
+    float* dt;              /* prompt: fp32 [T, H] step sizes */
+    void* cat;              /* prompt: gated, normed rows [T, cat_ld] */
+    const int32_t* pos_ptr; /* decode: position in device memory */
+    int32_t ld, H, V, V_p, N, N_p, G, taps, channels, ld_xbc, norm_groups;
+    int32_t pos0, T, cat_ld, f32;
+    float eps;
+} lb_ssm_params;
 
 /* ---- tensor-parallel exchange (comm.cu) ----------------------------------------------- */
 #define LB_TP_MAX 8

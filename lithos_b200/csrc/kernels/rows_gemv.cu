@@ -1,7 +1,7 @@
 // Dense bf16 rows x one fp32 vector for the decode step of bf16 models: one launch takes one or two matrices, builds the input
 // vector(s) in shared memory (RMS norm with the layer's weights; or the mixer's output with its per-head norm and gate, followed
-// by the feed-forward's activations) and finishes every row (store, ReLU-gated product of neighbouring rows, residual add, soft cap
-// with arg-max candidates).  The vector stays fp32; weights are exact in fp32, sums are fp32 in a fixed order.
+// by the feed-forward's activations) and finishes every row (store, gated product of neighbouring rows, squared ReLU, residual add, soft cap
+// with arg-max candidates).  A matrix may be a stack of experts of which the token uses a few: their rows, or their columns, follow one another.  The vector stays fp32; weights are exact in fp32, sums are fp32 in a fixed order.
 //
 // HBM-bound: one CTA per SM, every warp streams its own row segments with 1-D bulk copies through its own ring, so what is in flight
 // (ring bytes x 148) does not depend on registers.  Two rows share every read of the vector: shared memory moves 2 bytes of weights in,
@@ -46,6 +46,8 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
         for (int s = 0; s < S; ++s) mbar_init(&bars[warp * S + s], 1);
     if (tid == 0) mbar_init(&bars[LB_RG_WARPS * S], 1);
     mbar_fence_init();
+    __shared__ int sel_s[LB_RG_MAX_PARTS];
+    if (p.sel && tid < p.parts) sel_s[tid] = p.sel[(size_t)p.sel_row[0] * p.parts + tid];
     __syncthreads();
 
     // the warp's stages: items warp, warp + 8, ... (item = pair * split + piece), segments of the item in order
@@ -54,28 +56,50 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
     auto row_ptr = [&](int pair, int& mi) -> const uint16_t* {
         const int g = c + pair * G;
         mi = g >= pairs0;
+        if (p.sel && p.x_mode == LB_RG_X_NORM) { // the parts' rows one after the other, each part's from its expert
+            const int part_pairs = p.sel_rows >> 1, e = g / part_pairs;
+            return p.mat[0].w + ((size_t)sel_s[e] * part_pairs + (g - e * part_pairs)) * 2 * p.K;
+        }
         return mi ? p.mat[1].w + (size_t)(g - pairs0) * 2 * p.K : p.mat[0].w + (size_t)g * 2 * p.K;
+    };
+    // a row segment: its first column and length; with experts side by side along K a row is in pieces of k_part columns
+    const bool sel_k = p.sel && p.x_mode == LB_RG_X_CAT;
+    const size_t row_step = sel_k ? p.k_part : p.K, expert_pairs = sel_k ? (size_t)((p.mat[0].rows + 1) >> 1) : 0;
+    auto segment = [&](int seg, int& col, int& len, int& e) {
+        if (sel_k) {
+            e = seg / p.segs_part;
+            const int off = (seg - e * p.segs_part) * LB_RG_SEG;
+            col = e * p.k_part + off;
+            len = min(LB_RG_SEG, p.k_part - off);
+        } else {
+            col = seg * LB_RG_SEG;
+            len = min(LB_RG_SEG, p.K - col);
+        }
     };
     int r_item = warp, r_seg = 0, r_slot = 0; // next stage to request
     auto request = [&]() {
         if (r_item >= items) return;
         if (lane == 0) {
             const int pair = split == 1 ? r_item : r_item / split, seg = seg_lo + (r_item - pair * split) * spp + r_seg;
-            int mi;
-            const uint16_t* w = row_ptr(pair, mi) + (size_t)seg * LB_RG_SEG;
-            const uint32_t bytes = (uint32_t)min(LB_RG_SEG, p.K - seg * LB_RG_SEG) * 2u;
+            int mi, col, len, e = 0;
+            segment(seg, col, len, e);
+            const uint16_t* w = sel_k ? p.mat[0].w + ((size_t)sel_s[e] * expert_pairs + (c + pair * G)) * 2 * p.k_part + (col - e * p.k_part) : row_ptr(pair, mi) + col;
+            const uint32_t bytes = (uint32_t)len * 2u;
             unsigned char* dst = ring + (size_t)(warp * S + r_slot) * (LB_RG_SEG * 4);
             uint64_t* bar = &bars[warp * S + r_slot];
             mbar_arrive_expect_tx(bar, 2 * bytes);
             bulk_g2s(dst, w, bytes, bar, pol);
-            bulk_g2s(dst + LB_RG_SEG * 2, w + p.K, bytes, bar, pol);
+            bulk_g2s(dst + LB_RG_SEG * 2, w + row_step, bytes, bar, pol);
         }
         if (++r_seg == spp) { r_seg = 0; r_item += LB_RG_WARPS; }
         if (++r_slot == S) r_slot = 0;
     };
     for (int s = 0; s < S; ++s) request(); // weights are constants: asked for before the previous kernel has finished
 
-    // the norm weights are constants too: a thread's first 8 quads of them come in before the wait
+    // the norm weights are constants too: a thread's first 8 quads of them (of the two vectors, or weight and bias of one) come in before
+    // the wait
+    const bool layer_norm = p.norm == LB_NORM_LAYER;
+    const uint16_t* second = n_vec > 1 ? p.mat[1].norm_w : layer_norm ? p.mat[0].norm_b : nullptr;
     const bool quads = (p.width & 3) == 0;
     uint2 w_pre[2][8];
     if (p.x_mode == LB_RG_X_NORM && quads) {
@@ -84,7 +108,8 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
 #pragma unroll
             for (int u = 0; u < 8; ++u) {
                 const int i = 4 * (tid + u * LB_RG_THREADS);
-                w_pre[v][u] = v < n_vec && i < p.width ? __ldg(reinterpret_cast<const uint2*>(p.mat[v].norm_w + i)) : make_uint2(0u, 0u);
+                const uint16_t* src = v == 0 ? p.mat[0].norm_w : second;
+                w_pre[v][u] = src && i < p.width ? __ldg(reinterpret_cast<const uint2*>(src + i)) : make_uint2(0u, 0u);
             }
     }
     // the vector's parts come as bulk copies straight into its place (whole 16-byte pieces; what is left over by plain loads), so the
@@ -105,23 +130,42 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
         const bool here = mbar_wait(xbar, 0);
         if (!here && p.status) atomicExch(p.status, LB_DEV_TIMEOUT_FULL);
         __syncthreads();
-        float ss = 0.f;
-        for (int i = tid; i < p.K / 4; i += LB_RG_THREADS) {
-            const float4 v = *reinterpret_cast<const float4*>(xsm + 4 * i);
-            ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+        float mean = 0.f, ss = 0.f;
+        if (layer_norm) {
+            for (int i = tid; i < p.width; i += LB_RG_THREADS) mean += xsm[i];
+            mean = block_sum(mean, red) / (float)p.width;
+            for (int i = tid; i < p.width; i += LB_RG_THREADS) {
+                const float d = xsm[i] - mean;
+                ss += d * d;
+            }
+        } else {
+            for (int i = tid; i < p.K / 4; i += LB_RG_THREADS) {
+                const float4 v = *reinterpret_cast<const float4*>(xsm + 4 * i);
+                ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+            }
         }
         ss = block_sum(ss, red);
-        const float rinv = 1.0f / sqrtf(ss / (float)p.width + p.eps);
+        const float rinv = 1.0f / sqrtf(ss / (float)p.width + p.eps), one = p.norm == LB_NORM_RMS_1P ? 1.0f : 0.0f;
         if (quads) {
-            auto apply = [&](int i, uint2 a, uint2 b) { // quad at i with the norm weights of the one or two vectors
+            auto quad = [](uint2 w) {
+                return make_float4(__uint_as_float(w.x << 16), __uint_as_float(w.x & 0xffff0000u), __uint_as_float(w.y << 16), __uint_as_float(w.y & 0xffff0000u));
+            };
+            auto apply = [&](int i, uint2 a, uint2 b) { // quad at i with the norm weights of the one or two vectors (layer norm of one: weight, bias)
                 float4 v = *reinterpret_cast<const float4*>(xsm + i);
-                v.x *= rinv; v.y *= rinv; v.z *= rinv; v.w *= rinv;
+                v.x = (v.x - mean) * rinv; v.y = (v.y - mean) * rinv; v.z = (v.z - mean) * rinv; v.w = (v.w - mean) * rinv;
                 auto scaled = [&](uint2 w) {
-                    return make_float4(v.x * (1.0f + __uint_as_float(w.x << 16)), v.y * (1.0f + __uint_as_float(w.x & 0xffff0000u)),
-                                       v.z * (1.0f + __uint_as_float(w.y << 16)), v.w * (1.0f + __uint_as_float(w.y & 0xffff0000u)));
+                    const float4 f = quad(w);
+                    return make_float4(v.x * (one + f.x), v.y * (one + f.y), v.z * (one + f.z), v.w * (one + f.w));
                 };
-                *reinterpret_cast<float4*>(xsm + i) = scaled(a);
-                if (n_vec > 1) *reinterpret_cast<float4*>(xsm + p.K + i) = scaled(b);
+                auto shift = [&](float4 r, float4 o) { return make_float4(r.x + o.x, r.y + o.y, r.z + o.z, r.w + o.w); };
+                float4 r = scaled(a);
+                if (layer_norm) r = shift(r, quad(n_vec > 1 ? *reinterpret_cast<const uint2*>(p.mat[0].norm_b + i) : b));
+                *reinterpret_cast<float4*>(xsm + i) = r;
+                if (n_vec > 1) {
+                    r = scaled(b);
+                    if (layer_norm) r = shift(r, quad(*reinterpret_cast<const uint2*>(p.mat[1].norm_b + i)));
+                    *reinterpret_cast<float4*>(xsm + p.K + i) = r;
+                }
             };
 #pragma unroll
             for (int u = 0; u < 8; ++u) {
@@ -129,12 +173,17 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
                 if (i < p.width) apply(i, w_pre[0][u], w_pre[1][u]);
             }
             for (int i = 4 * (tid + 8 * LB_RG_THREADS); i < p.width; i += 4 * LB_RG_THREADS)
-                apply(i, *reinterpret_cast<const uint2*>(p.mat[0].norm_w + i), n_vec > 1 ? *reinterpret_cast<const uint2*>(p.mat[1].norm_w + i) : make_uint2(0u, 0u));
+                apply(i, *reinterpret_cast<const uint2*>(p.mat[0].norm_w + i), second ? *reinterpret_cast<const uint2*>(second + i) : make_uint2(0u, 0u));
         } else {
             for (int i = tid; i < p.width; i += LB_RG_THREADS) {
-                const float v = xsm[i] * rinv;
-                xsm[i] = v * (1.0f + bf16_bits_to_f32(p.mat[0].norm_w[i]));
-                if (n_vec > 1) xsm[p.K + i] = v * (1.0f + bf16_bits_to_f32(p.mat[1].norm_w[i]));
+                const float v = (xsm[i] - mean) * rinv;
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    if (e >= n_vec) continue;
+                    float r = v * (one + bf16_bits_to_f32(p.mat[e].norm_w[i]));
+                    if (layer_norm) r += bf16_bits_to_f32(p.mat[e].norm_b[i]);
+                    xsm[e * p.K + i] = r;
+                }
             }
         }
     } else {
@@ -157,7 +206,23 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
         const bool here = mbar_wait(xbar, 0);
         if (!here && p.status) atomicExch(p.status, LB_DEV_TIMEOUT_FULL);
         __syncthreads();
-        if (p.head_w) {
+        if (p.head_w && p.gate_first) { // gate, then the norm of every part; a part is a warp's work, or everybody's when there are few
+            if (p.gate)
+                for (int i = tid; i < n_mix; i += LB_RG_THREADS) {
+                    const float g = gate_s[i];
+                    xsm[i] *= g * rg_sigmoid(g);
+                }
+            __syncthreads();
+            const int n_part = n_mix / p.vdim, all = n_part < LB_RG_WARPS, step = all ? LB_RG_THREADS : 32, first = all ? tid : lane;
+            for (int h = all ? 0 : warp; h < n_part; h += all ? 1 : LB_RG_WARPS) {
+                float* o = xsm + (size_t)h * p.vdim;
+                float ss = 0.f;
+                for (int i = first; i < p.vdim; i += step) ss += o[i] * o[i];
+                ss = all ? block_sum(ss, red) : warp_sum(ss);
+                const float rinv = 1.0f / sqrtf(ss / (float)p.vdim + p.eps);
+                for (int i = first; i < p.vdim; i += step) o[i] *= rinv * bf16_bits_to_f32(__ldg(p.head_w + (size_t)h * p.vdim + i));
+            }
+        } else if (p.head_w) {
             const int heads = n_mix / p.vdim;
             for (int h = warp; h < heads; h += LB_RG_WARPS) {
                 float* o = xsm + (size_t)h * p.vdim;
@@ -191,7 +256,9 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
                 ok = false;
                 break;
             }
-            const int k0 = (seg0 + s) * LB_RG_SEG, n8 = min(LB_RG_SEG, p.K - k0) >> 3;
+            int k0, len, e;
+            segment(seg0 + s, k0, len, e);
+            const int n8 = len >> 3;
             const uint4* wa = reinterpret_cast<const uint4*>(ring + (size_t)(warp * S + slot) * (LB_RG_SEG * 4));
             const uint4* wb = wa + LB_RG_SEG / 8;
 #pragma unroll 4
@@ -258,6 +325,10 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
         const lb_rg_mat& M = p.mat[mi];
         if (M.y_mode == LB_DY_RELU_GLU) {
             M.y[n >> 1] = fmaxf(r[0], 0.f) * r[1];
+        } else if (M.y_mode == LB_DY_CLAMP_GLU) {
+            const int part = p.sel ? n / p.sel_rows : 0, i = (n - part * p.sel_rows) >> 1;
+            const float ga = fminf(r[0], p.limit), up = fminf(fmaxf(r[1], -p.limit), p.limit);
+            M.y[(size_t)part * p.y_part + i] = ga * rg_sigmoid(p.alpha * ga) * (up + 1.0f);
         } else {
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
@@ -265,6 +336,7 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
                 float v = r[e];
                 if (M.y_mode == LB_DY_RESIDUAL) v = fmaf(p.mult, v, M.y[n + e]);
                 else if (M.y_mode == LB_DY_SOFTCAP && p.cap > 0.f) v = p.cap * tanhf(v / p.cap);
+                else if (M.y_mode == LB_DY_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
                 M.y[n + e] = v;
                 if (v > best_v || (v == best_v && n + e < best_i)) { best_v = v; best_i = n + e; }
             }

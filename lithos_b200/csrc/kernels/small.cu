@@ -14,6 +14,22 @@ extern "C" __global__ void embed_bf16(const uint16_t* __restrict__ table, const 
         out[i] = bf16_bits_to_f32(table[base + i]);
 }
 
+// x[t] = E[token[t]] + B[row], row = (previous token * mul_prev + token * mul_cur) mod buckets, the last row (`buckets`) for a sequence's first
+// token.  `hist` holds a sequence's tokens by position.  A prompt's tokens are in it already (token == NULL, position pos0 + t); a decode step
+// brings one token, which is entered.  grid (.., tokens)
+extern "C" __global__ void embed_bigram(const uint16_t* __restrict__ table, const uint16_t* __restrict__ bigram, const int* __restrict__ token,
+                                        const int* __restrict__ pos_ptr, int pos0, int* __restrict__ hist, float* __restrict__ out, int D, int buckets,
+                                        int mul_prev, int mul_cur) {
+    pdl_wait();
+    const int t = blockIdx.y, pos = (pos_ptr ? pos_ptr[0] : pos0) + t, cur = token ? token[0] : hist[pos];
+    long long row = buckets;
+    if (pos > 0) row = ((long long)hist[pos - 1] * mul_prev + (long long)cur * mul_cur) % buckets;
+    if (token && blockIdx.x == 0 && threadIdx.x == 0) hist[pos] = cur;
+    const size_t e = (size_t)cur * D, b = (size_t)row * D, o = (size_t)t * D;
+    for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < D; i += gridDim.x * blockDim.x)
+        out[o + i] = bf16_bits_to_f32(table[e + i]) + bf16_bits_to_f32(bigram[b + i]);
+}
+
 // Greedy sampling: index of the maximum, FIRST maximum on ties (strict > in
 // inference/reduce.ls:225-227 and src/launcher.s:1060-1063).  One CTA; the
 // (value, index) pairs are combined with "greater value, else smaller index",

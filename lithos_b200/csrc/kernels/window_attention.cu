@@ -7,63 +7,16 @@
 //   wattn_rows_*   one query token per CTA row: the decode step (positions cut into slices merged by the last CTA), and prompts in fp32
 //   wattn_prepare  a prompt chunk's keys and values into the cache; its queries as two bf16 terms
 //   wattn_chunk_*  a prompt chunk on the tensor cores
-#include "common.cuh"
-#include "params.h"
+#include "mma_sync.cuh"
+#include "rotate.cuh"
 
-template <typename T> struct wa_t;
-template <> struct wa_t<__nv_bfloat16> {
-    static __device__ __forceinline__ void ld8(const __nv_bfloat16* p, float (&f)[8]) {
-        const uint4 u = *reinterpret_cast<const uint4*>(p);
-        const uint32_t w[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            f[2 * i] = __uint_as_float(w[i] << 16);
-            f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
-        }
-    }
-    static __device__ __forceinline__ float2 ld2(const __nv_bfloat16* p) {
-        const uint32_t u = *reinterpret_cast<const uint32_t*>(p);
-        return make_float2(__uint_as_float(u << 16), __uint_as_float(u & 0xffff0000u));
-    }
-    static __device__ __forceinline__ __nv_bfloat16 from(float v) { return __float2bfloat16_rn(v); }
-};
-template <> struct wa_t<float> {
-    static __device__ __forceinline__ void ld8(const float* p, float (&f)[8]) {
-        const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-        f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
-    }
-    static __device__ __forceinline__ float2 ld2(const float* p) { return *reinterpret_cast<const float2*>(p); }
-    static __device__ __forceinline__ float from(float v) { return v; }
-};
-
-__device__ __forceinline__ void wa_cp16(uint32_t dst, const void* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
-}
 struct wa_angles { // cosines and sines of a position: key / query pairs and value pairs
     float ck[LB_WA_MAX_DIM / 2], sk[LB_WA_MAX_DIM / 2], cv[LB_WA_MAX_DIM / 2], sv[LB_WA_MAX_DIM / 2];
 };
-__device__ __forceinline__ void wa_angle(double f, int pos, float& c, float& s) { // product and reduction modulo 2 pi in double
-    const double a = (double)pos * f, k = rint(a * 0.15915494309189535);
-    sincosf((float)fma(-k, 6.283185307179586, a), &s, &c);
-}
 __device__ __forceinline__ void wa_fill_angles(const lb_wattn_params& p, int pos, wa_angles& A) {
     for (int i = threadIdx.x; i < p.rot_dims / 2; i += blockDim.x) wa_angle(p.freq_k[i], pos, A.ck[i], A.sk[i]);
     if (p.freq_v)
         for (int i = threadIdx.x; i < p.vdim / 2; i += blockDim.x) wa_angle(p.freq_v[i], pos, A.cv[i], A.sv[i]);
-}
-// one warp: dst[0..dim) = rotated src (times mul)
-template <typename T>
-__device__ __forceinline__ void wa_warp_rotate(const float* src, T* dst, int dim, int rot_dims, const float* cs, const float* sn, float mul) {
-    for (int i = threadIdx.x & 31; i < (dim + 1) / 2; i += 32) {
-        float u = src[2 * i], v = 2 * i + 1 < dim ? src[2 * i + 1] : 0.f;
-        if (2 * i < rot_dims) {
-            const float a = u * cs[i] - v * sn[i];
-            v = v * cs[i] + u * sn[i];
-            u = a;
-        }
-        dst[2 * i] = wa_t<T>::from(u * mul);
-        if (2 * i + 1 < dim) dst[2 * i + 1] = wa_t<T>::from(v * mul);
-    }
 }
 template <typename T>
 __device__ __forceinline__ void wa_warp_value(const lb_wattn_params& p, const float* src, T* dst, const wa_angles& A) {
@@ -124,11 +77,11 @@ __device__ __forceinline__ void wattn_rows_body(const lb_wattn_params& p) {
         const int kq = p.dim_p / E, vq = p.vdim_p / E;
         for (int i = lane; i < 32 * kq; i += 32) {
             const int r = i / kq, c = i - r * kq;
-            wa_cp16(smem_u32(kt + r * ks_t + c * E), kc + (size_t)min(b + r, r1 - 1) * ks + c * E);
+            ms_cp16(smem_u32(kt + r * ks_t + c * E), kc + (size_t)min(b + r, r1 - 1) * ks + c * E);
         }
         for (int i = lane; i < 32 * vq; i += 32) {
             const int r = i / vq, c = i - r * vq;
-            wa_cp16(smem_u32(vt + r * vs_t + c * E), vc + (size_t)min(b + r, r1 - 1) * vs + c * E);
+            ms_cp16(smem_u32(vt + r * vs_t + c * E), vc + (size_t)min(b + r, r1 - 1) * vs + c * E);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -377,27 +330,8 @@ extern "C" __global__ void __launch_bounds__(256) wattn_prepare_bf16(const __gri
 extern "C" __global__ void __launch_bounds__(256) wattn_prepare_f32(const __grid_constant__ lb_wattn_params p) { wattn_prepare_body<float>(p); }
 
 // ---- a prompt chunk on the tensor cores -----------------------------------------------------------------------------
-__device__ __forceinline__ void wa_mma(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-        : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-        : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void wa_ldsm(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void wa_ldsm_t(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void wa_split(float x, float y, uint32_t& hi, uint32_t& lo) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-    const float2 hf = __bfloat1622float2(h);
-    const __nv_bfloat162 l = __floats2bfloat162_rn(x - hf.x, y - hf.y);
-    hi = *reinterpret_cast<const uint32_t*>(&h);
-    lo = *reinterpret_cast<const uint32_t*>(&l);
-}
-
 // grid (ceil(T G / LB_WA_ROWS), KV), block LB_WA_THREADS.  Query row R of a KV head = (token R / G, head R % G).  S = Q K^T and O = P V as
-// mma.sync m16n8k16 with Q and P in two bf16 terms, online soft-max in log2 units (the sink enters as a first score of 0), cache rows staged
+// mma.sync m16n8k16 with Q and P in two bf16 terms, online soft-max in log2 units (the sink enters as a first score: 0, or the head's own), cache rows staged
 // LB_WA_KV at a time from the first block start any row of the CTA sees.  NB: value features / 8 the accumulators hold.
 // dynamic shared memory: qh | ql [ROWS][2 dim_p + 16 B], then two stages of K [KV][2 dim_p + 16] and V [KV][2 vdim_p + 16]
 template <int NB>
@@ -414,22 +348,25 @@ __device__ __forceinline__ void wattn_chunk_body(const lb_wattn_params& p) {
     for (int i = t; i < LB_WA_ROWS * q16; i += LB_WA_THREADS) { // rows past the chunk repeat the last one; they are never stored
         const int r = i / q16, c = i - r * q16, R = min(R0 + r, n_rows - 1), s = R / G;
         const size_t src = ((size_t)s * p.H + kv * G + (R - s * G)) * p.dim_p + c * 8;
-        wa_cp16(smem_u32(qh_s + r * qst + c * 16), p.qh + src);
-        wa_cp16(smem_u32(ql_s + r * qst + c * 16), p.ql + src);
+        ms_cp16(smem_u32(qh_s + r * qst + c * 16), p.qh + src);
+        ms_cp16(smem_u32(ql_s + r * qst + c * 16), p.ql + src);
     }
     const int s_first = R0 / G, s_last = min(R0 + LB_WA_ROWS - 1, n_rows - 1) / G;
     const int first_key = p.block > 0 ? (p.pos0 + s_first) / p.block * p.block : 0, last_key = p.pos0 + s_last;
     const int n_blocks = (last_key - first_key) / LB_WA_KV + 1;
-    const unsigned char* kbase = reinterpret_cast<const unsigned char*>(p.k_cache) + (size_t)kv * p.dim_p * 2;
+    const int own_p = p.dim_p - p.tail_p, own16 = own_p / 8; // of a key: what the head has of its own
+    const unsigned char* kbase = reinterpret_cast<const unsigned char*>(p.k_cache) + (size_t)kv * own_p * 2;
+    const unsigned char* tbase = reinterpret_cast<const unsigned char*>(p.k_tail);
     const unsigned char* vbase = reinterpret_cast<const unsigned char*>(p.v_cache) + (size_t)kv * p.vdim_p * 2;
-    const size_t krow = (size_t)p.KV * p.dim_p * 2, vrow = (size_t)p.KV * p.vdim_p * 2;
+    const size_t krow = (size_t)p.KV * own_p * 2, vrow = (size_t)p.KV * p.vdim_p * 2, trow = (size_t)p.tail_ld * 2;
     auto stage = [&](int b) { // rows past the last one repeat it (finite values; masked below)
         unsigned char* dst = kv_s + (b & 1) * stage_bytes;
         for (int i = t; i < LB_WA_KV * (q16 + v16); i += LB_WA_THREADS) {
             const int r = i / (q16 + v16), c = i - r * (q16 + v16);
             const size_t row = (size_t)min(first_key + b * LB_WA_KV + r, last_key);
-            if (c < q16) wa_cp16(smem_u32(dst + r * qst + c * 16), kbase + row * krow + c * 16);
-            else wa_cp16(smem_u32(dst + LB_WA_KV * qst + r * vst + (c - q16) * 16), vbase + row * vrow + (c - q16) * 16);
+            if (c < own16) ms_cp16(smem_u32(dst + r * qst + c * 16), kbase + row * krow + c * 16);
+            else if (c < q16) ms_cp16(smem_u32(dst + r * qst + c * 16), tbase + row * trow + (c - own16) * 16);
+            else ms_cp16(smem_u32(dst + LB_WA_KV * qst + r * vst + (c - q16) * 16), vbase + row * vrow + (c - q16) * 16);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -445,7 +382,7 @@ __device__ __forceinline__ void wattn_chunk_body(const lb_wattn_params& p) {
     float m_run[2], l_run[2], acc[NB][4];
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
-        m_run[i] = p.sink ? 0.f : -1e30f;
+        m_run[i] = !p.sink ? -1e30f : p.sink_w ? bf16_bits_to_f32(p.sink_w[kv * G + min(R0 + warp * 16 + fg + 8 * i, n_rows - 1) % G]) * 1.4426950408889634f : 0.f;
         l_run[i] = p.sink ? 1.f : 0.f;
     }
 #pragma unroll
@@ -473,16 +410,16 @@ __device__ __forceinline__ void wattn_chunk_body(const lb_wattn_params& p) {
 #pragma unroll 4
             for (int c = 0; c < nkc; ++c) {
                 uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
-                wa_ldsm(qh_lane + c * 32, h0, h1, h2, h3);
-                wa_ldsm(ql_lane + c * 32, l0, l1, l2, l3);
+                ms_ldsm(qh_lane + c * 32, h0, h1, h2, h3);
+                ms_ldsm(ql_lane + c * 32, l0, l1, l2, l3);
 #pragma unroll
                 for (int jj = 0; jj < 2; ++jj) {
                     uint32_t b00, b01, b10, b11;
-                    wa_ldsm(k_addr + k_off + jj * 16 * qst + c * 32, b00, b01, b10, b11);
-                    wa_mma(sc[2 * jj], h0, h1, h2, h3, b00, b01);
-                    wa_mma(sc[2 * jj], l0, l1, l2, l3, b00, b01);
-                    wa_mma(sc[2 * jj + 1], h0, h1, h2, h3, b10, b11);
-                    wa_mma(sc[2 * jj + 1], l0, l1, l2, l3, b10, b11);
+                    ms_ldsm(k_addr + k_off + jj * 16 * qst + c * 32, b00, b01, b10, b11);
+                    ms_mma(sc[2 * jj], h0, h1, h2, h3, b00, b01);
+                    ms_mma(sc[2 * jj], l0, l1, l2, l3, b00, b01);
+                    ms_mma(sc[2 * jj + 1], h0, h1, h2, h3, b10, b11);
+                    ms_mma(sc[2 * jj + 1], l0, l1, l2, l3, b10, b11);
                 }
             }
             float corr[2];
@@ -506,7 +443,7 @@ __device__ __forceinline__ void wattn_chunk_body(const lb_wattn_params& p) {
                 for (int j = 0; j < 4; ++j) {
                     const float p0 = exp2f(sc[j][2 * i] - m_new), p1 = exp2f(sc[j][2 * i + 1] - m_new);
                     ps += p0 + p1;
-                    wa_split(p0, p1, ph[j][i], pl[j][i]);
+                    ms_split(p0, p1, ph[j][i], pl[j][i]);
                 }
                 ps += __shfl_xor_sync(0xffffffffu, ps, 1);
                 ps += __shfl_xor_sync(0xffffffffu, ps, 2);
@@ -521,11 +458,11 @@ __device__ __forceinline__ void wattn_chunk_body(const lb_wattn_params& p) {
 #pragma unroll
                     for (int kk = 0; kk < 2; ++kk) {
                         uint32_t v0, v1, v2, v3;
-                        wa_ldsm_t(v_addr + v_off + kk * 16 * vst + nb * 16, v0, v1, v2, v3);
-                        wa_mma(acc[nb], ph[2 * kk][0], ph[2 * kk][1], ph[2 * kk + 1][0], ph[2 * kk + 1][1], v0, v1);
-                        wa_mma(acc[nb], pl[2 * kk][0], pl[2 * kk][1], pl[2 * kk + 1][0], pl[2 * kk + 1][1], v0, v1);
-                        wa_mma(acc[nb + 1], ph[2 * kk][0], ph[2 * kk][1], ph[2 * kk + 1][0], ph[2 * kk + 1][1], v2, v3);
-                        wa_mma(acc[nb + 1], pl[2 * kk][0], pl[2 * kk][1], pl[2 * kk + 1][0], pl[2 * kk + 1][1], v2, v3);
+                        ms_ldsm_t(v_addr + v_off + kk * 16 * vst + nb * 16, v0, v1, v2, v3);
+                        ms_mma(acc[nb], ph[2 * kk][0], ph[2 * kk][1], ph[2 * kk + 1][0], ph[2 * kk + 1][1], v0, v1);
+                        ms_mma(acc[nb], pl[2 * kk][0], pl[2 * kk][1], pl[2 * kk + 1][0], pl[2 * kk + 1][1], v0, v1);
+                        ms_mma(acc[nb + 1], ph[2 * kk][0], ph[2 * kk][1], ph[2 * kk + 1][0], ph[2 * kk + 1][1], v2, v3);
+                        ms_mma(acc[nb + 1], pl[2 * kk][0], pl[2 * kk][1], pl[2 * kk + 1][0], pl[2 * kk + 1][1], v2, v3);
                     }
                 }
             }
