@@ -742,6 +742,35 @@ NUFALORN_SIZES = {  # width, feed-forward, heads, KV heads, head size, and the h
 }
 
 
+def layer_list_rows(args, ctx, m, n_prompt, vocab, steps, peak, tflops, algo_bytes, macs_per_token, name):
+    """prompt and decode throughput of an open model: one row of the table"""
+    import lithos_b200 as lb
+    toks = [int(t) for t in lb.fill_u32(n_prompt, 3, 999) % vocab]
+    m.prefill(toks)                     # untimed: allocates the prompt-pass buffers, brings the clocks up
+    m.prefill(toks)
+    best = None
+    for _ in range(5):
+        m.reset_state()
+        ctx.timer_start()
+        m.prefill(toks)
+        ms = ctx.timer_stop()
+        best = ms if best is None or ms < best else best
+    m.capture()
+    m.set_input(1, n_prompt)
+    m.replay(max(args.warmup, 10))
+    ctx.sync()
+    ctx.reset_launches()
+    ctx.timer_start()
+    m.replay(steps)
+    ms = ctx.timer_stop() / steps
+    assert ctx.device_status() == 0
+    return {"model": name, "decode_ms": round(ms, 4), "decode_tok_s": round(1e3 / ms, 1), "decode_bytes": algo_bytes,
+            "decode_frac_of_measured_hbm": round(algo_bytes / (ms * 1e-3) / 1e9 / peak, 3), "kernels_per_step": m.step_kernels,
+            "prompt_ms": round(best, 3), "prompt_tok_s": round(n_prompt / best * 1e3),
+            "prompt_tflops": round(2 * macs_per_token * n_prompt / best / 1e9, 1),
+            "prompt_frac_of_measured_bf16": round(2 * macs_per_token * n_prompt / best / 1e9 / tflops, 3)}
+
+
 def bench_nufalorn(args, local):
     import lithos_b200 as lb
     from lithos_b200 import model as M
@@ -758,31 +787,7 @@ def bench_nufalorn(args, local):
     rows = []
 
     def timed(m, algo_weights, state_bytes, attended_bytes, macs_per_token, name):
-        toks = [int(t) for t in lb.fill_u32(n_prompt, 3, 999) % vocab]
-        m.prefill(toks)                     # untimed: allocates the prompt-pass buffers, brings the clocks up
-        m.prefill(toks)
-        best = None
-        for _ in range(5):
-            m.reset_state()
-            ctx.timer_start()
-            m.prefill(toks)
-            ms = ctx.timer_stop()
-            best = ms if best is None or ms < best else best
-        m.capture()
-        m.set_input(1, n_prompt)
-        m.replay(max(args.warmup, 10))
-        ctx.sync()
-        ctx.reset_launches()
-        ctx.timer_start()
-        m.replay(steps)
-        ms = ctx.timer_stop() / steps
-        assert ctx.device_status() == 0
-        by = algo_weights + state_bytes + attended_bytes
-        rows.append({"model": name, "decode_ms": round(ms, 4), "decode_tok_s": round(1e3 / ms, 1), "decode_bytes": by,
-                     "decode_frac_of_measured_hbm": round(by / (ms * 1e-3) / 1e9 / peak, 3), "kernels_per_step": m.step_kernels,
-                     "prompt_ms": round(best, 3), "prompt_tok_s": round(n_prompt / best * 1e3),
-                     "prompt_tflops": round(2 * macs_per_token * n_prompt / best / 1e9, 1),
-                     "prompt_frac_of_measured_bf16": round(2 * macs_per_token * n_prompt / best / 1e9 / tflops, 3)})
+        rows.append(layer_list_rows(args, ctx, m, n_prompt, vocab, steps, peak, tflops, algo_weights + state_bytes + attended_bytes, macs_per_token, name))
 
     for key, (W, F, H, KV, D, (dk, dv, fq, fkv)) in NUFALORN_SIZES.items():
         if args.sizes and key not in args.sizes.split(","):
@@ -808,6 +813,88 @@ def bench_nufalorn(args, local):
     clocks = sampler.stop()
     ctx.close()
     return {"metric": "decode and prompt throughput, Nufalorn beside the int4 hybrid of equal size", "value": rows[0]["decode_tok_s"], "unit": "tok/s",
+            "n_gpus": 1, "higher_is_better": True, "data": "synthetic", "rows": rows, "clocks": clocks,
+            "peaks": {"hbm_gbs": peak, "bf16_tflops_sustained": tflops, "source": which},
+            "config": {"prompt_tokens": n_prompt, "decode_steps": steps, "vocab": vocab, "attention_block": block,
+                       "timing": "CUDA events; decode: graph replays back to back; prompt: best of 5; weights of a step exceed L2"}}
+
+
+# ------------------------------------------------------------------------------------------
+# workload "vobunex": the same measurement of the other layer-list design, beside Nufalorn at equal width, dense feed-forward and depth
+# ------------------------------------------------------------------------------------------
+VOBUNEX_SIZES = {  # width, dense feed-forward, attention heads, query latent, experts, experts per token, expert width; Nufalorn's heads and KV heads
+    "5120": (5120, 17408, 40, 1536, 32, 6, 1536, (40, 8)),
+    "4096": (4096, 12288, 32, 1536, 32, 6, 1536, (32, 8)),
+    "2048": (2048, 8192, 16, 1024, 64, 6, 1408, (16, 4)),
+}
+
+
+def vobunex_config(width, ff, heads, q_rank, experts, top, expert_ff, layers, vocab):
+    """one period = Mamba-2 + dense, Mamba-2 + experts, latent attention + experts, Mamba-2 + dense; inner width twice the model's"""
+    rot = {"base": 10000.0, "dims": 64, "scaling": {"factor": 40.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
+    att = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": q_rank, "kv_rank": 512, "scale": 192 ** -0.5, "rot": rot}
+    ssm = {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff, "limit": 7.0}, "router": {"experts": experts, "top": top}}
+    dense = {"kind": "dense", "ff": ff}
+    out = []
+    for i in range(layers):
+        k = i % 4
+        out.append({"type": "latent_attention" if k == 2 else "mamba2", "mixer": dict(att if k == 2 else ssm), "mlp": dict(dense if k in (0, 3) else moe)})
+    return {"architecture": "Vobunex", "layers": out, "width": width, "vocab": vocab, "norm": {"eps": 1e-5},
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 1031, "mul_cur": 7}}}
+
+
+def vobunex_work(cfg):
+    """(weight elements a token passes, the LM head not counted; state bytes a step reads and writes; cache bytes per position seen)"""
+    W, macs, state, cache = cfg["width"], 0, 0, 0
+    for layer in cfg["layers"]:
+        m, f = layer["mixer"], layer["mlp"]
+        n = m["heads"] * m["vdim"]
+        if layer["type"] == "mamba2":
+            macs += W * (2 * n + 2 * m["groups"] * m["state"] + m["heads"]) + n * W
+            state += 2 * 4 * m["heads"] * m["state"] * m["vdim"]
+        else:
+            macs += (W * (m["q_rank"] + m["kv_rank"] + m["rot_dim"]) + m["q_rank"] * m["heads"] * (m["dim"] + m["rot_dim"]) +
+                     m["kv_rank"] * m["heads"] * (m["dim"] + m["vdim"]) + n * W)
+            cache += 2 * (m["kv_rank"] + m["rot_dim"])
+        macs += 2 * W * f["ff"] if f["kind"] == "dense" else 3 * W * f["expert"]["ff"] * f["router"]["top"]
+    return macs, state, cache
+
+
+def bench_vobunex(args, local):
+    import lithos_b200 as lb
+    from lithos_b200 import model as M
+    peak, which = measured_hbm_peak()
+    try:
+        tflops = float(json.loads(PEAKS_FILE.read_text())["bf16_tflops_sustained"])
+    except Exception:
+        tflops = 1400.0
+    n_layers, n_prompt, vocab, block = (8 if args.layers == 64 else args.layers), args.prompt, 32768, 2048
+    steps = min(args.steps, 200)
+    ctx = lb.Context(local)
+    sampler = ClockSampler(local)
+    sampler.start()
+    rows = []
+    for key, (W, F, H, QR, E, top, EF, (nh, nkv)) in VOBUNEX_SIZES.items():
+        if args.sizes and key not in args.sizes.split(","):
+            continue
+        if args.only in ("", "vobunex"):
+            cfg = vobunex_config(W, F, H, QR, E, top, EF, n_layers, vocab)
+            m = M.Model.open_synthetic(ctx, cfg, n_prompt + steps + 512, "bfloat16", 5)
+            macs, state, cache = vobunex_work(cfg)
+            by = 2 * (macs + vocab * W) + state + cache * (n_prompt + steps // 2)
+            rows.append(layer_list_rows(args, ctx, m, n_prompt, vocab, steps, peak, tflops, by, macs, f"Vobunex {W}x{F}, {E} experts of {EF}, {n_layers} layers, bf16 weights"))
+            m.close()
+        if args.only in ("", "nufalorn"):
+            cfg = nufalorn_config(W, F, nh, nkv, 128, n_layers, vocab, block)
+            m = M.Model.open_synthetic(ctx, cfg, n_prompt + steps + 512, "bfloat16", 5)
+            n_att = sum(l["type"] == "attention" for l in cfg["layers"])
+            by = m.weight_bytes + (n_layers - n_att) * 2 * nh * 128 * 128 * 4 + n_att * ((n_prompt % block) + steps // 2 + 1) * nkv * 128 * 2 * 2
+            rows.append(layer_list_rows(args, ctx, m, n_prompt, vocab, steps, peak, tflops, by, m.weight_bytes // 2 - vocab * W, f"Nufalorn {W}x{F}, {n_layers} layers, bf16 weights"))
+            m.close()
+    clocks = sampler.stop()
+    ctx.close()
+    return {"metric": "decode and prompt throughput, Vobunex beside Nufalorn of equal size", "value": rows[0]["decode_tok_s"], "unit": "tok/s",
             "n_gpus": 1, "higher_is_better": True, "data": "synthetic", "rows": rows, "clocks": clocks,
             "peaks": {"hbm_gbs": peak, "bf16_tflops_sustained": tflops, "source": which},
             "config": {"prompt_tokens": n_prompt, "decode_steps": steps, "vocab": vocab, "attention_block": block,
@@ -986,16 +1073,16 @@ def main():
     ap.add_argument("--steps", type=int, default=None)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="native", choices=["native", "reference"])
-    ap.add_argument("--workload", default="decode", choices=["decode", "gemv", "chain", "batched", "timeline", "small", "prompt", "nufalorn"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "gemv", "chain", "batched", "timeline", "small", "prompt", "nufalorn", "vobunex"],
                     help="decode: the benchmark; gemv: config 0 alone; chain: the decode step's four GEMVs between two token "
                          "mixers as persistent gemv_chain launches alone (the small case used for ncu captures); small: the "
                          "one-figure measurements of configs 0, 1 and 2 alone (the ncu target for the DeltaNet and attention kernels)")
     ap.add_argument("--layers", type=int, default=64, help="decode workload: number of layers (64 = the benchmark definition)")
     ap.add_argument("--batched-shapes", default="", help="batched workload: comma-separated substrings of the shape names to run (default all)")
     ap.add_argument("--batched-batches", default="1,4,16,32,64,128,256", help="batched workload: batch sizes")
-    ap.add_argument("--sizes", default="", help="nufalorn workload: comma-separated widths to run (default all)")
-    ap.add_argument("--only", default="", choices=["", "nufalorn", "hybrid"], help="nufalorn workload: one of the two models")
-    ap.add_argument("--prompt", type=int, default=4096, help="nufalorn workload: prompt tokens")
+    ap.add_argument("--sizes", default="", help="nufalorn, vobunex workloads: comma-separated widths to run (default all)")
+    ap.add_argument("--only", default="", choices=["", "nufalorn", "vobunex", "hybrid"], help="nufalorn, vobunex workloads: one of the two models")
+    ap.add_argument("--prompt", type=int, default=4096, help="nufalorn, vobunex workloads: prompt tokens")
     ap.add_argument("--seed", type=int, default=20260413)
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     ap.add_argument("--prefill", action="store_true", help="decode workload, 1 GPU: build the 4096-token state by running a seeded random prompt through "
@@ -1030,8 +1117,8 @@ def main():
         if rank == 0:
             print(json.dumps(out), flush=True)
         return
-    if args.workload in ("chain", "batched", "prompt", "nufalorn"):
-        out = {"chain": bench_chain, "batched": bench_batched, "prompt": bench_prompt_chunks, "nufalorn": bench_nufalorn}[args.workload](args, local)
+    if args.workload in ("chain", "batched", "prompt", "nufalorn", "vobunex"):
+        out = {"chain": bench_chain, "batched": bench_batched, "prompt": bench_prompt_chunks, "nufalorn": bench_nufalorn, "vobunex": bench_vobunex}[args.workload](args, local)
         if rank == 0:
             print(json.dumps(out), flush=True)
         return
