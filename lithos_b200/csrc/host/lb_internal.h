@@ -121,9 +121,13 @@ int lb_driver_load(char* err, size_t errlen); /* LB_OK or LB_ERR_NO_DRIVER */
     X(pf_attn_prepare)                \
     X(pf_attn_chunk)                  \
     X(rows_gemv)                      \
+    X(rows_gemv_rms)                  \
+    X(rows_gemv_ln)                   \
+    X(rows_gemv_experts)              \
     X(gemm_bf16_tc)                   \
     X(gemm_f32_simt)                  \
     X(norm_rows2)                     \
+    X(norm_rows_any)                  \
     X(moe_plan)                       \
     X(wattn_rows_b2n2)                \
     X(wattn_rows_b4n2)                \

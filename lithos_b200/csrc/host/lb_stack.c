@@ -475,9 +475,12 @@ static void fill_decay(const lb_model* m, int i, lb_decay_params2* p, CUdevicept
  * ring fewer than five stages (the mixer's part must lie in the first half) */
 static int launch_rows(lb_model* m, lb_rows_gemv_params* p) {
     lb_ctx* c = m->c;
+    const int normed = p->x_mode == LB_RG_X_NORM;
+    const int kernel = p->sel ? LBK_rows_gemv_experts : normed && p->norm == LB_NORM_LAYER ? LBK_rows_gemv_ln : normed && p->norm == LB_NORM_RMS ? LBK_rows_gemv_rms : LBK_rows_gemv;
     int P = 0;
+    if (p->sel && normed && p->norm != LB_NORM_LAYER) return lb_fail(c, LB_ERR_INVALID, "model: experts behind another norm than layer norm");
     for (int i = 0; i < p->n_mat; i++) P += (p->mat[i].rows + 1) / 2;
-    const int n_vec = p->x_mode == LB_RG_X_NORM ? p->n_mat : 1, limit = c->max_smem_optin - ((c->fn_static_smem[LBK_rows_gemv] + 1023) & ~1023);
+    const int n_vec = p->x_mode == LB_RG_X_NORM ? p->n_mat : 1, limit = c->max_smem_optin - ((c->fn_static_smem[kernel] + 1023) & ~1023);
     const int by_columns = p->sel && p->x_mode == LB_RG_X_CAT; /* experts side by side along K */
     if (!p->sel) p->parts = 1;
     if (!by_columns) p->k_part = p->K;
@@ -501,7 +504,7 @@ static int launch_rows(lb_model* m, lb_rows_gemv_params* p) {
     if (ks > 1 + can_halve) ks = 1 + can_halve;
     if (p->stages < 1) return lb_fail(c, LB_ERR_INVALID, "model: a row of %d columns does not fit the decode step's shared memory", p->K);
     void* params[] = {p};
-    return lb_launch_cluster(c, LBK_rows_gemv, (unsigned)(c->sm_count / ks), (unsigned)ks, 1, LB_RG_THREADS, (unsigned)smem, params, 1, (unsigned)ks);
+    return lb_launch_cluster(c, kernel, (unsigned)(c->sm_count / ks), (unsigned)ks, 1, LB_RG_THREADS, (unsigned)smem, params, 1, (unsigned)ks);
 }
 
 /* Tokens per product tile, and what a product then costs in units of one wave of 256-token tiles: fewer tokens per tile make more tiles
@@ -787,7 +790,8 @@ static lb_norm2_params norm_params(const lb_model* m, CUdeviceptr x, CUdeviceptr
 }
 static int launch_norm(lb_model* m, lb_norm2_params* p, int T) {
     void* params[] = {p};
-    return lb_launch(m->c, LBK_norm_rows2, (unsigned)T, 1, 1, 256, 0, params, 1);
+    const int plain = p->norm == LB_NORM_RMS_1P && p->ld_x == p->width && !p->y && !p->scatter;
+    return lb_launch(m->c, plain ? LBK_norm_rows2 : LBK_norm_rows_any, (unsigned)T, 1, 1, 256, 0, params, 1);
 }
 static int norm_rows(lb_model* m, CUdeviceptr x, CUdeviceptr w0, CUdeviceptr h0, CUdeviceptr w1, CUdeviceptr h1, int T) {
     lb_norm2_params p = norm_params(m, x, w0, 0, h0);

@@ -48,6 +48,56 @@ __device__ __forceinline__ float dg_clamp_glu(float gate, float up, float limit,
     return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
 }
 
+// a warp's 32 weight rows (lane: row n) x n_t tokens from t0 on: out of tensor memory, finished, stored
+template <int MODE>
+__device__ __forceinline__ void dg_finish(const lb_dgemm_params& p, int m, uint32_t acc, int n, int t0, int n_t, int ld) {
+    const int lane = threadIdx.x & 31;
+    const bool live = n < p.rows[m];
+    const int hn = MODE == LB_DY_HEADS ? n / p.head[m] : 0, col = MODE == LB_DY_HEADS ? hn * p.head_p[m] + (n - hn * p.head[m]) : n;
+    for (int c = 0; c < n_t; c += 16) {
+        uint32_t r[16];
+        tmem_ld16(acc + (uint32_t)c, r);
+        tmem_ld_wait();
+        if (MODE == LB_DY_HEADS || MODE == LB_DY_RELU2) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+                if (!live || c + j >= n_t) continue;
+                float v = __uint_as_float(r[j]);
+                if (MODE == LB_DY_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
+                const size_t o = (size_t)(t0 + c + j) * ld + col;
+                if (MODE == LB_DY_RELU2 && p.y_f32[m]) reinterpret_cast<float*>(p.y[m])[o] = v;
+                else reinterpret_cast<__nv_bfloat16*>(p.y[m])[o] = __float2bfloat16_rn(v);
+            }
+        } else if (MODE == LB_DY_RELU_GLU || MODE == LB_DY_CLAMP_GLU) {
+            const bool st = live && !(lane & 1);
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+                const float gate = __uint_as_float(r[j]), up = __uint_as_float(__shfl_xor_sync(0xffffffffu, r[j], 1));
+                const float v = MODE == LB_DY_RELU_GLU ? fmaxf(gate, 0.f) * up : dg_clamp_glu(gate, up, p.limit, p.alpha);
+                if (st && c + j < n_t) {
+                    const size_t o = (size_t)(t0 + c + j) * ld + (n >> 1);
+                    if (p.y_f32[m]) reinterpret_cast<float*>(p.y[m])[o] = v;
+                    else reinterpret_cast<__nv_bfloat16*>(p.y[m])[o] = __float2bfloat16_rn(v);
+                }
+            }
+        } else {
+            float* y = reinterpret_cast<float*>(p.y[m]) + (size_t)(t0 + c) * ld + n;
+            float old[16];
+            if (MODE == LB_DY_RESIDUAL) {
+#pragma unroll
+                for (int j = 0; j < 16; ++j) old[j] = live && c + j < n_t ? y[(size_t)j * ld] : 0.f;
+            }
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+                float v = __uint_as_float(r[j]);
+                if (MODE == LB_DY_RESIDUAL) v = fmaf(p.mult, v, old[j]);
+                else if (MODE == LB_DY_SOFTCAP && p.cap > 0.f) v = p.cap * tanhf(v / p.cap);
+                if (live && c + j < n_t) y[(size_t)j * ld] = v;
+            }
+        }
+    }
+}
+
 extern "C" __global__ void __launch_bounds__(LB_DG_THREADS, 1) gemm_bf16_tc(const __grid_constant__ lb_dgemm_params p) {
     extern __shared__ __align__(1024) unsigned char dg_sm[];
     __shared__ __align__(8) uint64_t bar_full[LB_DG_MAX_STAGES], bar_empty[LB_DG_MAX_STAGES], bar_acc[2], bar_free[2];
@@ -148,48 +198,15 @@ extern "C" __global__ void __launch_bounds__(LB_DG_THREADS, 1) gemm_bf16_tc(cons
             }
             tc_fence_after();
             const int mode = p.y_mode[m], ld = p.ld_y[m], n_t = min(NT, d.end - t0);
-            const bool live = n < p.rows[m];
-            const int hn = mode == LB_DY_HEADS ? n / p.head[m] : 0, hcol = hn * p.head_p[m] + (n - hn * p.head[m]);
-            for (int c = 0; c < n_t; c += 16) {
-                uint32_t r[16];
-                tmem_ld16(tmem + ((uint32_t)(32 * quad) << 16) + (uint32_t)(b * NT + c), r);
-                tmem_ld_wait();
-                if (mode == LB_DY_HEADS || mode == LB_DY_RELU2) {
-#pragma unroll
-                    for (int j = 0; j < 16; ++j) {
-                        if (!live || c + j >= n_t) continue;
-                        const float v = __uint_as_float(r[j]), v0 = fmaxf(v, 0.f);
-                        const size_t o = (size_t)(t0 + c + j) * ld + (mode == LB_DY_HEADS ? hcol : n);
-                        if (mode == LB_DY_RELU2 && p.y_f32[m]) reinterpret_cast<float*>(p.y[m])[o] = v0 * v0;
-                        else reinterpret_cast<__nv_bfloat16*>(p.y[m])[o] = __float2bfloat16_rn(mode == LB_DY_HEADS ? v : v0 * v0);
-                    }
-                } else if (mode == LB_DY_RELU_GLU || mode == LB_DY_CLAMP_GLU) {
-                    const bool st = live && !(lane & 1);
-#pragma unroll
-                    for (int j = 0; j < 16; ++j) {
-                        const float ga = __uint_as_float(r[j]), up = __uint_as_float(__shfl_xor_sync(0xffffffffu, r[j], 1));
-                        const float v = mode == LB_DY_RELU_GLU ? fmaxf(ga, 0.f) * up : dg_clamp_glu(ga, up, p.limit, p.alpha);
-                        if (st && c + j < n_t) {
-                            const size_t o = (size_t)(t0 + c + j) * ld + (n >> 1);
-                            if (p.y_f32[m]) reinterpret_cast<float*>(p.y[m])[o] = v;
-                            else reinterpret_cast<__nv_bfloat16*>(p.y[m])[o] = __float2bfloat16_rn(v);
-                        }
-                    }
-                } else {
-                    float* y = reinterpret_cast<float*>(p.y[m]) + (size_t)(t0 + c) * ld + n;
-                    float old[16];
-                    if (mode == LB_DY_RESIDUAL) {
-#pragma unroll
-                        for (int j = 0; j < 16; ++j) old[j] = live && c + j < n_t ? y[(size_t)j * ld] : 0.f;
-                    }
-#pragma unroll
-                    for (int j = 0; j < 16; ++j) {
-                        float v = __uint_as_float(r[j]);
-                        if (mode == LB_DY_RESIDUAL) v = fmaf(p.mult, v, old[j]);
-                        else if (mode == LB_DY_SOFTCAP && p.cap > 0.f) v = p.cap * tanhf(v / p.cap);
-                        if (live && c + j < n_t) y[(size_t)j * ld] = v;
-                    }
-                }
+            const uint32_t acc = tmem + ((uint32_t)(32 * quad) << 16) + (uint32_t)(b * NT);
+            switch (mode) {
+                case LB_DY_RELU_GLU: dg_finish<LB_DY_RELU_GLU>(p, m, acc, n, t0, n_t, ld); break;
+                case LB_DY_CLAMP_GLU: dg_finish<LB_DY_CLAMP_GLU>(p, m, acc, n, t0, n_t, ld); break;
+                case LB_DY_RELU2: dg_finish<LB_DY_RELU2>(p, m, acc, n, t0, n_t, ld); break;
+                case LB_DY_HEADS: dg_finish<LB_DY_HEADS>(p, m, acc, n, t0, n_t, ld); break;
+                case LB_DY_RESIDUAL: dg_finish<LB_DY_RESIDUAL>(p, m, acc, n, t0, n_t, ld); break;
+                case LB_DY_SOFTCAP: dg_finish<LB_DY_SOFTCAP>(p, m, acc, n, t0, n_t, ld); break;
+                default: dg_finish<LB_DY_STORE>(p, m, acc, n, t0, n_t, ld); break;
             }
             tc_fence_before();
             __syncwarp();
@@ -304,13 +321,16 @@ __device__ __forceinline__ void nr_store1(const lb_norm2_params& p, void* h, siz
     if (p.f32) reinterpret_cast<float*>(h)[o] = r;
     else reinterpret_cast<__nv_bfloat16*>(h)[o] = __float2bfloat16_rn(r);
 }
-extern "C" __global__ void __launch_bounds__(256, 4) norm_rows2(const __grid_constant__ lb_norm2_params p) {
+// ANY false: LB_NORM_RMS_1P of rows of `width`, nothing added, nothing scattered
+template <bool ANY>
+__device__ __forceinline__ void norm_rows2_body(const lb_norm2_params& p) {
     __shared__ float red[40];
     const int t = threadIdx.x, tok = blockIdx.x;
-    const bool quads = (p.width & 3) == 0 && (p.ld_x & 3) == 0 && (p.ld_y & 3) == 0 && p.width <= 4 * NR_Q * 256;
-    const float one = p.norm == LB_NORM_RMS_1P ? 1.0f : 0.0f;
+    const bool quads = (p.width & 3) == 0 && (!ANY || ((p.ld_x & 3) == 0 && (p.ld_y & 3) == 0)) && p.width <= 4 * NR_Q * 256;
+    const float one = !ANY || p.norm == LB_NORM_RMS_1P ? 1.0f : 0.0f;
+    const bool layer_norm = ANY && p.norm == LB_NORM_LAYER, adds = ANY && p.y, scatters = ANY && p.scatter;
     pdl_wait();
-    float* x = p.x + (size_t)tok * p.ld_x;
+    float* x = p.x + (size_t)tok * (ANY ? p.ld_x : p.width);
     float4 v[NR_Q];
     float mean = 0.f, ss = 0.f;
     if (quads) {
@@ -319,7 +339,7 @@ extern "C" __global__ void __launch_bounds__(256, 4) norm_rows2(const __grid_con
             const int i = 4 * (t + 256 * u);
             v[u] = i < p.width ? *reinterpret_cast<const float4*>(x + i) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
-        if (p.y) {
+        if (adds) {
 #pragma unroll
             for (int u = 0; u < NR_Q; ++u) {
                 const int i = 4 * (t + 256 * u);
@@ -335,7 +355,7 @@ extern "C" __global__ void __launch_bounds__(256, 4) norm_rows2(const __grid_con
                 *reinterpret_cast<float4*>(x + i) = v[u];
             }
         }
-        if (p.norm == LB_NORM_LAYER) {
+        if (layer_norm) {
 #pragma unroll
             for (int u = 0; u < NR_Q; ++u) mean += (v[u].x + v[u].y) + (v[u].z + v[u].w);
             mean = block_sum(mean, red) / (float)p.width;
@@ -346,9 +366,9 @@ extern "C" __global__ void __launch_bounds__(256, 4) norm_rows2(const __grid_con
 #pragma unroll
         for (int u = 0; u < NR_Q; ++u) ss += (v[u].x * v[u].x + v[u].y * v[u].y) + (v[u].z * v[u].z + v[u].w * v[u].w);
     } else {
-        if (p.y)
+        if (adds)
             for (int i = t; i < p.width; i += 256) x[i] = fmaf(p.y_mult, nr_added(p, tok, i), x[i]); // read again by this thread alone
-        if (p.norm == LB_NORM_LAYER) {
+        if (layer_norm) {
             for (int i = t; i < p.width; i += 256) mean += x[i];
             mean = block_sum(mean, red) / (float)p.width;
         }
@@ -361,8 +381,8 @@ extern "C" __global__ void __launch_bounds__(256, 4) norm_rows2(const __grid_con
     ss = block_sum(ss, red);
     const float rinv = 1.0f / sqrtf(ss / (float)p.width + p.eps);
     pdl_launch_dependents();
-    if (!p.h[0]) return; // only the sum was asked for
-    const int copies = p.scatter ? p.top : 1;
+    if (ANY && !p.h[0]) return; // only the sum was asked for
+    const int copies = scatters ? p.top : 1;
     if (quads) {
 #pragma unroll
         for (int u = 0; u < NR_Q; ++u) {
@@ -373,11 +393,11 @@ extern "C" __global__ void __launch_bounds__(256, 4) norm_rows2(const __grid_con
                 if (!p.h[e]) continue;
                 const float4 w = nr_quad(p.w[e], i);
                 float4 r = make_float4(v[u].x * rinv * (one + w.x), v[u].y * rinv * (one + w.y), v[u].z * rinv * (one + w.z), v[u].w * rinv * (one + w.w));
-                if (p.norm == LB_NORM_LAYER) {
+                if (layer_norm) {
                     const float4 b = nr_quad(p.b[e], i);
                     r.x += b.x; r.y += b.y; r.z += b.z; r.w += b.w;
                 }
-                for (int k = 0; k < copies; ++k) nr_store4(p, p.h[e], (size_t)(p.scatter ? p.scatter[(size_t)tok * p.top + k] : tok) * p.ld + i, r);
+                for (int k = 0; k < copies; ++k) nr_store4(p, p.h[e], (size_t)(scatters ? p.scatter[(size_t)tok * p.top + k] : tok) * p.ld + i, r);
             }
         }
     }
@@ -387,11 +407,13 @@ extern "C" __global__ void __launch_bounds__(256, 4) norm_rows2(const __grid_con
         for (int e = 0; e < 2; ++e) {
             if (!p.h[e]) continue;
             float r = i < p.width ? xv * (one + bf16_bits_to_f32(p.w[e][i])) : 0.f;
-            if (p.norm == LB_NORM_LAYER && i < p.width) r += bf16_bits_to_f32(p.b[e][i]);
-            for (int k = 0; k < copies; ++k) nr_store1(p, p.h[e], (size_t)(p.scatter ? p.scatter[(size_t)tok * p.top + k] : tok) * p.ld + i, r);
+            if (layer_norm && i < p.width) r += bf16_bits_to_f32(p.b[e][i]);
+            for (int k = 0; k < copies; ++k) nr_store1(p, p.h[e], (size_t)(scatters ? p.scatter[(size_t)tok * p.top + k] : tok) * p.ld + i, r);
         }
     }
 }
+extern "C" __global__ void __launch_bounds__(256, 4) norm_rows2(const __grid_constant__ lb_norm2_params p) { norm_rows2_body<false>(p); }
+extern "C" __global__ void __launch_bounds__(256, 4) norm_rows_any(const __grid_constant__ lb_norm2_params p) { norm_rows2_body<true>(p); }
 
 // The chunk's (token, expert) assignments sorted by expert: the row of every assignment, and the token tiles (of at most NT assignments of one
 // expert).  One CTA of 1024 threads per launch.

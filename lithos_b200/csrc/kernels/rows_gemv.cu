@@ -24,7 +24,9 @@ __device__ __forceinline__ float2 rg_ld_cluster(const float* local_ptr, uint32_t
 }
 __device__ __forceinline__ float rg_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 
-extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const __grid_constant__ lb_rows_gemv_params p) {
+// NORM: the norm of LB_RG_X_NORM; SEL: matrices are stacks of experts
+template <int NORM, bool SEL>
+__device__ __forceinline__ void rows_gemv_body(const lb_rows_gemv_params& p) {
     extern __shared__ __align__(16) unsigned char rg_sm[];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int G = gridDim.x, c = blockIdx.x, S = p.stages;
@@ -47,7 +49,7 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
     if (tid == 0) mbar_init(&bars[LB_RG_WARPS * S], 1);
     mbar_fence_init();
     __shared__ int sel_s[LB_RG_MAX_PARTS];
-    if (p.sel && tid < p.parts) sel_s[tid] = p.sel[(size_t)p.sel_row[0] * p.parts + tid];
+    if (SEL && tid < p.parts) sel_s[tid] = p.sel[(size_t)p.sel_row[0] * p.parts + tid];
     __syncthreads();
 
     // the warp's stages: items warp, warp + 8, ... (item = pair * split + piece), segments of the item in order
@@ -56,17 +58,17 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
     auto row_ptr = [&](int pair, int& mi) -> const uint16_t* {
         const int g = c + pair * G;
         mi = g >= pairs0;
-        if (p.sel && p.x_mode == LB_RG_X_NORM) { // the parts' rows one after the other, each part's from its expert
+        if (SEL && p.x_mode == LB_RG_X_NORM) { // the parts' rows one after the other, each part's from its expert
             const int part_pairs = p.sel_rows >> 1, e = g / part_pairs;
             return p.mat[0].w + ((size_t)sel_s[e] * part_pairs + (g - e * part_pairs)) * 2 * p.K;
         }
         return mi ? p.mat[1].w + (size_t)(g - pairs0) * 2 * p.K : p.mat[0].w + (size_t)g * 2 * p.K;
     };
     // a row segment: its first column and length; with experts side by side along K a row is in pieces of k_part columns
-    const bool sel_k = p.sel && p.x_mode == LB_RG_X_CAT;
+    const bool sel_k = SEL && p.x_mode == LB_RG_X_CAT;
     const size_t row_step = sel_k ? p.k_part : p.K, expert_pairs = sel_k ? (size_t)((p.mat[0].rows + 1) >> 1) : 0;
     auto segment = [&](int seg, int& col, int& len, int& e) {
-        if (sel_k) {
+        if (SEL && sel_k) {
             e = seg / p.segs_part;
             const int off = (seg - e * p.segs_part) * LB_RG_SEG;
             col = e * p.k_part + off;
@@ -83,7 +85,7 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
             const int pair = split == 1 ? r_item : r_item / split, seg = seg_lo + (r_item - pair * split) * spp + r_seg;
             int mi, col, len, e = 0;
             segment(seg, col, len, e);
-            const uint16_t* w = sel_k ? p.mat[0].w + ((size_t)sel_s[e] * expert_pairs + (c + pair * G)) * 2 * p.k_part + (col - e * p.k_part) : row_ptr(pair, mi) + col;
+            const uint16_t* w = SEL && sel_k ? p.mat[0].w + ((size_t)sel_s[e] * expert_pairs + (c + pair * G)) * 2 * p.k_part + (col - e * p.k_part) : row_ptr(pair, mi) + col;
             const uint32_t bytes = (uint32_t)len * 2u;
             unsigned char* dst = ring + (size_t)(warp * S + r_slot) * (LB_RG_SEG * 4);
             uint64_t* bar = &bars[warp * S + r_slot];
@@ -98,7 +100,7 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
 
     // the norm weights are constants too: a thread's first 8 quads of them (of the two vectors, or weight and bias of one) come in before
     // the wait
-    const bool layer_norm = p.norm == LB_NORM_LAYER;
+    constexpr bool layer_norm = NORM == LB_NORM_LAYER;
     const uint16_t* second = n_vec > 1 ? p.mat[1].norm_w : layer_norm ? p.mat[0].norm_b : nullptr;
     const bool quads = (p.width & 3) == 0;
     uint2 w_pre[2][8];
@@ -145,7 +147,7 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
             }
         }
         ss = block_sum(ss, red);
-        const float rinv = 1.0f / sqrtf(ss / (float)p.width + p.eps), one = p.norm == LB_NORM_RMS_1P ? 1.0f : 0.0f;
+        const float rinv = 1.0f / sqrtf(ss / (float)p.width + p.eps), one = NORM == LB_NORM_RMS_1P ? 1.0f : 0.0f;
         if (quads) {
             auto quad = [](uint2 w) {
                 return make_float4(__uint_as_float(w.x << 16), __uint_as_float(w.x & 0xffff0000u), __uint_as_float(w.y << 16), __uint_as_float(w.y & 0xffff0000u));
@@ -326,7 +328,7 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
         if (M.y_mode == LB_DY_RELU_GLU) {
             M.y[n >> 1] = fmaxf(r[0], 0.f) * r[1];
         } else if (M.y_mode == LB_DY_CLAMP_GLU) {
-            const int part = p.sel ? n / p.sel_rows : 0, i = (n - part * p.sel_rows) >> 1;
+            const int part = SEL ? n / p.sel_rows : 0, i = (n - part * p.sel_rows) >> 1;
             const float ga = fminf(r[0], p.limit), up = fminf(fmaxf(r[1], -p.limit), p.limit);
             M.y[(size_t)part * p.y_part + i] = ga * rg_sigmoid(p.alpha * ga) * (up + 1.0f);
         } else {
@@ -361,3 +363,11 @@ extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) rows_gemv(const _
     }
     if (KS > 1) rg_cluster_sync(); // nobody leaves while the other CTA still reads its sums
 }
+#define RG_KERNEL(name, NORM, SEL)                                                                                                     \
+    extern "C" __global__ void __launch_bounds__(LB_RG_THREADS, 1) name(const __grid_constant__ lb_rows_gemv_params p) { \
+        rows_gemv_body<NORM, SEL>(p);                                                                                                  \
+    }
+RG_KERNEL(rows_gemv, LB_NORM_RMS_1P, false)
+RG_KERNEL(rows_gemv_rms, LB_NORM_RMS, false)
+RG_KERNEL(rows_gemv_ln, LB_NORM_LAYER, false)
+RG_KERNEL(rows_gemv_experts, LB_NORM_LAYER, true)
