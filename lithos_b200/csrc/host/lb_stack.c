@@ -23,6 +23,7 @@
 #include <math.h>
 
 #define ST_CHUNK 1024 /* largest chunk of a prompt; stack_chunk picks the model's */
+#define ST_CHUNK_EXPERTS 2048 /* ... where the weights of experts are read once per chunk */
 #define ST_STREAMS 4
 #define ST_LAT_ABSORB 16 /* latent attention: portions of fewer tokens do not make keys and values of every cached position */
 #define ST_MOE_TILE 64 /* token tile of the fp32 expert products */
@@ -854,7 +855,7 @@ static int pf_ssm(lb_model* m, pf_set* w, int i, int pos0, int T) {
     void* params[] = {&p};
     LB_TRY(lb_launch(c, LBK_ssm_conv, (unsigned)((p.ld_xbc + D->heads + 255) / 256), (unsigned)((T + 7) / 8), 1, 256, 0, params, 1));
     static const int k_f32[3] = {LBK_ssm_scan_f32_64, LBK_ssm_scan_f32_128, LBK_ssm_scan_f32_256}, k_tc[3] = {LBK_ssm_chunk_64, LBK_ssm_chunk_128, LBK_ssm_chunk_256};
-    const int row = 2 * L->N_p + 16, smem = 2 * LB_SSM_SEG * row + 4 * LB_SSM_SEG * 80 + 3 * L->N_p * 80 + 2 * LB_SSM_SEG * 4;
+    const int row = 2 * L->N_p + 16, smem = 2 * LB_SSM_SEG * row + (row >= 240 ? 1 : 4) * LB_SSM_SEG * 80 + 3 * L->N_p * 80 + 2 * LB_SSM_SEG * 4; /* as ssm_chunk lays it out */
     LB_TRY(lb_launch(c, (S->esz == 4 ? k_f32 : k_tc)[state_size(D)], (unsigned)D->heads, (unsigned)(L->V_p / LB_SSM_COLS), 1, 128, S->esz == 4 ? 0u : (unsigned)smem, params, 1));
     return lb_launch(c, LBK_ssm_finish, (unsigned)T, (unsigned)D->norm_groups, 1, 128, (unsigned)(L->n_mix / D->norm_groups * 4), params, 1);
 }
@@ -1039,21 +1040,32 @@ static void stack_destroy(lb_model* m) {
 static const lb_arch k_stack = {"stack", ST_STREAMS, stack_reset_state, stack_snapshot, stack_state_ptr, stack_step_layers, stack_head,
                                 stack_head_ctas, stack_head_rows, stack_pf_sizes, stack_pf_layer, stack_destroy};
 
+/* the expert products of a chunk in the units of product_cost: full tiles (the rate does not fall as much as a dense product's, the tiles of an
+ * expert read the same operands), or the time to read every expert's weights from HBM (a wave of tiles takes as long as HBM_ROWS rows of them) */
+#define HBM_ROWS 14000.0
+static double experts_cost(const lb_model* m, const lb_stack_layer* D, int rows, int K, int T) {
+    const stack_t* S = S_of(m);
+    const int nt = moe_tile(S, D, T), tiles = D->experts * ((T * D->top / D->experts + nt - 1) / nt) * ((rows + LB_DG_ROWS - 1) / LB_DG_ROWS);
+    const double flops = (double)((tiles + m->c->sm_count - 1) / m->c->sm_count) * (nt >= 256 ? 1.0 : nt >= 128 ? 0.55 : 0.36), bytes = D->experts * (double)rows / HBM_ROWS;
+    return K * (flops > bytes ? flops : bytes);
+}
+
 /* tokens per prompt chunk: the multiple of 256 whose products fill whole waves of SMs best */
 static int stack_chunk(const lb_model* m) {
     const stack_t* S = S_of(m);
     double best = 1e30;
     int chunk = 256;
     if (S->esz == 4 && S->max_latq) return chunk; /* an absorbed chunk keeps a latent query per token and head */
-    if (S->max_top) return ST_CHUNK;              /* the more tokens, the more of them an expert's weights serve */
-    for (int T = 256; T <= ST_CHUNK; T += 256) {
+    for (int T = 256; T <= (S->max_top ? ST_CHUNK_EXPERTS : ST_CHUNK); T += 256) {
         double cost = 0;
         for (int i = 0; i < S->d.n_layers; i++) {
             const st_layer* L = &S->L[i];
             int nt;
             if (S->d.serial) {
                 const st_mat* w[] = {&L->in, &L->uq, &L->out, &L->ff, &L->down};
-                for (int k = 0; k < 5; k++)
+                const int moe = has_experts(S, i);
+                if (moe) cost += experts_cost(m, &S->d.layer[i], 2 * S->d.layer[i].ff, L->ff.K, T) + experts_cost(m, &S->d.layer[i], S->d.width, L->down.K, T);
+                for (int k = 0; k < (moe ? 3 : 5); k++)
                     if (w[k]->w) cost += w[k]->K * product_cost(m->c, (w[k]->rows + LB_DG_ROWS - 1) / LB_DG_ROWS, T, &nt);
                 continue;
             }

@@ -423,7 +423,18 @@ extern "C" __global__ void __launch_bounds__(1024) moe_plan(const __grid_constan
     count[t] = 0;
     __syncthreads();
     pdl_wait(); // the buffers written here may still be read by the kernels before
-    for (int a = t; a < n; a += 1024) p.place[a] = atomicAdd(&count[p.table[(size_t)p.tokens[a / p.top] * p.top + a % p.top]], 1);
+    auto expert = [&](int a) {
+        const int s = a / p.top;
+        return p.table[(size_t)p.tokens[s] * p.top + (a - s * p.top)];
+    };
+    for (int a0 = t; a0 < n; a0 += 8 * 1024) { // the reads of eight assignments, then their places among their experts' ones
+        int e[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) e[k] = a0 + k * 1024 < n ? expert(a0 + k * 1024) : -1;
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+            if (e[k] >= 0) p.place[a0 + k * 1024] = atomicAdd(&count[e[k]], 1);
+    }
     __syncthreads();
     // exclusive sums over experts of assignments and of tiles
     const int c = t < p.experts ? count[t] : 0, nt = (c + p.NT - 1) / p.NT;
@@ -442,6 +453,16 @@ extern "C" __global__ void __launch_bounds__(1024) moe_plan(const __grid_constan
     if (t == 1023) p.n_tiles[0] = bt + it;
     for (int k = 0; k < nt; ++k) reinterpret_cast<int4*>(p.tiles)[tile0[t] + k] = make_int4(t, first[t] + k * p.NT, first[t] + c, 0);
     __syncthreads();
-    for (int a = t; a < n; a += 1024) p.place[a] += first[p.table[(size_t)p.tokens[a / p.top] * p.top + a % p.top]];
+    for (int a0 = t; a0 < n; a0 += 8 * 1024) {
+        int e[8], q[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+            e[k] = a0 + k * 1024 < n ? expert(a0 + k * 1024) : -1;
+            q[k] = e[k] >= 0 ? p.place[a0 + k * 1024] : 0;
+        }
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+            if (e[k] >= 0) p.place[a0 + k * 1024] = q[k] + first[e[k]];
+    }
     pdl_launch_dependents();
 }

@@ -132,22 +132,27 @@ __device__ __forceinline__ void lat_rows_body(const lb_latent_params& p) {
     // rows of a block with old <= (row >= pos0) <= new...: rows before pos0 exist since an earlier step
     auto stage = [&](int b, bool old_rows, bool new_rows) {
         unsigned char* dst = kv_s + (p.stages > 1 ? b & 1 : 0) * (LB_LA_KEYS * st);
-        for (int i = t; i < LB_LA_KEYS * c16; i += 128) {
-            const int r = i / c16, c = i - r * c16, row = min(k0 + b * LB_LA_KEYS + r, k1 - 1);
-            if (row < pos0 ? old_rows : new_rows) ms_cp16(smem_u32(dst + r * st + c * 16), cache + ((size_t)row * ld_c + c * 8) * 2);
+        for (int r = warp; r < LB_LA_KEYS; r += 4) {
+            const int row = min(k0 + b * LB_LA_KEYS + r, k1 - 1);
+            if (!(row < pos0 ? old_rows : new_rows)) continue;
+            for (int c = lane; c < c16; c += 32) ms_cp16(smem_u32(dst + r * st + c * 16), cache + ((size_t)row * ld_c + c * 8) * 2);
         }
     };
     stage(0, true, false);
     pdl_wait();
     stage(0, false, true);
     asm volatile("cp.async.commit_group;" ::: "memory");
-    for (int i = t; i < 16 * (ld_c / 2); i += 128) { // rows past the last one repeat it; they are not stored
-        const int r = i / (ld_c / 2), c = i - r * (ld_c / 2);
-        const float2 q = *reinterpret_cast<const float2*>(p.ql + (size_t)min(R0 + r, n_rows - 1) * ld_c + 2 * c);
-        uint32_t hi, lo;
-        ms_split(q.x * 1.4426950408889634f, q.y * 1.4426950408889634f, hi, lo);
-        *reinterpret_cast<uint32_t*>(qh_s + r * st + c * 4) = hi;
-        *reinterpret_cast<uint32_t*>(ql_s + r * st + c * 4) = lo;
+    for (int r = warp; r < 16; r += 4) { // rows past the last one repeat it; they are not stored
+        const float4* q = reinterpret_cast<const float4*>(p.ql + (size_t)min(R0 + r, n_rows - 1) * ld_c);
+#pragma unroll 5
+        for (int c = lane; c < ld_c / 4; c += 32) {
+            const float4 v = q[c];
+            uint2 hi, lo;
+            ms_split(v.x * 1.4426950408889634f, v.y * 1.4426950408889634f, hi.x, lo.x);
+            ms_split(v.z * 1.4426950408889634f, v.w * 1.4426950408889634f, hi.y, lo.y);
+            *reinterpret_cast<uint2*>(qh_s + r * st + c * 8) = hi;
+            *reinterpret_cast<uint2*>(ql_s + r * st + c * 8) = lo;
+        }
     }
     int lim[2];
 #pragma unroll
@@ -364,7 +369,8 @@ extern "C" __global__ void __launch_bounds__(128) lat_rows_f32(const __grid_cons
 // four per warp, a lane has eight (or, from rank_p 256, sixteen) columns of each, asked for before the wait
 template <typename TC>
 __device__ __forceinline__ void lat_out_body(const lb_latent_params& p) {
-    __shared__ float o_s[LB_LA_MAX_RANK], f_s[LB_LA_MAX_SPLITS];
+    __shared__ __align__(16) float o_s[LB_LA_MAX_RANK];
+    __shared__ float f_s[LB_LA_MAX_SPLITS];
     const int h = blockIdx.x, t = threadIdx.x, lane = t & 31, warp = t >> 5, row0 = blockIdx.y * 32 + warp * 4;
     const int t0 = blockIdx.z * LB_LA_TOKENS, t1 = min(p.T, t0 + LB_LA_TOKENS);
     uint4 w[4][2];
@@ -404,11 +410,15 @@ __device__ __forceinline__ void lat_out_body(const lb_latent_params& p) {
             for (int i = 0; i < LB_LA_MAX_SPLITS / 32; ++i) f_s[lane + 32 * i] = m[i] / L;
         }
         __syncthreads();
-        for (int c = t; c < p.rank_p; c += LA_THREADS) {
-            float a = 0.f;
-#pragma unroll 8
-            for (int q = 0; q < used; ++q) a = fmaf(f_s[q], part[(size_t)q * rec + c], a);
-            o_s[c] = a;
+        if (2 * t < p.rank_p) {
+            float2 a = make_float2(0.f, 0.f);
+#pragma unroll 16
+            for (int q = 0; q < used; ++q) {
+                const float2 v = *reinterpret_cast<const float2*>(part + (size_t)q * rec + 2 * t);
+                a.x = fmaf(f_s[q], v.x, a.x);
+                a.y = fmaf(f_s[q], v.y, a.y);
+            }
+            *reinterpret_cast<float2*>(o_s + 2 * t) = a;
         }
         __syncthreads();
         float sum[4];

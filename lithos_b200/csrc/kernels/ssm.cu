@@ -121,12 +121,15 @@ extern "C" __global__ void __launch_bounds__(256) ssm_conv(const __grid_constant
                 if (k > 0 && pos >= 0) past[k] = s >= 0 ? p.proj[(size_t)s * p.ld + inner + ch] : p.ring[(size_t)(pos % p.taps) * p.channels + ch];
             }
         }
+        float cur[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) cur[u] = ch >= 0 && u < nt ? __ldcs(p.proj + (size_t)(t0 + u) * p.ld + inner + ch) : 0.f;
 #pragma unroll
         for (int u = 0; u < 8; ++u) {
             if (u >= nt) break;
             float v = 0.f;
             if (ch >= 0) {
-                past[0] = p.proj[(size_t)(t0 + u) * p.ld + inner + ch];
+                past[0] = cur[u];
                 float s = bias;
 #pragma unroll
                 for (int k = LB_SSM_MAX_TAPS - 1; k >= 0; --k) s = fmaf(w[k], past[k], s);
@@ -152,7 +155,8 @@ extern "C" __global__ void __launch_bounds__(256) ssm_conv(const __grid_constant
 // as products mma.sync m16n8k16: B, C and x are bf16 (the convolution's activations); the fp32 factors -- the state, the weights of (i, j), the
 // scaled x -- enter as three bf16 terms, which carry all their 24 bits; sums are fp32.  Warp w has tokens 16 w .. 16 w + 15 of the block as
 // rows of y, and the state rows of the tiles w, w + 4, ... (MT of them) in registers.
-// dynamic shared memory: B, C [64][N_p + 8], x [64][40], S terms [3][N_p][40], scaled x terms [3][64][40], all bf16; c, dt [64] fp32
+// dynamic shared memory: B, C [64][N_p + 8], x [64][40], S terms [3][N_p][40], scaled x terms [3][64][40] (in C's place where they fit, so that
+// three CTAs share an SM), all bf16; c, dt [64] fp32
 #define SC_XST 80 /* bytes of a row of 32 columns and 16 bytes of padding */
 template <int MT>
 __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
@@ -161,8 +165,10 @@ __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
     const int h = blockIdx.x, col0 = blockIdx.y * LB_SSM_COLS, g = h / (p.H / p.G);
     const int bst = 2 * p.N_p + 16, n16 = p.N_p / 8, nk = p.N_p / 16;
     unsigned char *b_s = sc_sm, *c_s = b_s + LB_SSM_SEG * bst, *x_s = c_s + LB_SSM_SEG * bst, *s_s = x_s + LB_SSM_SEG * SC_XST,
-                  *w_s = s_s + 3 * p.N_p * SC_XST;
-    float* cum = reinterpret_cast<float*>(w_s + 3 * LB_SSM_SEG * SC_XST);
+                  *end_s = s_s + 3 * p.N_p * SC_XST;
+    const bool shared_w = bst >= 3 * SC_XST;
+    unsigned char* w_s = shared_w ? c_s : end_s;
+    float* cum = reinterpret_cast<float*>(end_s + (shared_w ? 0 : 3 * LB_SSM_SEG * SC_XST));
     float* dts = cum + LB_SSM_SEG;
     const uint32_t s_term = p.N_p * SC_XST, w_term = LB_SSM_SEG * SC_XST;
     const float a_neg = -expf(bf16_bits_to_f32(p.a_log[h])), dskip = bf16_bits_to_f32(p.d[h]);
@@ -171,25 +177,18 @@ __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
     const uint16_t* xbc = reinterpret_cast<const uint16_t*>(p.xbc);
     const uint16_t *gx = xbc + (size_t)h * p.V_p + col0, *gb = xbc + (size_t)p.H * p.V_p + (size_t)g * p.N_p, *gc = gb + (size_t)p.G * p.N_p;
     // tokens past the chunk repeat its last one (finite values); their step size is 0 and they are not stored
-    auto load_b = [&](int blk) {
-        for (int i = t; i < LB_SSM_SEG * n16; i += 128) {
-            const int r = i / n16, c = i - r * n16;
-            ms_cp16(smem_u32(b_s + r * bst + c * 16), gb + (size_t)min(blk * LB_SSM_SEG + r, p.T - 1) * p.ld_xbc + c * 8);
+    auto load = [&](int blk) {
+        for (int r = warp; r < LB_SSM_SEG; r += 4) {
+            const size_t row = (size_t)min(blk * LB_SSM_SEG + r, p.T - 1) * p.ld_xbc;
+            for (int c = lane; c < n16; c += 32) {
+                ms_cp16(smem_u32(b_s + r * bst + c * 16), gb + row + c * 8);
+                ms_cp16(smem_u32(c_s + r * bst + c * 16), gc + row + c * 8);
+            }
+            if (lane < 4) ms_cp16(smem_u32(x_s + r * SC_XST + lane * 16), gx + row + lane * 8);
         }
+        asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    auto load_cx = [&](int blk) {
-        for (int i = t; i < LB_SSM_SEG * n16; i += 128) {
-            const int r = i / n16, c = i - r * n16;
-            ms_cp16(smem_u32(c_s + r * bst + c * 16), gc + (size_t)min(blk * LB_SSM_SEG + r, p.T - 1) * p.ld_xbc + c * 8);
-        }
-        for (int i = t; i < LB_SSM_SEG * 4; i += 128) {
-            const int r = i >> 2, c = i & 3;
-            ms_cp16(smem_u32(x_s + r * SC_XST + c * 16), gx + (size_t)min(blk * LB_SSM_SEG + r, p.T - 1) * p.ld_xbc + c * 8);
-        }
-    };
-    load_b(0);
-    load_cx(0);
-    asm volatile("cp.async.commit_group;" ::: "memory");
+    load(0);
 
     // the state: tile mt of this warp is rows 16 (warp + 4 mt) + fg (+ 8), columns 8 nt + 2 ft (+ 1)
     float st[MT][4][4];
@@ -248,18 +247,6 @@ __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         const float c_end = cum[LB_SSM_SEG - 1];
-        // scaled x
-        for (int i = t; i < LB_SSM_SEG * 16; i += 128) {
-            const int r = i >> 4, c = i & 15;
-            const float w = dts[r] * expf(c_end - cum[r]);
-            const uint32_t u = *reinterpret_cast<const uint32_t*>(x_s + r * SC_XST + c * 4);
-            uint32_t a, b, d;
-            ms_split3(w * __uint_as_float(u << 16), w * __uint_as_float(u & 0xffff0000u), a, b, d);
-            unsigned char* dst = w_s + r * SC_XST + c * 4;
-            *reinterpret_cast<uint32_t*>(dst) = a;
-            *reinterpret_cast<uint32_t*>(dst + w_term) = b;
-            *reinterpret_cast<uint32_t*>(dst + 2 * w_term) = d;
-        }
         // C . B and C . S of the warp's 16 tokens
         float sc[8][4], y[4][4];
 #pragma unroll
@@ -328,8 +315,20 @@ __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
                 if (col0 + c + 1 < p.V) dst[c + 1] = fmaf(dskip, __uint_as_float(u & 0xffff0000u), y[nt][2 * r + 1]);
             }
         }
-        __syncthreads(); // scaled x is there; C, x and the old state's terms have been read
-        if (blk + 1 < n_blk) load_cx(blk + 1);
+        __syncthreads(); // C and the old state's terms have been read
+        // scaled x
+        for (int i = t; i < LB_SSM_SEG * 16; i += 128) {
+            const int r = i >> 4, c = i & 15;
+            const float w = dts[r] * expf(c_end - cum[r]);
+            const uint32_t u = *reinterpret_cast<const uint32_t*>(x_s + r * SC_XST + c * 4);
+            uint32_t a, b, d;
+            ms_split3(w * __uint_as_float(u << 16), w * __uint_as_float(u & 0xffff0000u), a, b, d);
+            unsigned char* dst = w_s + r * SC_XST + c * 4;
+            *reinterpret_cast<uint32_t*>(dst) = a;
+            *reinterpret_cast<uint32_t*>(dst + w_term) = b;
+            *reinterpret_cast<uint32_t*>(dst + 2 * w_term) = d;
+        }
+        __syncthreads();
         const float e_end = expf(c_end);
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) {
@@ -356,10 +355,9 @@ __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
         }
         if (blk + 1 < n_blk) {
             put_state();
-            __syncthreads(); // everybody is done with B, c and dt
-            load_b(blk + 1);
+            __syncthreads(); // everybody is done with B, x, scaled x, c and dt
+            load(blk + 1);
         }
-        asm volatile("cp.async.commit_group;" ::: "memory");
     }
     pdl_launch_dependents();
 #pragma unroll
@@ -372,8 +370,8 @@ __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
                 if (n < p.N && col0 + c < p.V) S[(size_t)n * p.V + c] = st[mt][nt][e];
             }
 }
-extern "C" __global__ void __launch_bounds__(128) ssm_chunk_64(const __grid_constant__ lb_ssm_params p) { ssm_chunk_body<1>(p); }
-extern "C" __global__ void __launch_bounds__(128) ssm_chunk_128(const __grid_constant__ lb_ssm_params p) { ssm_chunk_body<2>(p); }
+extern "C" __global__ void __launch_bounds__(128, 3) ssm_chunk_64(const __grid_constant__ lb_ssm_params p) { ssm_chunk_body<1>(p); }
+extern "C" __global__ void __launch_bounds__(128, 3) ssm_chunk_128(const __grid_constant__ lb_ssm_params p) { ssm_chunk_body<2>(p); }
 extern "C" __global__ void __launch_bounds__(128) ssm_chunk_256(const __grid_constant__ lb_ssm_params p) { ssm_chunk_body<4>(p); }
 
 // fp32: grid (H, ceil(V / 32)), block 128, threads as in ssm_step; the operands of SF_TOK tokens at a time in shared memory
