@@ -525,7 +525,7 @@ static int launch_tc(lb_ctx* c, lb_dgemm_params* p, int tiles) { /* operand stag
     const int stage = LB_DG_ROWS * LB_DG_KB * 2 + p->NT * LB_DG_KB * 2;
     p->stages = 200 * 1024 / stage;
     if (p->stages > LB_DG_MAX_STAGES) p->stages = LB_DG_MAX_STAGES;
-    p->tmem_cols = 2 * p->NT < 32 ? 32 : 2 * p->NT;
+    for (p->tmem_cols = 32; p->tmem_cols < 2 * p->NT;) p->tmem_cols *= 2;
     void* params[] = {p};
     return lb_launch(c, LBK_gemm_bf16_tc, (unsigned)(tiles < c->sm_count ? tiles : c->sm_count), 1, 1, LB_DG_THREADS, (unsigned)(p->stages * stage), params, 1);
 }
@@ -561,10 +561,16 @@ static int launch_products(lb_model* m, const st_prod* pr, int n, int T) {
 }
 
 /* the expert products of a chunk: `n` assignments sorted by expert, tile by tile of the plan */
-static int moe_tile(const stack_t* S, const lb_stack_layer* D, int T) { /* assignments per tile: about an expert's share */
+static double tile_cost(int nt) { const double c = 0.1 + 0.9 * nt / 256.0; return c < 0.33 ? 0.33 : c; } /* the table of product_cost, any width */
+static int moe_tile(const stack_t* S, const lb_stack_layer* D, int T) { /* assignments per tile: an expert's share and some more, in as few tiles as pays */
     if (S->esz == 4) return ST_MOE_TILE;
-    int nt = 16;
-    while (nt < 256 && nt * D->experts < T * D->top) nt *= 2;
+    const double share = (double)T * D->top / D->experts, want = share + 2.0 * sqrt(share);
+    double best = 1e30;
+    int nt = 256;
+    for (int k = (int)(want / 256.0) + 1, n = 0; n < 3; n++, k++) {
+        const int w = pad_to((int)ceil(want / k), 16), c = w > 256 ? 256 : w;
+        if (k * tile_cost(c) < best) { best = k * tile_cost(c); nt = c; }
+    }
     return nt;
 }
 static size_t plan_ints(int T, int top, int experts, int nt) { return (size_t)pad_to(T * top, 4) + 4 + 4 * (size_t)(experts + T * top / nt + 1); }
@@ -853,7 +859,7 @@ static int pf_ssm(lb_model* m, pf_set* w, int i, int pos0, int T) {
     fill_ssm(m, i, &p, w->st.proj);
     p.pos0 = pos0; p.T = T; p.xbc = (void*)w->st.xbc; p.dt = (float*)w->st.dt; p.y = (float*)w->st.o; p.cat = (void*)w->st.cat; p.cat_ld = L->out.K;
     void* params[] = {&p};
-    LB_TRY(lb_launch(c, LBK_ssm_conv, (unsigned)((p.ld_xbc + D->heads + 255) / 256), (unsigned)((T + 7) / 8), 1, 256, 0, params, 1));
+    LB_TRY(lb_launch(c, LBK_ssm_conv, (unsigned)((p.ld_xbc + D->heads + 255) / 256), (unsigned)((T + LB_SSM_CONV_TOKENS - 1) / LB_SSM_CONV_TOKENS), 1, 256, 0, params, 1));
     static const int k_f32[3] = {LBK_ssm_scan_f32_64, LBK_ssm_scan_f32_128, LBK_ssm_scan_f32_256}, k_tc[3] = {LBK_ssm_chunk_64, LBK_ssm_chunk_128, LBK_ssm_chunk_256};
     const int row = 2 * L->N_p + 16, smem = 2 * LB_SSM_SEG * row + (row >= 240 ? 1 : 4) * LB_SSM_SEG * 80 + 3 * L->N_p * 80 + 2 * LB_SSM_SEG * 4; /* as ssm_chunk lays it out */
     LB_TRY(lb_launch(c, (S->esz == 4 ? k_f32 : k_tc)[state_size(D)], (unsigned)D->heads, (unsigned)(L->V_p / LB_SSM_COLS), 1, 128, S->esz == 4 ? 0u : (unsigned)smem, params, 1));
@@ -1046,7 +1052,7 @@ static const lb_arch k_stack = {"stack", ST_STREAMS, stack_reset_state, stack_sn
 static double experts_cost(const lb_model* m, const lb_stack_layer* D, int rows, int K, int T) {
     const stack_t* S = S_of(m);
     const int nt = moe_tile(S, D, T), tiles = D->experts * ((T * D->top / D->experts + nt - 1) / nt) * ((rows + LB_DG_ROWS - 1) / LB_DG_ROWS);
-    const double flops = (double)((tiles + m->c->sm_count - 1) / m->c->sm_count) * (nt >= 256 ? 1.0 : nt >= 128 ? 0.55 : 0.36), bytes = D->experts * (double)rows / HBM_ROWS;
+    const double flops = (double)((tiles + m->c->sm_count - 1) / m->c->sm_count) * tile_cost(nt), bytes = D->experts * (double)rows / HBM_ROWS;
     return K * (flops > bytes ? flops : bytes);
 }
 

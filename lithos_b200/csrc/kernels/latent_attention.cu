@@ -132,26 +132,35 @@ __device__ __forceinline__ void lat_rows_body(const lb_latent_params& p) {
     // rows of a block with old <= (row >= pos0) <= new...: rows before pos0 exist since an earlier step
     auto stage = [&](int b, bool old_rows, bool new_rows) {
         unsigned char* dst = kv_s + (p.stages > 1 ? b & 1 : 0) * (LB_LA_KEYS * st);
-        for (int r = warp; r < LB_LA_KEYS; r += 4) {
+        for (int r = t >> 3; r < LB_LA_KEYS; r += 16) { // eight threads per row
             const int row = min(k0 + b * LB_LA_KEYS + r, k1 - 1);
             if (!(row < pos0 ? old_rows : new_rows)) continue;
-            for (int c = lane; c < c16; c += 32) ms_cp16(smem_u32(dst + r * st + c * 16), cache + ((size_t)row * ld_c + c * 8) * 2);
+            const unsigned char* src = cache + (size_t)row * ld_c * 2;
+            const uint32_t to = smem_u32(dst + r * st);
+#pragma unroll 3
+            for (int c = t & 7; c < c16; c += 8) ms_cp16(to + c * 16, src + c * 16);
         }
     };
     stage(0, true, false);
     pdl_wait();
     stage(0, false, true);
     asm volatile("cp.async.commit_group;" ::: "memory");
-    for (int r = warp; r < 16; r += 4) { // rows past the last one repeat it; they are not stored
+    { // rows past the last one repeat it; they are not stored.  Eight threads per row, nine quads of each in flight
+        const int r = t >> 3;
         const float4* q = reinterpret_cast<const float4*>(p.ql + (size_t)min(R0 + r, n_rows - 1) * ld_c);
-#pragma unroll 5
-        for (int c = lane; c < ld_c / 4; c += 32) {
-            const float4 v = q[c];
-            uint2 hi, lo;
-            ms_split(v.x * 1.4426950408889634f, v.y * 1.4426950408889634f, hi.x, lo.x);
-            ms_split(v.z * 1.4426950408889634f, v.w * 1.4426950408889634f, hi.y, lo.y);
-            *reinterpret_cast<uint2*>(qh_s + r * st + c * 8) = hi;
-            *reinterpret_cast<uint2*>(ql_s + r * st + c * 8) = lo;
+        for (int c0 = t & 7; c0 < ld_c / 4; c0 += 72) {
+            float4 v[9];
+#pragma unroll
+            for (int k = 0; k < 9; ++k) v[k] = c0 + 8 * k < ld_c / 4 ? q[c0 + 8 * k] : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int k = 0; k < 9; ++k) {
+                if (c0 + 8 * k >= ld_c / 4) continue;
+                uint2 hi, lo;
+                ms_split(v[k].x * 1.4426950408889634f, v[k].y * 1.4426950408889634f, hi.x, lo.x);
+                ms_split(v[k].z * 1.4426950408889634f, v[k].w * 1.4426950408889634f, hi.y, lo.y);
+                *reinterpret_cast<uint2*>(qh_s + r * st + (c0 + 8 * k) * 8) = hi;
+                *reinterpret_cast<uint2*>(ql_s + r * st + (c0 + 8 * k) * 8) = lo;
+            }
         }
     }
     int lim[2];
@@ -175,7 +184,7 @@ __device__ __forceinline__ void lat_rows_body(const lb_latent_params& p) {
         } else asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         const uint32_t blk = smem_u32(kv_s) + (p.stages > 1 ? b & 1 : 0) * (LB_LA_KEYS * st);
-        float sc[2][4] = {};
+        float sc[2][4] = {}, sl[2][4] = {};
 #pragma unroll 4
         for (int c = 0; c < nkc; ++c) {
             uint32_t h0, h1, h2, h3, l0, l1, l2, l3, b0, b1, b2, b3;
@@ -183,10 +192,14 @@ __device__ __forceinline__ void lat_rows_body(const lb_latent_params& p) {
             ms_ldsm(ql_lane + c * 32, l0, l1, l2, l3);
             ms_ldsm(blk + k_off + c * 32, b0, b1, b2, b3);
             ms_mma(sc[0], h0, h1, h2, h3, b0, b1);
-            ms_mma(sc[0], l0, l1, l2, l3, b0, b1);
             ms_mma(sc[1], h0, h1, h2, h3, b2, b3);
-            ms_mma(sc[1], l0, l1, l2, l3, b2, b3);
+            ms_mma(sl[0], l0, l1, l2, l3, b0, b1);
+            ms_mma(sl[1], l0, l1, l2, l3, b2, b3);
         }
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) sc[j][e] += sl[j][e];
         const int key0 = k0 + b * LB_LA_KEYS + warp * 16 + 2 * ft;
 #pragma unroll
         for (int r = 0; r < 2; ++r) { // maxima of the warp's 16 keys

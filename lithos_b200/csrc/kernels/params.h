@@ -463,6 +463,7 @@ typedef struct {
 #define LB_SSM_MAX_STATE 256
 #define LB_SSM_SEG 64  /* tokens per block of ssm_chunk_* */
 #define LB_SSM_COLS 32 /* value columns per CTA */
+#define LB_SSM_CONV_TOKENS 16 /* tokens per thread of ssm_conv */
 typedef struct {
     const float* proj;      /* fp32 [T, ld]: z [H V] | x [H V] | B [G N] | C [G N] | dt [H] */
     const uint16_t* conv_w; /* bf16 [channels, taps], last column = the current token */

@@ -94,9 +94,9 @@ extern "C" __global__ void __launch_bounds__(128) ssm_step_64(const __grid_const
 extern "C" __global__ void __launch_bounds__(128) ssm_step_128(const __grid_constant__ lb_ssm_params p) { ssm_step_body<32>(p); }
 extern "C" __global__ void __launch_bounds__(128) ssm_step_256(const __grid_constant__ lb_ssm_params p) { ssm_step_body<64>(p); }
 
-// grid (ceil((ld_xbc + H) / 256), ceil(T / 8)), block 256: a thread makes one (padded) channel, or one head's step sizes, of eight tokens
+// grid (ceil((ld_xbc + H) / 256), ceil(T / 16)), block 256: a thread makes one (padded) channel, or one head's step sizes, of LB_SSM_CONV_TOKENS tokens
 extern "C" __global__ void __launch_bounds__(256) ssm_conv(const __grid_constant__ lb_ssm_params p) {
-    const int i = blockIdx.x * 256 + threadIdx.x, t0 = blockIdx.y * 8, nt = min(8, p.T - t0), inner = p.H * p.V;
+    const int i = blockIdx.x * 256 + threadIdx.x, t0 = blockIdx.y * LB_SSM_CONV_TOKENS, nt = min(LB_SSM_CONV_TOKENS, p.T - t0), inner = p.H * p.V;
     const int nx = p.H * p.V_p, nb = p.G * p.N_p;
     pdl_wait();
     if (i < p.ld_xbc) {
@@ -121,11 +121,11 @@ extern "C" __global__ void __launch_bounds__(256) ssm_conv(const __grid_constant
                 if (k > 0 && pos >= 0) past[k] = s >= 0 ? p.proj[(size_t)s * p.ld + inner + ch] : p.ring[(size_t)(pos % p.taps) * p.channels + ch];
             }
         }
-        float cur[8];
+        float cur[LB_SSM_CONV_TOKENS];
 #pragma unroll
-        for (int u = 0; u < 8; ++u) cur[u] = ch >= 0 && u < nt ? __ldcs(p.proj + (size_t)(t0 + u) * p.ld + inner + ch) : 0.f;
+        for (int u = 0; u < LB_SSM_CONV_TOKENS; ++u) cur[u] = ch >= 0 && u < nt ? __ldcs(p.proj + (size_t)(t0 + u) * p.ld + inner + ch) : 0.f;
 #pragma unroll
-        for (int u = 0; u < 8; ++u) {
+        for (int u = 0; u < LB_SSM_CONV_TOKENS; ++u) {
             if (u >= nt) break;
             float v = 0.f;
             if (ch >= 0) {
