@@ -169,6 +169,9 @@ int lb_driver_load(char* err, size_t errlen); /* LB_OK or LB_ERR_NO_DRIVER */
     X(ssm_step_64)                    \
     X(ssm_step_128)                   \
     X(ssm_step_256)                   \
+    X(ssm_local_64)                   \
+    X(ssm_local_128)                  \
+    X(ssm_local_256)                  \
     X(ssm_conv)                       \
     X(ssm_chunk_64)                   \
     X(ssm_chunk_128)                  \

@@ -27,6 +27,7 @@
 #define ST_STREAMS 4
 #define ST_LAT_ABSORB 16 /* latent attention: portions of fewer tokens do not make keys and values of every cached position */
 #define ST_MOE_TILE 64 /* token tile of the fp32 expert products */
+#define ST_SSM_SEGS 8  /* most segments of a chunk through a state-space recurrence */
 #define ST_SEG 128     /* tokens of a chunk a recurrence walks one after the other; segments run side by side */
 
 typedef struct {
@@ -862,7 +863,21 @@ static int pf_ssm(lb_model* m, pf_set* w, int i, int pos0, int T) {
     LB_TRY(lb_launch(c, LBK_ssm_conv, (unsigned)((p.ld_xbc + D->heads + 255) / 256), (unsigned)((T + LB_SSM_CONV_TOKENS - 1) / LB_SSM_CONV_TOKENS), 1, 256, 0, params, 1));
     static const int k_f32[3] = {LBK_ssm_scan_f32_64, LBK_ssm_scan_f32_128, LBK_ssm_scan_f32_256}, k_tc[3] = {LBK_ssm_chunk_64, LBK_ssm_chunk_128, LBK_ssm_chunk_256};
     const int row = 2 * L->N_p + 16, smem = 2 * LB_SSM_SEG * row + (row >= 240 ? 1 : 4) * LB_SSM_SEG * 80 + 3 * L->N_p * 80 + 2 * LB_SSM_SEG * 4; /* as ssm_chunk lays it out */
-    LB_TRY(lb_launch(c, (S->esz == 4 ? k_f32 : k_tc)[state_size(D)], (unsigned)D->heads, (unsigned)(L->V_p / LB_SSM_COLS), 1, 128, S->esz == 4 ? 0u : (unsigned)smem, params, 1));
+    static const int k_local[3] = {LBK_ssm_local_64, LBK_ssm_local_128, LBK_ssm_local_256};
+    const unsigned slabs = (unsigned)(L->V_p / LB_SSM_COLS), heads = (unsigned)D->heads;
+    if (S->esz == 4) LB_TRY(lb_launch(c, k_f32[state_size(D)], heads, slabs, 1, 128, 0, params, 1));
+    else {
+        /* as many segments side by side as CTAs fit on the SMs, four blocks of tokens each at least */
+        const int blocks = (T + LB_SSM_SEG - 1) / LB_SSM_SEG, fit = c->sm_count * (L->N_p <= 128 ? 3 : 1) / (int)(heads * slabs);
+        int P = fit < blocks / 4 ? fit : blocks / 4;
+        if (P > ST_SSM_SEGS) P = ST_SSM_SEGS;
+        if (P < 1) P = 1;
+        p.seg = (blocks + P - 1) / P * LB_SSM_SEG;
+        P = (T + p.seg - 1) / p.seg;
+        p.seg_state = (float*)w->st.seg_state; p.seg_decay = (float*)w->st.seg_decay;
+        if (P > 1) LB_TRY(lb_launch(c, k_local[state_size(D)], heads, slabs, (unsigned)P - 1, 128, (unsigned)smem, params, 1));
+        LB_TRY(lb_launch(c, k_tc[state_size(D)], heads, slabs, (unsigned)P, 128, (unsigned)smem, params, 1));
+    }
     return lb_launch(c, LBK_ssm_finish, (unsigned)T, (unsigned)D->norm_groups, 1, 128, (unsigned)(L->n_mix / D->norm_groups * 4), params, 1);
 }
 
@@ -1125,7 +1140,8 @@ static int stack_build(lb_model* m, const lb_stack_desc* d, lb_weight_source* sr
                 MAX(S->max_q, D->heads * kd); MAX(S->max_kx, D->heads * L->dim_p); MAX(S->max_vx, D->heads * L->vdim_p);
             }
         } else if (D->mixer == LB_MIX_SSM) {
-            MAX(S->max_heads, D->heads); MAX(S->max_xbc, D->heads * L->V_p + 2 * D->groups * L->N_p); MAX(S->max_o, D->heads * D->vdim);
+            MAX(S->max_state, state_bytes(D));
+            MAX(S->max_heads, D->heads); MAX(S->max_dk, D->heads); MAX(S->max_xbc, D->heads * L->V_p + 2 * D->groups * L->N_p); MAX(S->max_o, D->heads * D->vdim);
         } else if (D->mixer == LB_MIX_ATTENTION) {
             MAX(S->max_q, D->heads * L->dim_p);
             /* slices of the decode attention: one tile of 32 rows per warp each, as many as keep one CTA per SM */

@@ -477,10 +477,13 @@ typedef struct {
     float* y;               /* fp32 [T, H V] */
     void* xbc;              /* prompt: x [H, V_p] | B [G, N_p] | C [G, N_p] after the convolution, bf16 (or fp32), padding zero, rows of ld_xbc */
     float* dt;              /* prompt: fp32 [T, H] step sizes */
+    float* seg_state;       /* prompt in segments: fp32 [segments, H, N, V] and ... */
+    float* seg_decay;       /* ... [segments, H], logarithms */
     void* cat;              /* prompt: gated, normed rows [T, cat_ld] */
     const int32_t* pos_ptr; /* decode: position in device memory */
     int32_t ld, H, V, V_p, N, N_p, G, taps, channels, ld_xbc, norm_groups;
     int32_t pos0, T, cat_ld, f32;
+    int32_t seg;            /* ssm_chunk, ssm_local: tokens per segment, a multiple of LB_SSM_SEG (T or more: one segment) */
     float eps;
 } lb_ssm_params;
 

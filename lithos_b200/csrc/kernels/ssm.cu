@@ -4,7 +4,8 @@
 // A column of a head's state needs only that column of x, so a CTA owns LB_SSM_COLS columns of one head.
 //   ssm_step_*     one token (decode): convolution, state read and written once, read-out
 //   ssm_conv       a prompt chunk's convolved channels and step sizes
-//   ssm_chunk_*    a prompt chunk on the tensor cores, block by block of LB_SSM_SEG tokens, the state on chip between blocks
+//   ssm_chunk_*    a prompt chunk on the tensor cores, block by block of LB_SSM_SEG tokens, the state on chip between blocks; where the heads
+//                  are few, in segments side by side: ssm_local_* carries each from a zero state, ssm_chunk_* starts each from its true state
 //   ssm_scan_f32_* the same token by token in fp32
 //   ssm_finish     gate, norm in parts, and the convolution's last inputs into the ring
 #include "mma_sync.cuh"
@@ -149,7 +150,7 @@ extern "C" __global__ void __launch_bounds__(256) ssm_conv(const __grid_constant
     pdl_launch_dependents();
 }
 
-// grid (H, ceil(V / 32)), block 128 (4 warps).  With c_i the sum of a = -exp(A_log) dt over the block's tokens up to i, a block of tokens does
+// grid (H, ceil(V / 32), segments), block 128 (4 warps).  With c_i the sum of a = -exp(A_log) dt over the block's tokens up to i, a block of tokens does
 //   y_i = exp(c_i) S^T C_i + sum_(j <= i) exp(c_i - c_j) dt_j (C_i . B_j) x_j + D x_i
 //   S  <- exp(c_end) S + sum_j B_j (exp(c_end - c_j) dt_j x_j)^T
 // as products mma.sync m16n8k16: B, C and x are bf16 (the convolution's activations); the fp32 factors -- the state, the weights of (i, j), the
@@ -157,8 +158,11 @@ extern "C" __global__ void __launch_bounds__(256) ssm_conv(const __grid_constant
 // rows of y, and the state rows of the tiles w, w + 4, ... (MT of them) in registers.
 // dynamic shared memory: B, C [64][N_p + 8], x [64][40], S terms [3][N_p][40], scaled x terms [3][64][40] (in C's place where they fit, so that
 // three CTAs share an SM), all bf16; c, dt [64] fp32
+// Segments (gridDim.z = P > 1; segment g is tokens g * seg .. of the chunk): LOCAL (first launch, P - 1 segments) leaves what each segment makes of
+// a zero state (segment 0: of the sequence's state) and its summed log decay, and keeps the sequence's state in the last place; the second
+// launch makes a segment's start from those before it, and the last segment leaves the sequence's state.
 #define SC_XST 80 /* bytes of a row of 32 columns and 16 bytes of padding */
-template <int MT>
+template <int MT, bool LOCAL>
 __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
     extern __shared__ __align__(16) unsigned char sc_sm[];
     const int t = threadIdx.x, lane = t & 31, warp = t >> 5, fg = lane >> 2, ft = lane & 3;
@@ -172,17 +176,18 @@ __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
     float* dts = cum + LB_SSM_SEG;
     const uint32_t s_term = p.N_p * SC_XST, w_term = LB_SSM_SEG * SC_XST;
     const float a_neg = -expf(bf16_bits_to_f32(p.a_log[h])), dskip = bf16_bits_to_f32(p.d[h]);
-    const int n_blk = (p.T + LB_SSM_SEG - 1) / LB_SSM_SEG;
+    const int seg = blockIdx.z, P = LOCAL ? gridDim.z + 1 : gridDim.z, tok_lo = seg * p.seg, tok_hi = min(p.T, tok_lo + p.seg);
+    const int n_blk = (tok_hi - tok_lo + LB_SSM_SEG - 1) / LB_SSM_SEG;
     pdl_wait();
     const uint16_t* xbc = reinterpret_cast<const uint16_t*>(p.xbc);
     const uint16_t *gx = xbc + (size_t)h * p.V_p + col0, *gb = xbc + (size_t)p.H * p.V_p + (size_t)g * p.N_p, *gc = gb + (size_t)p.G * p.N_p;
-    // tokens past the chunk repeat its last one (finite values); their step size is 0 and they are not stored
+    // tokens past the segment repeat its last one (finite values); their step size is 0 and they are not stored
     auto load = [&](int blk) {
         for (int r = warp; r < LB_SSM_SEG; r += 4) {
-            const size_t row = (size_t)min(blk * LB_SSM_SEG + r, p.T - 1) * p.ld_xbc;
+            const size_t row = (size_t)min(tok_lo + blk * LB_SSM_SEG + r, tok_hi - 1) * p.ld_xbc;
             for (int c = lane; c < n16; c += 32) {
                 ms_cp16(smem_u32(b_s + r * bst + c * 16), gb + row + c * 8);
-                ms_cp16(smem_u32(c_s + r * bst + c * 16), gc + row + c * 8);
+                if (!LOCAL) ms_cp16(smem_u32(c_s + r * bst + c * 16), gc + row + c * 8);
             }
             if (lane < 4) ms_cp16(smem_u32(x_s + r * SC_XST + lane * 16), gx + row + lane * 8);
         }
@@ -192,16 +197,38 @@ __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
 
     // the state: tile mt of this warp is rows 16 (warp + 4 mt) + fg (+ 8), columns 8 nt + 2 ft (+ 1)
     float st[MT][4][4];
-    float* S = p.state + (size_t)h * p.N * p.V + col0;
+    const size_t corner = (size_t)h * p.N * p.V + col0, all = (size_t)p.H * p.N * p.V;
+    auto each = [&](auto f) { // f(value, offset from the head's corner) of what exists of the state
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+            for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int n = 16 * (warp + 4 * mt) + fg + 8 * (e >> 1), c = 8 * nt + 2 * ft + (e & 1);
+                    if (n < p.N && col0 + c < p.V) f(st[mt][nt][e], (size_t)n * p.V + c);
+                }
+    };
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
         for (int nt = 0; nt < 4; ++nt)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int n = 16 * (warp + 4 * mt) + fg + 8 * (e >> 1), c = 8 * nt + 2 * ft + (e & 1);
-                st[mt][nt][e] = n < p.N && col0 + c < p.V ? S[(size_t)n * p.V + c] : 0.f;
-            }
+            for (int e = 0; e < 4; ++e) st[mt][nt][e] = 0.f;
+    float* first = P > 1 ? p.seg_state + (size_t)(P - 1) * all + corner : nullptr; // the sequence's state, kept
+    if (LOCAL ? seg == 0 : P == 1) {
+        each([&](float& v, size_t o) { v = p.state[corner + o]; });
+        if (LOCAL) each([&](float& v, size_t o) { first[o] = v; });
+    } else if (!LOCAL && seg == 0) {
+        each([&](float& v, size_t o) { v = first[o]; });
+    } else if (!LOCAL) {
+        each([&](float& v, size_t o) { v = p.seg_state[corner + o]; });
+        for (int q = 1; q < seg; ++q) {
+            const float d = expf(p.seg_decay[(size_t)q * p.H + h]);
+            each([&](float& v, size_t o) { v = fmaf(d, v, p.seg_state[(size_t)q * all + corner + o]); });
+        }
+    }
+    float log_decay = 0.f; // LOCAL: of the segment so far
     auto put_state = [&]() {
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) {
@@ -220,7 +247,7 @@ __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
                 }
         }
     };
-    put_state();
+    if (!LOCAL) put_state();
     const uint32_t a_row = (warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * bst + (lane >> 4) * 16; // A operand: rows of C
     const uint32_t k_row = ((lane & 7) + ((lane >> 4) << 3)) * bst + ((lane >> 3) & 1) * 16;          // B operand: rows of B as columns
     const uint32_t t_row = ((lane & 7) + ((lane >> 3) & 1) * 8) * SC_XST + (lane >> 4) * 16;          // B operand: rows are k (transposing load)
@@ -228,10 +255,10 @@ __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
     const uint32_t ub = smem_u32(b_s), uc = smem_u32(c_s), ux = smem_u32(x_s), us = smem_u32(s_s), uw = smem_u32(w_s);
 
     for (int blk = 0; blk < n_blk; ++blk) {
-        const int tok0 = blk * LB_SSM_SEG;
+        const int tok0 = tok_lo + blk * LB_SSM_SEG;
         if (warp == 0) { // step sizes and the running sum of log decays: lane has tokens 2 lane, 2 lane + 1
             const int i0 = tok0 + 2 * lane;
-            const float d0 = i0 < p.T ? p.dt[(size_t)i0 * p.H + h] : 0.f, d1 = i0 + 1 < p.T ? p.dt[(size_t)(i0 + 1) * p.H + h] : 0.f;
+            const float d0 = i0 < tok_hi ? p.dt[(size_t)i0 * p.H + h] : 0.f, d1 = i0 + 1 < tok_hi ? p.dt[(size_t)(i0 + 1) * p.H + h] : 0.f;
             const float a0 = a_neg * d0, a1 = a_neg * d1;
             float s = a0 + a1;
 #pragma unroll
@@ -247,7 +274,7 @@ __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         const float c_end = cum[LB_SSM_SEG - 1];
-        // C . B and C . S of the warp's 16 tokens
+        if (!LOCAL) { // C . B and C . S of the warp's 16 tokens
         float sc[8][4], y[4][4];
 #pragma unroll
         for (int j = 0; j < 8; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
@@ -305,7 +332,7 @@ __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
             const int tok = tok0 + i0 + 8 * r;
-            if (tok >= p.T) continue;
+            if (tok >= tok_hi) continue;
             float* dst = p.y + ((size_t)tok * p.H + h) * p.V + col0;
 #pragma unroll
             for (int nt = 0; nt < 4; ++nt) {
@@ -315,7 +342,9 @@ __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
                 if (col0 + c + 1 < p.V) dst[c + 1] = fmaf(dskip, __uint_as_float(u & 0xffff0000u), y[nt][2 * r + 1]);
             }
         }
-        __syncthreads(); // C and the old state's terms have been read
+        }
+        if (!LOCAL) __syncthreads(); // C and the old state's terms have been read
+        log_decay += c_end;
         // scaled x
         for (int i = t; i < LB_SSM_SEG * 16; i += 128) {
             const int r = i >> 4, c = i & 15;
@@ -354,25 +383,25 @@ __device__ __forceinline__ void ssm_chunk_body(const lb_ssm_params& p) {
             }
         }
         if (blk + 1 < n_blk) {
-            put_state();
+            if (!LOCAL) put_state();
             __syncthreads(); // everybody is done with B, x, scaled x, c and dt
             load(blk + 1);
         }
     }
     pdl_launch_dependents();
-#pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-        for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int n = 16 * (warp + 4 * mt) + fg + 8 * (e >> 1), c = 8 * nt + 2 * ft + (e & 1);
-                if (n < p.N && col0 + c < p.V) S[(size_t)n * p.V + c] = st[mt][nt][e];
-            }
+    if (LOCAL) {
+        each([&](float& v, size_t o) { p.seg_state[(size_t)seg * all + corner + o] = v; });
+        if (blockIdx.y == 0 && t == 0) p.seg_decay[(size_t)seg * p.H + h] = log_decay;
+    } else if (seg == P - 1) {
+        each([&](float& v, size_t o) { p.state[corner + o] = v; });
+    }
 }
-extern "C" __global__ void __launch_bounds__(128, 3) ssm_chunk_64(const __grid_constant__ lb_ssm_params p) { ssm_chunk_body<1>(p); }
-extern "C" __global__ void __launch_bounds__(128, 3) ssm_chunk_128(const __grid_constant__ lb_ssm_params p) { ssm_chunk_body<2>(p); }
-extern "C" __global__ void __launch_bounds__(128) ssm_chunk_256(const __grid_constant__ lb_ssm_params p) { ssm_chunk_body<4>(p); }
+#define SC_KERNELS(n, MT, BLOCKS)                                                                                                                            \
+    extern "C" __global__ void __launch_bounds__(128, BLOCKS) ssm_chunk_##n(const __grid_constant__ lb_ssm_params p) { ssm_chunk_body<MT, false>(p); } \
+    extern "C" __global__ void __launch_bounds__(128, BLOCKS) ssm_local_##n(const __grid_constant__ lb_ssm_params p) { ssm_chunk_body<MT, true>(p); }
+SC_KERNELS(64, 1, 3)
+SC_KERNELS(128, 2, 3)
+SC_KERNELS(256, 4, 1)
 
 // fp32: grid (H, ceil(V / 32)), block 128, threads as in ssm_step; the operands of SF_TOK tokens at a time in shared memory
 #define SF_TOK 8

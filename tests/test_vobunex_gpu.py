@@ -217,14 +217,14 @@ def test_slow_decay_keeps_a_distant_token(ctx, lb, tmp_path, dtype):
         w["l0.mix.dt_bias"][:] = C.bf16(np.float32([-4, -3, -2, -1]))
         w["embed"][0] *= 8
     c = Case(tmp_path, ctx, cfg, 47, tweak=tweak)
-    n = 400
+    n = 1000                                          # several segments side by side in a prompt's chunk
     toks = np.random.default_rng(9).integers(1, 60, n)
     toks[0] = 0
     toks = toks.tolist()
     want = c.want(toks)
     m = c.open(dtype, n)
     check(m.forward(toks, 0, list(range(n))), want, dtype, "prompt")
-    for cuts in ([63, 2, 64, 1, 128, 65, 77], [2, 398], [300] + [1] * 100):
+    for cuts in ([63, 2, 64, 1, 128, 65, 677], [2, 998], [513, 387] + [1] * 100):
         m.reset_state()
         check(feed(m, toks, cuts), want, dtype, cuts)
     m.close()
