@@ -416,6 +416,7 @@ int lb_model_generate(lb_model* m, const int* prompt, int n_prompt, int max_new,
 /* ---- model registry -----------------------------------------------------------------------
  * A model directory holds config.json and the weights; config.json's "architecture" names the model class:
  *   "Nufalorn"        bf16 models built from a list of layers (config.json: layers, width, vocab, norm, ...; *.safetensors)
+ *   "Vobunex"         another design of that kind: latent attention, Mamba-2, table-routed experts
  *   "Qwen3.5-hybrid"  the int4 hybrid above (config.json: the fields of lb_model_cfg; weight_index.bin, written over the
  *                     directory's *.safetensors files when missing)
  * The model is then driven through the same lb_model_* calls, whatever its class.  max_ctx: positions the caches hold.
