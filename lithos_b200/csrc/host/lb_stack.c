@@ -495,7 +495,7 @@ static int launch_rows(lb_model* m, lb_rows_gemv_params* p) {
     for (ks = 1; ks <= 1 + can_halve; ks++) {
         const int ctas = c->sm_count / ks, max_pairs = (P + ctas - 1) / ctas, segs = (p->segs + ks - 1) / ks;
         p->x_cols = ks == 1 ? p->K : segs * LB_RG_SEG;
-        p->split = max_pairs >= 64 ? 1 : segs;
+        p->split = max_pairs >= LB_RG_WARPS ? 1 : segs; /* pieces, each with its sum over the warp, only where warps would have no row pair at all */
         for (p->stages = 5; p->stages >= 1; p->stages--) {
             smem = (size_t)LB_RG_WARPS * p->stages * LB_RG_SEG * 4 + (size_t)n_vec * p->x_cols * 4 + (p->gate ? (size_t)((p->n_mix + 3) & ~3) * 4 : 0) +
                    (size_t)2 * max_pairs * p->split * 4 + 40 * 4 + ((size_t)LB_RG_WARPS * p->stages + 1) * 8;

@@ -5,7 +5,7 @@
 //
 // HBM-bound: one CTA per SM, every warp streams its own row segments with 1-D bulk copies through its own ring, so what is in flight
 // (ring bytes x 148) does not depend on registers.  Two rows share every read of the vector: shared memory moves 2 bytes of weights in,
-// 2 out and 2 bytes of vector per weight.  Narrow launches (few pairs per CTA, long rows) cut a pair into segments, one per warp turn;
+// 2 out and 2 bytes of vector per weight.  Narrow launches (fewer pairs than warps per CTA) cut a pair into segments, one per warp turn;
 // the segments of a pair are added in order, so a result does not depend on the schedule.  Where the vector is so long that it would leave
 // the ring too shallow, two CTAs (a cluster) take half of K each: half the vector to gather and to hold, and the sums of the two halves are
 // added, in order, through distributed shared memory.
